@@ -93,6 +93,12 @@ class PagedKVNeed:
       return 1 << 62
     return (first_page + 1) * page_size + (self.window - 1)
 
+  def covers(self, reader: "PagedKVNeed") -> bool:
+    """True if a cache with this need still holds, at every length, all that `reader` can see."""
+    if self.window is None:
+      return True
+    return type(reader) is PagedKVNeed and reader.window is not None and reader.window <= self.window
+
   def pool_pages(self, *, page_size: int, max_slots: int, max_seq_len: int, all_pages: int,
                  step_tokens: int, burst_tokens: int) -> int:
     """Pages the group's pool needs so that it never runs out before a pool that keeps every
@@ -104,6 +110,43 @@ class PagedKVNeed:
     if self.window is None:
       return all_pages
     per_slot = -(-(self.window - 1 + max(burst_tokens, 1)) // page_size) + 2
+    per_slot = min(per_slot, -(-max_seq_len // page_size))
+    return min(all_pages, max_slots * per_slot + -(-step_tokens // page_size))
+
+
+@dataclasses.dataclass(frozen=True)
+class ChunkedKVNeed(PagedKVNeed):
+  """Keys and values of the query's own chunk: with chunks of C tokens, counted from position 0,
+  position i sees the tokens from (i // C) * C on, so everything before the chunk of the next query
+  is given back.  `chunks` names the chunk sizes of all layers that read the cache; a page goes
+  when none of them can see it any more."""
+
+  chunks: tuple[int, ...] = ()
+
+  def group_key(self) -> tuple:
+    return ("chunks", tuple(sorted(set(self.chunks))))
+
+  def first_needed_page(self, lengths: np.ndarray, page_size: int) -> np.ndarray:
+    lengths = np.asarray(lengths, dtype=np.int64)
+    first = lengths
+    for size in self.chunks:
+      first = np.minimum(first, lengths // size * size)
+    return first // page_size
+
+  def first_needed_page_of(self, length: int, page_size: int) -> int:
+    return min(length // size * size for size in self.chunks) // page_size
+
+  def release_length(self, first_page: int, page_size: int) -> int | None:
+    # every reader's chunk has to start at or behind the end of the page
+    end = (first_page + 1) * page_size
+    return max(-(-end // size) * size for size in self.chunks)
+
+  def covers(self, reader: PagedKVNeed) -> bool:
+    return isinstance(reader, ChunkedKVNeed) and set(reader.chunks) <= set(self.chunks)
+
+  def pool_pages(self, *, page_size: int, max_slots: int, max_seq_len: int, all_pages: int,
+                 step_tokens: int, burst_tokens: int) -> int:
+    per_slot = -(-(max(self.chunks) + max(burst_tokens, 1)) // page_size) + 2
     per_slot = min(per_slot, -(-max_seq_len // page_size))
     return min(all_pages, max_slots * per_slot + -(-step_tokens // page_size))
 

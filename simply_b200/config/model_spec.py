@@ -49,6 +49,9 @@ class LayerCall:
   writes_cache: False for a call that only reads a cache another call wrote.
   add_embedding: True adds the embedding's output (the stream as it stood before the first
     layer) to the stream once more, right before this call.
+  mixer_cache: name of an earlier call's cache whose mixer's part this call's mixer reads without
+    writing it; the call still has a cache of its own for what the block itself keeps per request.
+    Both blocks' needs are dictionaries with the entry "mixer".
   stream_input: (name of one of the model's `stream_inputs`, pass number): that step rewrites the
     stream right before this call (it sees the embedding's output as well).
   """
@@ -57,6 +60,7 @@ class LayerCall:
   cache: str | None = None
   writes_cache: bool = True
   add_embedding: bool = False
+  mixer_cache: str | None = None
   stream_input: tuple[str, int] | None = None
 
 
@@ -96,6 +100,9 @@ class ModelSpec:
       if call.stream_input is not None and call.stream_input[0] not in self.stream_inputs:
         raise ValueError(f"layer call {call.layer!r} names the stream input {call.stream_input[0]!r}, "
                          "which the model does not define")
+      if call.mixer_cache is not None and call.mixer_cache not in written:
+        raise ValueError(f"layer call {call.layer!r} reads the mixer's cache of {call.mixer_cache!r}, "
+                         "but no earlier call writes it")
       if call.writes_cache:
         written.add(cache)
       elif cache not in written:

@@ -17,14 +17,21 @@ and a layer without a feed-forward has only the first line.
   h += mixer(norm(h)) + feed_forward(norm(h))
 With `branch_scales` each result is first multiplied by a learned factor per channel:
   h += s_mixer * mixer(norm(h)) + s_ff * feed_forward(norm(h))
+With a norm of its own for the feed-forward (`names["feed_forward_norm"]`) both still read the same h:
+  h += mixer(norm_1(h)) + feed_forward(norm_2(h))
+With `token_shift` the mixer reads, in place of y = norm_1(h), y + (y' - y) * shift with a learned
+factor per channel and y' the previous token's y (zeros before the first; the last y is part of
+a request's state).  The pending branches' adds, both norms and the shift are one kernel.
 """
 
 from __future__ import annotations
 
+import dataclasses
 from typing import Any
 
 import torch
 
+from simply_b200.cache.needs import SlotStateNeed
 from simply_b200.config.model_spec import PartSpec
 from simply_b200.parts.base import Block, FeedForward, Mixer, Norm, build_part
 from simply_b200.parts.feedforward import NoFeedForward
@@ -110,6 +117,18 @@ class ResidualStream:
     if self.lanes is not None:
       return self.read_lanes(self._ones(ctx), norm, ctx, rows)
     return self._combine(norm, ctx, rows)
+
+  def normed_twice(self, norm: Norm, norm2: Norm | None, shift: torch.Tensor | None, state: torch.Tensor | None,
+                   ctx: Any) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """(norm(h + pending), norm2(h + pending)) in the activation dtype; with `shift` (float32 [width]) the
+    first is moved towards the previous token's, whose last one `state` [slots, width] keeps (float32)."""
+    if self.lanes is not None or not isinstance(norm, RMSNorm) or not isinstance(norm2, (RMSNorm, type(None))):
+      raise TypeError("two norms of one stream in one kernel: RMS norms, and a stream that is kept once")
+    if self._post is not None or self._second_post is not None:
+      self.flush(ctx)
+    self.h, y, y2 = ctx.ops.residual_two_norms(self.h, self._branch, self._second, norm, norm2, shift, state, ctx)
+    self._branch = self._second = None
+    return y, y2
 
   def _ones(self, ctx: Any) -> torch.Tensor:
     key = ("stream_ones", self.lanes.shape[1])
@@ -229,9 +248,12 @@ class ParallelResidualBlock(Block):
   results are added to the stream."""
 
   def __init__(self, prefix: str, width: int, norm: PartSpec, mixer: Mixer, feed_forward: FeedForward,
-               names: dict[str, str] | None = None, branch_scales: dict[str, str] | None = None):
+               names: dict[str, str] | None = None, branch_scales: dict[str, str] | None = None,
+               token_shift: str | None = None):
     """`branch_scales`: {"mixer": name, "feed_forward": name}, tensors [width] after the layer's
-    prefix by which the sublayers' results are multiplied before they join the stream."""
+    prefix by which the sublayers' results are multiplied before they join the stream.
+    `names`: {"norm": name, "feed_forward_norm": name (only where the feed-forward has a norm of its
+    own)}.  `token_shift`: name of the tensor [width] of the shift's factors."""
     self.prefix = prefix
     self.mixer = mixer
     self.feed_forward = None if isinstance(feed_forward, NoFeedForward) else feed_forward
@@ -240,6 +262,14 @@ class ParallelResidualBlock(Block):
     if role is not None:
       params["name"] = f"{prefix}.{role}"  # the scale's whole tensor name
     self.norm = build_part(NORMS, PartSpec(norm.kind, f"{prefix}.norm", params))
+    self.width = width
+    self.shift_name = f"{prefix}.{token_shift}" if token_shift is not None else None
+    self.shift: torch.Tensor | None = None
+    role2 = (names or {}).get("feed_forward_norm")
+    self.two_norms = role2 is not None
+    self.feed_forward_norm = None
+    if self.two_norms:  # (a layer without a feed-forward does not use it, but its folder may hold it)
+      self.feed_forward_norm = build_part(NORMS, PartSpec(norm.kind, f"{prefix}.{role2}", {**params, "name": f"{prefix}.{role2}"}))
     scales = branch_scales or {}
     def scale(role: str):
       if role not in scales:
@@ -249,25 +279,45 @@ class ParallelResidualBlock(Block):
     self.feed_forward_scale = scale("feed_forward") if self.feed_forward is not None else None
 
   def _parts(self) -> list:
-    return [p for p in (self.mixer, self.feed_forward, self.norm, self.mixer_scale, self.feed_forward_scale)
+    second = self.feed_forward_norm if self.feed_forward is not None else None
+    return [p for p in (self.mixer, self.feed_forward, self.norm, second, self.mixer_scale, self.feed_forward_scale)
             if p is not None]
 
   def cache_need(self):
-    return self.mixer.cache_need()
+    if self.shift_name is None:
+      return self.mixer.cache_need()
+    needs = {"shift": SlotStateNeed((self.width,), "float32")}
+    if self.mixer.cache_need() is not None:
+      needs["mixer"] = self.mixer.cache_need()
+    return needs
 
   @property
   def graph_safe(self) -> bool:
     return all(p.graph_safe for p in self._parts())
 
   def tensor_specs(self) -> list[TensorSpec]:
-    return [s for p in self._parts() for s in p.tensor_specs()]
+    specs = [s for p in self._parts() for s in p.tensor_specs()]
+    if self.two_norms and self.feed_forward is None:
+      specs += [dataclasses.replace(s, optional=True) for s in self.feed_forward_norm.tensor_specs()]
+    if self.shift_name is not None:
+      specs.append(TensorSpec(self.shift_name, (self.width,), "scale", precision="stored"))
+    return specs
 
   def bind(self, tensors, ops) -> None:
     for p in self._parts():
       p.bind(tensors, ops)
+    if self.shift_name is not None:
+      self.shift = tensors[self.shift_name].float().contiguous()
 
   def forward(self, stream: ResidualStream, ctx: Any, cache: Any, writes_cache: bool = True) -> None:
-    y = stream.normed(self.norm, ctx)
+    if self.shift is None and not self.two_norms:
+      y = y2 = stream.normed(self.norm, ctx)
+    else:
+      state = None
+      if self.shift is not None:
+        state, cache = cache["shift"].storage, cache.get("mixer")
+      norm2 = self.feed_forward_norm if self.two_norms else self.norm
+      y, y2 = stream.normed_twice(self.norm, norm2 if self.feed_forward is not None else None, self.shift, state, ctx)
     stream.add(self.mixer.forward(y, ctx, cache, writes_cache), self.mixer_scale, ctx)
     if self.feed_forward is not None:
-      stream.add(self.feed_forward.forward(y, ctx), self.feed_forward_scale, ctx)
+      stream.add(self.feed_forward.forward(y2, ctx), self.feed_forward_scale, ctx)

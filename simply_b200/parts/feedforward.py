@@ -106,6 +106,32 @@ class LearnedActivationFeedForward(FeedForward):
     return self.down_proj(ctx.ops.linear_xielu(x, self.up_proj.weight, self.act, self.factors), ctx)
 
 
+@FEED_FORWARDS.register("activated")
+class ActivatedFeedForward(FeedForward):
+  """down(act(up(x))) without a gate, no biases.  `activation` "relu_squared": max(z, 0)^2."""
+
+  graph_safe = True
+
+  def __init__(self, prefix: str, width: int, hidden: int, activation: str = "relu_squared",
+               names: dict[str, str] | None = None):
+    if activation != "relu_squared":
+      raise ValueError(f"{prefix}: known activations without a gate: relu_squared")
+    names = names or {}
+    self.prefix, self.width, self.hidden = prefix, width, hidden
+    self.up_proj = Linear(f"{prefix}.{names.get('up', 'up')}", hidden, width)
+    self.down_proj = Linear(f"{prefix}.{names.get('down', 'down')}", width, hidden)
+
+  def tensor_specs(self) -> list[TensorSpec]:
+    return [self.up_proj.spec(), self.down_proj.spec()]
+
+  def bind(self, tensors, ops) -> None:
+    self.up_proj.bind(tensors)
+    self.down_proj.bind(tensors)
+
+  def forward(self, x: torch.Tensor, ctx: Any) -> torch.Tensor:
+    return self.down_proj(ctx.ops.linear_relu_squared(x, self.up_proj.weight), ctx)
+
+
 @FEED_FORWARDS.register("none")
 class NoFeedForward(FeedForward):
   """A layer without a feed-forward: block arrangements skip it."""

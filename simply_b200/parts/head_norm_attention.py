@@ -19,7 +19,15 @@ any of these, each switched by a parameter:
 * `projection_bias`: q, k and v each have a bias (tensor `<name>.b`), added in float32 to the
   projection before the rotation;
 * `distance_bias`: the score of query i and key j loses r1_h * log(1 + r2_h * (i - j)), with two
-  learned numbers per query head (tensors `r1`, `r2`), in float32.
+  learned numbers per query head (tensors `r1`, `r2`), in float32;
+* `distance_slopes`: the score loses slope_h * (i - j) with the fixed slopes 2^(-8 (h + 1) / heads);
+* `chunk` C (in place of a window): a query sees the keys of its own chunk only, from
+  (i // C) * C on, with chunks counted from the sequence's start;
+* `sink`: the softmax's denominator also holds exp(sink_h), a learned number per head without a key
+  or a value (tensor `sink`);
+* `project_kv=False`: the layer has no k and v tensors and reads the cache another layer writes.
+  `cache_chunks`: the chunk sizes of all layers that read this layer's cache (None among them: one
+  sees every token), which the cache has to serve.
 
 q, k, (v) and the gate come out of one fused product.
 """
@@ -30,14 +38,15 @@ from typing import Any
 
 import torch
 
-from simply_b200.cache.needs import PagedKVNeed
+from simply_b200.cache.needs import ChunkedKVNeed, PagedKVNeed
 from simply_b200.parts.base import Mixer
 from simply_b200.parts.linear import Linear, fuse_rows
 from simply_b200.parts.normed_attention import rotation_frequencies
 from simply_b200.registry import MIXERS
 from simply_b200.weights.loader import TensorSpec
 
-_NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "r1": "r1", "r2": "r2", "bias": "b"}
+_NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "r1": "r1", "r2": "r2", "bias": "b",
+          "sink": "sink"}
 
 
 @MIXERS.register("head_norm_attention")
@@ -49,7 +58,9 @@ class HeadNormAttention(Mixer):
                score_scale: float, eps: float, score_softcap: float = 0.0, window: int | None = None,
                rotary: dict | None = None, head_norm: bool = True, tie_values: bool = True,
                output_gate: bool = True, names: dict[str, str] | None = None, value_dim: int | None = None,
-               gate_per_head: bool = False, projection_bias: bool = False, distance_bias: bool = False):
+               gate_per_head: bool = False, projection_bias: bool = False, distance_bias: bool = False,
+               distance_slopes: bool = False, chunk: int | None = None, sink: bool = False, project_kv: bool = True,
+               cache_chunks: tuple = ()):
     if num_heads % num_kv_heads:
       raise ValueError(f"{prefix}: num_heads {num_heads} is no multiple of num_kv_heads {num_kv_heads}")
     self.prefix, self.width = prefix, width
@@ -68,30 +79,44 @@ class HeadNormAttention(Mixer):
     if self.tie_values and self.value_dim != head_dim:
       raise ValueError(f"{prefix}: tied values have the keys' size")
     self.gate_per_head, self.projection_bias = bool(gate_per_head), bool(projection_bias)
-    self.distance_bias = bool(distance_bias)
+    self.distance_bias, self.distance_slopes = bool(distance_bias), bool(distance_slopes)
+    if self.distance_bias and self.distance_slopes:
+      raise ValueError(f"{prefix}: a score loses one kind of distance term")
+    if chunk is not None and (window is not None or chunk <= 0):
+      raise ValueError(f"{prefix}: a chunk has a positive size and takes the place of a window")
+    self.chunk, self.has_sink, self.project_kv = chunk, bool(sink), bool(project_kv)
+    self.cache_chunks = tuple(cache_chunks)
+    if self.tie_values and not self.project_kv:
+      raise ValueError(f"{prefix}: tied values need a key projection")
     n = self.names = {**_NAMES, **(names or {})}
     self.q_proj = Linear(f"{prefix}.{n['q']}", num_heads * head_dim, width)
-    self.k_proj = Linear(f"{prefix}.{n['k']}", num_kv_heads * head_dim, width)
-    self.v_proj = None if self.tie_values else Linear(f"{prefix}.{n['v']}", num_kv_heads * self.value_dim, width)
+    self.k_proj = Linear(f"{prefix}.{n['k']}", num_kv_heads * head_dim, width) if self.project_kv else None
+    self.v_proj = None if self.tie_values or not self.project_kv else Linear(f"{prefix}.{n['v']}", num_kv_heads * self.value_dim, width)
     gate_rows = num_heads if self.gate_per_head else num_heads * self.value_dim
     self.g_proj = Linear(f"{prefix}.{n['g']}", gate_rows, width) if self.output_gate else None
     self.o_proj = Linear(f"{prefix}.{n['o']}", width, num_heads * self.value_dim)
-    self.in_weight = self.rot_freq = self.in_bias = self.distance = None
+    self.in_weight = self.rot_freq = self.in_bias = self.distance = self.sink = None
     self.gate_offset = 0
 
   def _inputs(self) -> list[Linear]:
     return [p for p in (self.q_proj, self.k_proj, self.v_proj, self.g_proj) if p is not None]
 
   def cache_need(self):
-    return PagedKVNeed(self.num_kv_heads, self.head_dim, self.window,
-                       value_dim=None if self.value_dim == self.head_dim else self.value_dim)
+    value_dim = None if self.value_dim == self.head_dim else self.value_dim
+    chunks = set(self.cache_chunks) | {self.chunk}
+    if None in chunks:
+      return PagedKVNeed(self.num_kv_heads, self.head_dim, self.window, value_dim=value_dim)
+    return ChunkedKVNeed(self.num_kv_heads, self.head_dim, value_dim=value_dim, chunks=tuple(sorted(chunks)))
 
   def graph_plans(self, ops, batch: int, bucket: int, max_burst: int, page_size: int) -> list:
+    opts: dict[str, Any] = {}  # (only what differs from the plain case)
+    if self.chunk is not None:
+      opts["key_chunk"] = self.chunk
     if self.value_dim != self.head_dim:
-      return []  # (the general kernel needs no list)
+      opts["value_dim"] = self.value_dim
     plan = ops.attention_graph_plan(
         window=self.window, num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, head_dim=self.head_dim,
-        batch=batch, bucket=bucket, max_burst=max_burst, page_size=page_size)
+        batch=batch, bucket=bucket, max_burst=max_burst, page_size=page_size, **opts)
     return [plan] if plan is not None else []
 
   def tensor_specs(self) -> list[TensorSpec]:
@@ -102,6 +127,8 @@ class HeadNormAttention(Mixer):
     if self.distance_bias:
       specs += [TensorSpec(f"{self.prefix}.{self.names[r]}", (self.num_heads,), "gain", precision="stored")
                 for r in ("r1", "r2")]
+    if self.has_sink:
+      specs.append(TensorSpec(f"{self.prefix}.{self.names['sink']}", (self.num_heads,), "scale", precision="stored"))
     return specs
 
   def _biased(self) -> list[Linear]:
@@ -110,6 +137,8 @@ class HeadNormAttention(Mixer):
   def bind(self, tensors, ops) -> None:
     if self.head_dim % 2 == 0 and self.value_dim == self.head_dim:  # (the general kernel takes the rest)
       ops.check_attention(self.head_dim, self.num_heads, self.num_kv_heads)
+    elif self.value_dim != self.head_dim:
+      ops.check_attention(self.head_dim, self.num_heads, self.num_kv_heads, self.value_dim)
     w = fuse_rows([tensors[p.name] for p in self._inputs()])
     extra = -w.shape[0] % 8  # whole 16-byte groups of output features for the products' stores
     self.in_weight = torch.cat([w, w.new_zeros(extra, w.shape[1])]).contiguous() if extra else w
@@ -119,6 +148,12 @@ class HeadNormAttention(Mixer):
       self.in_bias = torch.cat([tensors[f"{p.name}.{self.names['bias']}"].float() for p in self._biased()]).contiguous()
     if self.distance_bias:  # [2, heads]: r1, then r2
       self.distance = torch.stack([tensors[f"{self.prefix}.{self.names[r]}"].float() for r in ("r1", "r2")]).contiguous()
+    device = self.in_weight.device
+    if self.distance_slopes:  # [1, heads]
+      h = torch.arange(1, self.num_heads + 1, dtype=torch.float64)
+      self.distance = torch.exp2(-8.0 * h / self.num_heads).float()[None].to(device).contiguous()
+    if self.has_sink:
+      self.sink = tensors[f"{self.prefix}.{self.names['sink']}"].float().contiguous()
     if self.rotary:
       freq = rotation_frequencies(self.rotary["dims"], self.rotary["base"])
       self.rot_freq = torch.from_numpy(freq).to(self.in_weight.device)
@@ -139,17 +174,23 @@ class HeadNormAttention(Mixer):
       opts["value_dim"] = self.value_dim
     if self.distance is not None:
       opts["distance_bias"] = self.distance
+    if self.sink is not None:
+      opts["sink"] = self.sink
+    if self.chunk is not None:
+      opts["key_chunk"] = self.chunk
     return opts
 
   def forward(self, x: torch.Tensor, ctx: Any, cache: Any, writes_cache: bool = True) -> torch.Tensor:
     ops = ctx.ops
+    if writes_cache and not self.project_kv:
+      raise ValueError(f"{self.prefix}: a mixer without k/v projections cannot write a cache")
     block_table = ctx.block_tables[cache.group]
     proj = ops.linear(x, self.in_weight)  # q | k | (v) | (gate)
     q = ops.rotate_headnorm_store(
         proj, self.eps, self.score_scale, self.rot_freq,
         interleaved=bool(self.rotary) and self.rotary.get("layout", "neighbours") == "neighbours",
         head_norm=self.head_norm, tie_values=self.tie_values, num_heads=self.num_heads,
-        num_kv_heads=self.num_kv_heads, head_dim=self.head_dim,
+        num_kv_heads=self.num_kv_heads if self.project_kv else 0, head_dim=self.head_dim,
         storage=cache.storage if writes_cache else None, block_table=block_table, ctx=ctx,
         **self._store_options())
     o = ops.paged_attention(

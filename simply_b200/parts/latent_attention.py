@@ -10,10 +10,13 @@ Per token, from the mixer's input y:
   s   = scale * (q_plain . k_h + turn(q_rot) . k_r)
 
 over the keys that the window admits (`window` W: the token itself and the W - 1 before it), with
-a softmax whose denominator also holds exp(sink_h), a learned number per head that has no key and
-no value.  Head h's result is multiplied by sigmoid(W_g y)_h and the heads side by side go through
-W_o.  The rotation pairs dimension i of the rotated part with dimension i + dims/2 and turns them
-by position * base^(-2 i / dims).
+a softmax whose denominator also holds exp(sink_h) with `sink`, a learned number per head that has
+no key and no value.  With `output_gate` head h's result is multiplied by sigmoid(W_g y)_h
+(`gate_per_head`; else every element by a sigmoid of its own), and the heads side by side go
+through W_o.  The rotation (`rotary` = {dims, base, layout, scaling}) pairs dimension i of the rotated
+part with dimension i + dims/2 (`layout` "halves") or dimension 2i with 2i + 1 ("neighbours") and
+turns them by position times the pair's frequency (`scaled_frequencies`: base^(-2 i / dims), or
+YaRN's with `scaling`, whose factor on cosines and sines acts on queries and keys alike).
 
 The cache holds c and k_r only: one row of kv_rank + rotated_dim numbers per token.  Since
 q_plain . (W_uk,h c) = (W_uk,h^T q_plain) . c and sum_j p_j W_uv,h c_j = W_uv,h sum_j p_j c_j, every head
@@ -31,6 +34,7 @@ import torch
 from simply_b200.cache.needs import PagedKVNeed
 from simply_b200.parts.base import Mixer
 from simply_b200.parts.linear import Linear, fuse_rows
+from simply_b200.parts.position import scaled_frequencies
 from simply_b200.registry import MIXERS
 from simply_b200.weights.loader import TensorSpec
 
@@ -46,7 +50,7 @@ class LatentAttention(Mixer):
   def __init__(self, prefix: str, width: int, num_heads: int, head_dim: int, rotated_dim: int, value_dim: int,
                query_rank: int, kv_rank: int, score_scale: float, eps: float, rotary: dict | None = None,
                window: int | None = None, sink: bool = True, output_gate: bool = True,
-               names: dict[str, str] | None = None):
+               names: dict[str, str] | None = None, gate_per_head: bool = True):
     self.prefix, self.width = prefix, width
     self.num_heads, self.head_dim, self.rotated_dim, self.value_dim = num_heads, head_dim, rotated_dim, value_dim
     self.query_rank, self.kv_rank = query_rank, kv_rank
@@ -54,6 +58,13 @@ class LatentAttention(Mixer):
     self.window = window
     self.rot_dims = int(rotary["dims"]) if rotary else 0
     self.rot_base = float(rotary["base"]) if rotary else 1.0
+    self.rot_scaling = dict(rotary["scaling"]) if rotary and rotary.get("scaling") else None
+    layout = (rotary or {}).get("layout", "halves")
+    if layout not in ("neighbours", "halves"):
+      raise ValueError(f"{prefix}: rotary layout must be 'neighbours' or 'halves'")
+    # (only what differs from the plain case is passed on to the kernel table)
+    self.turn_options: dict[str, Any] = {"interleaved": True} if layout == "neighbours" else {}
+    self.gate_per_head = bool(gate_per_head)
     if self.rot_dims % 2 or self.rot_dims > rotated_dim:
       raise ValueError(f"{prefix}: the rotation takes an even number of dims, at most rotated_dim")
     self.has_sink, self.has_gate = bool(sink), bool(output_gate)
@@ -64,7 +75,8 @@ class LatentAttention(Mixer):
     self.kv_down = Linear(f"{p}.{n['kv_down']}", kv_rank + rotated_dim, width)
     self.key_up = Linear(f"{p}.{n['key_up']}", num_heads * head_dim, kv_rank)
     self.value_up = Linear(f"{p}.{n['value_up']}", num_heads * value_dim, kv_rank)
-    self.gate_proj = Linear(f"{p}.{n['gate']}", num_heads, width) if self.has_gate else None
+    gate_rows = num_heads if self.gate_per_head else num_heads * value_dim
+    self.gate_proj = Linear(f"{p}.{n['gate']}", gate_rows, width) if self.has_gate else None
     self.o_proj = Linear(f"{p}.{n['out']}", width, num_heads * value_dim)
     self.row_dim = kv_rank + rotated_dim  # what the cache holds per token
 
@@ -98,11 +110,12 @@ class LatentAttention(Mixer):
     self.query_norm = t[self._name("query_norm")].float().contiguous()
     self.kv_norm = t[self._name("kv_norm")].float().contiguous()
     self.sink = t[self._name("sink")].float().contiguous() if self.has_sink else None
-    half = self.rot_dims // 2
     self.freq = None
-    if half:
-      i = torch.arange(half, dtype=torch.float64)
-      self.freq = (self.rot_base ** (-2.0 * i / self.rot_dims)).to(torch.float32).to(self.query_norm.device)
+    if self.rot_dims:
+      freq, amplitude = scaled_frequencies(self.rot_dims, self.rot_base, self.rot_scaling)
+      self.freq = torch.from_numpy(freq).to(self.query_norm.device)
+      if amplitude != 1.0:
+        self.turn_options["amplitude"] = amplitude
 
   def forward(self, x: torch.Tensor, ctx: Any, cache: Any, writes_cache: bool = True) -> torch.Tensor:
     ops = ctx.ops
@@ -111,14 +124,15 @@ class LatentAttention(Mixer):
     # norms of both latents, the shared key part turned, the token's row into its page
     cq = ops.latent_prepare(down, self.query_norm, self.kv_norm, self.eps, self.freq, query_rank=self.query_rank,
                             kv_rank=self.kv_rank, rotated_dim=self.rotated_dim,
-                            storage=cache.storage if writes_cache else None, block_table=table, ctx=ctx)
+                            storage=cache.storage if writes_cache else None, block_table=table, ctx=ctx,
+                            **self.turn_options)
     q = ops.linear(cq, self.query_up.weight)
     asked = ops.latent_queries(q, self.key_up_t, self.freq, self.score_scale, ctx, num_heads=self.num_heads,
-                               head_dim=self.head_dim, rotated_dim=self.rotated_dim)
+                               head_dim=self.head_dim, rotated_dim=self.rotated_dim, **self.turn_options)
     mixed = ops.paged_attention(asked, cache.storage, table, ctx, num_heads=self.num_heads, num_kv_heads=1,
                                 head_dim=self.row_dim, logit_softcap=0.0, window=self.window,
                                 value_dim=self.kv_rank, values_in_keys=True, sink=self.sink)
     out = ops.head_linear(mixed, self.value_up_w)  # [T, heads * value_dim]
     if self.has_gate:
-      out = ops.sigmoid_gate(out, down, self.query_rank + self.row_dim, per=self.value_dim)
+      out = ops.sigmoid_gate(out, down, self.query_rank + self.row_dim, per=self.value_dim if self.gate_per_head else 1)
     return self.o_proj(out, ctx)

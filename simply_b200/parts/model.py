@@ -14,6 +14,7 @@ from typing import Any
 
 import torch
 
+from simply_b200.cache.needs import PagedKVNeed
 from simply_b200.config.model_spec import ModelSpec
 from simply_b200.parts.base import Block, build_part
 from simply_b200.parts.block import ResidualStream
@@ -24,6 +25,7 @@ from simply_b200.weights.loader import TensorSpec
 from simply_b200.parts import attention as _attention  # noqa: F401
 from simply_b200.parts import delta_rule as _delta_rule  # noqa: F401
 from simply_b200.parts import experts as _experts  # noqa: F401
+from simply_b200.parts import linear_attention as _linear_attention  # noqa: F401
 from simply_b200.parts import forget_gate as _forget_gate  # noqa: F401
 from simply_b200.parts import head_norm_attention as _head_norm_attention  # noqa: F401
 from simply_b200.parts import hyper_connection as _hyper_connection  # noqa: F401
@@ -90,24 +92,28 @@ class DecoderModel:
     needs: dict[str, Any] = {}
     for call, cache in zip(self.spec.run_order, self.cache_names):
       need = self.blocks[call.layer].cache_need()
+      if call.mixer_cache is not None:
+        self._check_reader(call.layer, call.mixer_cache, need["mixer"], needs[call.mixer_cache]["mixer"])
+        need = {key: part for key, part in need.items() if key != "mixer"}
       if call.writes_cache:
         if cache in needs and needs[cache] != need:
           raise ValueError(f"cache {cache!r} is written by calls with different needs")
         needs[cache] = need
     for call, cache in zip(self.spec.run_order, self.cache_names):
       if not call.writes_cache:
-        need, have = self.blocks[call.layer].cache_need(), needs[cache]
-        same = (type(need) is type(have)) and not isinstance(have, dict) and all(
-            getattr(need, f) == getattr(have, f) for f in ("num_kv_heads", "head_dim", "value_dim")
-            if hasattr(have, f))
-        if not same:
-          raise ValueError(f"layer {call.layer!r} cannot read cache {cache!r}: {need} vs {have}")
-        kept, wanted = getattr(have, "window", None), getattr(need, "window", None)
-        if kept is not None and (wanted is None or wanted > kept):
-          raise ValueError(
-              f"layer {call.layer!r} wants to see {wanted or 'all'} keys of cache {cache!r}, "
-              f"which keeps only a window of {kept}")
+        self._check_reader(call.layer, cache, self.blocks[call.layer].cache_need(), needs[cache])
     return needs
+
+  @staticmethod
+  def _check_reader(layer: str, cache: str, need: Any, have: Any) -> None:
+    """Refuses a layer that reads a cache of other shapes, or one that gives back what it needs."""
+    same = not isinstance(have, dict) and not isinstance(need, dict) and isinstance(have, PagedKVNeed) == isinstance(
+        need, PagedKVNeed) and all(
+            getattr(need, f) == getattr(have, f) for f in ("num_kv_heads", "head_dim", "value_dim") if hasattr(have, f))
+    if not same:
+      raise ValueError(f"layer {layer!r} cannot read cache {cache!r}: {need} vs {have}")
+    if isinstance(have, PagedKVNeed) and not have.covers(need):
+      raise ValueError(f"layer {layer!r} wants to see more keys of cache {cache!r} than it keeps: {need} vs {have}")
 
   # ---- forward --------------------------------------------------------------
   def forward(self, ctx: Any, caches: dict[str, Any]) -> torch.Tensor | None:
@@ -131,7 +137,10 @@ class DecoderModel:
       if call.stream_input is not None:
         name, index = call.stream_input
         self.stream_inputs[name].forward(stream, kept, index, ctx)
-      self.blocks[call.layer].forward(stream, ctx, caches.get(cache), call.writes_cache)
+      handle = caches.get(cache)
+      if call.mixer_cache is not None:
+        handle = {**(handle or {}), "mixer": caches[call.mixer_cache]["mixer"]}
+      self.blocks[call.layer].forward(stream, ctx, handle, call.writes_cache and call.mixer_cache is None)
       if layer_outputs is not None:
         layer_outputs.append(stream.total(ctx))
     if ctx.logit_rows.numel() == 0:

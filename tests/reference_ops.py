@@ -27,7 +27,7 @@ class ReferenceOps:
     self.name = "reference"
 
   # ---- checks ---------------------------------------------------------------
-  def check_attention(self, head_dim, num_heads, num_kv_heads):
+  def check_attention(self, head_dim, num_heads, num_kv_heads, value_dim=None):
     pass
 
   # ---- dense ----------------------------------------------------------------
@@ -137,6 +137,25 @@ class ReferenceOps:
     zn = torch.clamp(z, max=0.0)
     return torch.where(z > 0, ap * z * z + 0.5 * z, an * (torch.expm1(zn) - zn) + 0.5 * z).to(self.dtype)
 
+  def linear_relu_squared(self, x, w):
+    return torch.relu(self.linear(x, w).float()).pow(2).to(self.dtype)
+
+  def residual_two_norms(self, h, branch, branch2, norm, norm2, shift, state, ctx):
+    for b in (branch, branch2):
+      if b is not None:
+        h = h + b.float()
+    y = self._rms(h, norm.weight, norm.eps, norm.plus_one)
+    y2 = self._rms(h, norm2.weight, norm2.eps, norm2.plus_one).to(self.dtype) if norm2 is not None else None
+    if shift is not None:
+      before = torch.empty_like(y)
+      for b in range(ctx.num_seqs):
+        r0, r1, slot = (int(ctx.host["cu_q"][b]), int(ctx.host["cu_q"][b + 1]), int(ctx.host["slots"][b]))
+        before[r0] = state[slot]
+        before[r0 + 1:r1] = y[r0:r1 - 1]
+        state[slot] = y[r1 - 1]
+      y = y + (before - y) * shift
+    return h, y.to(self.dtype), y2
+
   def gather_rows(self, x, rows):
     return x[rows.long()].clone()
 
@@ -183,12 +202,12 @@ class ReferenceOps:
   # ---- attention ------------------------------------------------------------
   def paged_attention(self, q, storage, block_table, ctx, *, num_heads, num_kv_heads, head_dim,
                       logit_softcap, window, value_dim=None, pooled=None, values_in_keys=False, sink=None,
-                      distance_bias=None):
+                      distance_bias=None, key_chunk=None):
     if (pooled is not None or (value_dim is not None and value_dim != head_dim) or values_in_keys or sink is not None
-        or distance_bias is not None):
+        or distance_bias is not None or key_chunk is not None):
       assert not logit_softcap
       return self._general_attention(q, storage, block_table, ctx, num_heads, num_kv_heads, head_dim,
-                                     value_dim or head_dim, window, pooled, values_in_keys, sink, distance_bias)
+                                     value_dim or head_dim, window, pooled, values_in_keys, sink, distance_bias, key_chunk)
     t = q.shape[0]
     out = torch.zeros(t, num_heads, head_dim, dtype=torch.float32, device=q.device)
     group = num_heads // num_kv_heads
@@ -287,7 +306,7 @@ class ReferenceOps:
     return y.reshape(t, num_heads * dim).to(self.dtype)
 
   def _general_attention(self, q, storage, block_table, ctx, num_heads, num_kv_heads, head_dim, value_dim,
-                         window, pooled, values_in_keys=False, sink=None, distance_bias=None):
+                         window, pooled, values_in_keys=False, sink=None, distance_bias=None, key_chunk=None):
     t = q.shape[0]
     ps = ctx.page_size
     if values_in_keys:  # one row per entry: the key, whose first value_dim numbers are the value
@@ -304,6 +323,8 @@ class ReferenceOps:
       for r in range(r0, r1):
         i = start + r - r0
         lo = 0 if window is None else max(i - window + 1, 0)
+        if key_chunk is not None:  # the query's own chunk only
+          lo = i // key_chunk * key_chunk
         j = torch.arange(lo, i + 1, device=q.device)
         page = block_table[b, j // ps].long()
         assert (page >= 0).all(), "attention would read a page the request does not hold"
@@ -323,7 +344,10 @@ class ReferenceOps:
         for n in range(num_heads):
           m = n // group
           scores = k[:, m] @ q[r, n].float()
-          if distance_bias is not None:  # [2, heads]: the score loses r1 log(1 + r2 distance)
+          if distance_bias is not None and distance_bias.shape[0] == 1:  # [1, heads]: slope * distance
+            assert pooled is None
+            scores = scores - distance_bias[0, n] * (i - j).float()
+          elif distance_bias is not None:  # [2, heads]: the score loses r1 log(1 + r2 distance)
             assert pooled is None
             scores = scores - distance_bias[0, n] * torch.log1p(distance_bias[1, n] * (i - j).float())
           if sink is None:
@@ -391,6 +415,26 @@ class ReferenceOps:
       s = state[slot].clone()
       for r in range(r0, r1):
         s = f[r][:, :, None] * s + (1.0 - f[r])[:, :, None] * v[r][:, None, :]
+        out[r] = torch.einsum("hdv,hd->hv", s, q[r])
+      state[slot] = s
+    return out
+
+  # ---- gated linear attention -----------------------------------------------------
+  def gated_linear_scan(self, pre, low_offset, decay_out_t, decay_bias, tau, state, ctx, *, num_heads, head_dim,
+                        value_dim):
+    t, n = pre.shape[0], num_heads * head_dim
+    q = (pre[:, :n].float() * head_dim ** -0.5).reshape(t, num_heads, head_dim)
+    k = pre[:, n:2 * n].float().reshape(t, num_heads, head_dim)
+    v = pre[:, 2 * n:2 * n + num_heads * value_dim].float().reshape(t, num_heads, value_dim)
+    z = pre[:, low_offset:low_offset + decay_out_t.shape[0]].float() @ decay_out_t + decay_bias
+    keep = torch.exp(torch.nn.functional.logsigmoid(z) / tau).reshape(t, num_heads, head_dim)
+    out = torch.empty(t, num_heads, value_dim, dtype=torch.float32, device=pre.device)
+    for b in range(ctx.num_seqs):
+      r0, r1 = int(ctx.host["cu_q"][b]), int(ctx.host["cu_q"][b + 1])
+      slot = int(ctx.host["slots"][b])
+      s = state[slot].clone()
+      for r in range(r0, r1):
+        s = keep[r][:, :, None] * s + k[r][:, :, None] * v[r][:, None, :]
         out[r] = torch.einsum("hdv,hd->hv", s, q[r])
       state[slot] = s
     return out
@@ -484,13 +528,14 @@ class ReferenceOps:
         state[slot, n] = s
     return out
 
-  def gated_head_norm(self, o, low, gate_offset, weight, eps, num_heads, value_dim):
+  def gated_head_norm(self, o, low, gate_offset, weight, eps, num_heads, value_dim, gate="sigmoid"):
     t = o.shape[0]
     y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * weight.float()[None, None, :]
     if low is None:
       return y.reshape(t, num_heads * value_dim).to(self.dtype)
-    gate = torch.sigmoid(low[:, gate_offset:gate_offset + num_heads * value_dim].float())
-    return (y.reshape(t, num_heads * value_dim) * gate).to(self.dtype)
+    g = low[:, gate_offset:gate_offset + num_heads * value_dim].float()
+    g = torch.sigmoid(g) * (g if gate == "silu" else 1.0)
+    return (y.reshape(t, num_heads * value_dim) * g).to(self.dtype)
 
   def normed_mean(self, branches, scales, eps):
     total = 0
@@ -551,24 +596,33 @@ class ReferenceOps:
 
   # ---- attention over latents -----------------------------------------------------------
   @staticmethod
-  def _turn_part(x, positions, freq):
-    """Dims i and i + n of the first 2n dims of x [T, ..., D] turn by positions * freq[i]."""
+  def _turn_part(x, positions, freq, interleaved=False, amplitude=1.0):
+    """Dims i and i + n (interleaved: 2i and 2i + 1) of the first 2n dims of x [T, ..., D] turn by
+    positions * freq[i]."""
+    if freq is not None and interleaved:
+      n = freq.numel()
+      order = list(range(0, 2 * n, 2)) + list(range(1, 2 * n, 2)) + list(range(2 * n, x.shape[-1]))
+      turned = ReferenceOps._turn_part(x[..., order], positions, freq, False, amplitude)
+      out = torch.empty_like(turned)
+      out[..., order] = turned
+      return out
     if freq is None:
       return x
     n = freq.numel()
     angle = positions.float()[:, None] * freq.float()[None, :]
     while angle.dim() < x.dim():
       angle = angle[:, None]
-    c, s = torch.cos(angle), torch.sin(angle)
+    c, s = amplitude * torch.cos(angle), amplitude * torch.sin(angle)
     a, b = x[..., :n], x[..., n:2 * n]
     return torch.cat([a * c - b * s, b * c + a * s, x[..., 2 * n:]], dim=-1)
 
   def latent_prepare(self, down, query_norm, kv_norm, eps, freq, *, query_rank, kv_rank, rotated_dim, storage,
-                     block_table, ctx):
+                     block_table, ctx, interleaved=False, amplitude=1.0):
     d = down.float()
     cq = self._rms(d[:, :query_rank], query_norm, eps, False)
     c = self._rms(d[:, query_rank:query_rank + kv_rank], kv_norm, eps, False)
-    kr = self._turn_part(d[:, query_rank + kv_rank:query_rank + kv_rank + rotated_dim], ctx.positions, freq)
+    kr = self._turn_part(d[:, query_rank + kv_rank:query_rank + kv_rank + rotated_dim], ctx.positions, freq,
+                         interleaved, amplitude)
     if storage is not None:
       ps = ctx.page_size
       pos = ctx.positions.long()
@@ -578,11 +632,12 @@ class ReferenceOps:
       rows[page, pos % ps] = torch.cat([c, kr], dim=1).to(storage.dtype)
     return cq.to(self.dtype)
 
-  def latent_queries(self, q, key_up_t, freq, scale, ctx, *, num_heads, head_dim, rotated_dim):
+  def latent_queries(self, q, key_up_t, freq, scale, ctx, *, num_heads, head_dim, rotated_dim, interleaved=False,
+                     amplitude=1.0):
     t = q.shape[0]
     qh = q.float().reshape(t, num_heads, head_dim + rotated_dim)
     plain = torch.einsum("thd,hrd->thr", qh[..., :head_dim], key_up_t.float())
-    turned = self._turn_part(qh[..., head_dim:], ctx.positions, freq)
+    turned = self._turn_part(qh[..., head_dim:], ctx.positions, freq, interleaved, amplitude)
     return (torch.cat([plain, turned], dim=-1) * scale).reshape(t, -1).to(self.dtype)
 
   def head_linear(self, x, w):
