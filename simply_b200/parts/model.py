@@ -113,7 +113,8 @@ class DecoderModel:
     if not same:
       raise ValueError(f"layer {layer!r} cannot read cache {cache!r}: {need} vs {have}")
     if isinstance(have, PagedKVNeed) and not have.covers(need):
-      raise ValueError(f"layer {layer!r} wants to see more keys of cache {cache!r} than it keeps: {need} vs {have}")
+      kept = f"a window of {have.window}" if have.window is not None else f"what {have} sees"
+      raise ValueError(f"layer {layer!r} wants to see {need.window or 'all'} keys of cache {cache!r}, which keeps only {kept}")
 
   # ---- forward --------------------------------------------------------------
   def forward(self, ctx: Any, caches: dict[str, Any]) -> torch.Tensor | None:
