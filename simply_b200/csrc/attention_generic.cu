@@ -20,7 +20,9 @@
 // head_dim numbers whose first v_dim are its value as well (a cache of latents; a page then holds
 // key rows only).  `sink`: one learned number per query head whose exponential joins the softmax's
 // denominator; it has no key and no value.  `distance`: two learned numbers r1, r2 per query head
-// ([2, heads]); the score of query i and key j loses r1 * log(1 + r2 * (i - j)) (float32, log1pf).
+// ([2, heads]); the score of query i and key j loses r1 * log(1 + r2 * (i - j)) (float32, log1pf);
+// with `linear` one number r1 per head ([heads]), and the score loses r1 * (i - j).  `chunk` C (without
+// a window): a query sees the keys from (i / C) * C on, its own chunk's.
 //
 // This is the true 32-bit path's attention and the fallback of the bfloat16
 // path for shapes its tensor-core kernels refuse.
@@ -121,9 +123,10 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ ca
                                int head_dim, int v_dim, int page_size, int num_pages, float cap, int window,
                                const T* __restrict__ pool, const int* __restrict__ pool_table,
                                int pool_max_pages, int pool_len, int pool_pages, int tied,
-                               const float* __restrict__ sink, const float* __restrict__ distance, int* err) {
+                               const float* __restrict__ sink, const float* __restrict__ distance, int linear,
+                               int chunk, int* err) {
   const float r1 = distance != nullptr ? distance[blockIdx.x % num_q_heads] : 0.f;  // (weights: before the wait)
-  const float r2 = distance != nullptr ? distance[num_q_heads + blockIdx.x % num_q_heads] : 0.f;
+  const float r2 = distance != nullptr && !linear ? distance[num_q_heads + blockIdx.x % num_q_heads] : 0.f;
   pdl_wait_block();
   pdl_launch_dependents();
   // head_dim floats of q, then per warp its running maximum, sum and v_dim partial results
@@ -139,7 +142,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ ca
   for (int d = threadIdx.x; d < head_dim; d += blockDim.x) qs[d] = to_f32<T>(qp[d]);
   __syncthreads();
 
-  const int lo = window > 0 ? max(pos - window + 1, 0) : 0;
+  const int lo = window > 0 ? max(pos - window + 1, 0) : chunk > 0 ? pos / chunk * chunk : 0;
   float m_run = -0.5f * FLT_MAX, l_run = 0.f;
   float acc[GEN_MAX_DPL];
 #pragma unroll
@@ -186,7 +189,8 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ ca
         vr = tied ? kr : cache + page * page_stride + value_base + row * v_dim;
       }
     }
-    const float minus = distance != nullptr && j <= pos ? r1 * log1pf(r2 * (float)(pos - j)) : 0.f;
+    float minus = 0.f;
+    if (distance != nullptr && j <= pos) minus = r1 * (linear ? (float)(pos - j) : log1pf(r2 * (float)(pos - j)));
     gen_tile<T>(kr, vr, qs, head_dim, v_dim, cap, minus, lane, m_run, l_run, acc);
   }
   // The warps' parts meet in warp order (the same order whatever the step holds).
@@ -229,10 +233,11 @@ extern "C" int sb_paged_attention_general(const void* q, int dtype, const void* 
                                           int head_dim, int v_dim, int page_size, int num_pages, float cap,
                                           int window, const void* pool, const int* pool_table,
                                           int pool_max_pages, int pool_len, int pool_pages, int tied,
-                                          const float* sink, const float* distance, int* err,
-                                          cudaStream_t stream) {
+                                          const float* sink, const float* distance, int linear, int chunk,
+                                          int* err, cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (distance != nullptr && pool != nullptr) return -13;
+  if (chunk > 0 && (pool != nullptr || window > 0)) return -13;
   if (tied && (pool != nullptr || v_dim > head_dim)) return -13;
   // (the values' sums live in registers, GEN_MAX_DPL per lane; a key row only passes through)
   if (head_dim <= 0 || head_dim > 4096 || v_dim <= 0 || v_dim > 32 * GEN_MAX_DPL) return -7;
@@ -245,12 +250,12 @@ extern "C" int sb_paged_attention_general(const void* q, int dtype, const void* 
     sb_launch(paged_attention_generic_kernel<float>, blocks, GEN_WARPS * 32, smem, stream, (const float*)q,
         (const float*)cache, block_table, max_pages, token_seq, positions, (float*)out, num_tokens,
         num_q_heads, num_kv_heads, head_dim, v_dim, page_size, num_pages, cap, window, (const float*)pool, pool_table,
-        pool_max_pages, pool_len, pool_pages, tied, sink, distance, err);
+        pool_max_pages, pool_len, pool_pages, tied, sink, distance, linear, chunk, err);
   else
     sb_launch(paged_attention_generic_kernel<bf16>, blocks, GEN_WARPS * 32, smem, stream, (const bf16*)q,
         (const bf16*)cache, block_table, max_pages, token_seq, positions, (bf16*)out, num_tokens,
         num_q_heads, num_kv_heads, head_dim, v_dim, page_size, num_pages, cap, window, (const bf16*)pool, pool_table,
-        pool_max_pages, pool_len, pool_pages, tied, sink, distance, err);
+        pool_max_pages, pool_len, pool_pages, tied, sink, distance, linear, chunk, err);
   SB_LAUNCH_CHECK();
   return 0;
 }
@@ -262,5 +267,5 @@ extern "C" int sb_paged_attention_generic(const void* q, int dtype, const void* 
                                           int* err, cudaStream_t stream) {
   return sb_paged_attention_general(q, dtype, cache, block_table, max_pages, token_seq, positions, out, num_tokens,
                                     num_q_heads, num_kv_heads, head_dim, head_dim, page_size, num_pages, cap,
-                                    window, nullptr, nullptr, 0, 0, 0, 0, nullptr, nullptr, err, stream);
+                                    window, nullptr, nullptr, 0, 0, 0, 0, nullptr, nullptr, 0, 0, err, stream);
 }

@@ -111,6 +111,20 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   return scratch[32];
 }
 
+// A decode graph pads its batch by repeating the last request's row.  What such a row computes must not
+// depend on whether the slot's state has been written meanwhile, so the first row of a slot does the
+// work of all: returns how many rows (one token each, next to one another) share row b's slot, or 0
+// when an earlier row does.  Called by whole warps.
+__device__ __forceinline__ int rows_sharing_slot(const int* slots, int b, int num_seqs) {
+  const int slot = slots[b], lane = threadIdx.x & 31;
+  bool earlier = false;
+  for (int i = lane; i < b; i += 32) earlier |= slots[i] == slot;
+  if (__any_sync(0xffffffffu, earlier)) return 0;
+  int later = 0;
+  for (int i = b + 1 + lane; i < num_seqs; i += 32) later += slots[i] == slot ? 1 : 0;
+  return 1 + __reduce_add_sync(0xffffffffu, later);
+}
+
 // Programmatic dependent launch.  Every kernel of the engine begins with
 // `pdl_wait(); pdl_launch_dependents();` (or does work that depends on nothing written by
 // earlier kernels, such as fetching weights, before the two).  The wait blocks until every

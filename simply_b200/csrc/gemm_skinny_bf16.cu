@@ -227,6 +227,9 @@ skinny_gemm_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, void*
         // Round to bfloat16 first, as the unfused path stores the product before it activates.
         z = __bfloat162float(__float2bfloat16_rn(z));
         z = z > 0.f ? fmaf(cap * z, z, 0.5f * z) : fmaf(rs.act_b, expm1f(z) - z, 0.5f * z);
+      } else if (act == 6) {
+        z = fmaxf(__bfloat162float(__float2bfloat16_rn(z)), 0.f);
+        z *= z;
       }
       reinterpret_cast<bf16*>(out)[o] = __float2bfloat16_rn(z);
     } else if (EPI == 1) {
@@ -322,6 +325,12 @@ extern "C" int sb_gemm_skinny_bf16_xielu(const void* x, const void* w, void* out
   RopeStore rs{};
   rs.act_b = b;
   return skinny_dispatch(x, w, out, M, N, K, 0, a, 5, warps_override, stream, rs);
+}
+
+// max(x . w^T, 0)^2, stored as bfloat16.
+extern "C" int sb_gemm_skinny_bf16_relu_squared(const void* x, const void* w, void* out, int M, int N, int K,
+                                                int warps_override, cudaStream_t stream) {
+  return skinny_dispatch(x, w, out, M, N, K, 0, 0.f, 6, warps_override, stream, RopeStore{});
 }
 
 // The fused q, k, v projection of an attention layer for at most 16 tokens: product, rotation,

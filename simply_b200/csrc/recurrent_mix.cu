@@ -217,6 +217,8 @@ delta_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
     if (threadIdx.x == 0) atomicOr(err, SB_ERR_BAD_SLOT);
     return;
   }
+  const int copies = rows_sharing_slot(slots, b, gridDim.y);
+  if (copies == 0) return;  // an earlier row of the slot does this row's work
   const int g_head = h / (H / G);
   const int cols_pad = (cols + 3) & ~3;
   const int buffer = SCAN_CHUNK * (3 * d + cols_pad + 4);
@@ -354,11 +356,12 @@ delta_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, cons
 #pragma unroll
         for (int o = 1; o < RS; o <<= 1) od += __shfl_xor_sync(0xffffffffu, od, o);
       }
-      if (on && rs == 0) out[((size_t)(first + base + i) * H + h) * dv + col] = od;
+      if (on && rs == 0)
+        for (int c = 0; c < copies; ++c) out[((size_t)(first + base + i + c) * H + h) * dv + col] = od;
     }
     __syncthreads();  // the buffer is filled again two chunks on
   }
-  if (on && first_row_of_slot(slots, b)) {
+  if (on) {
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
       const int row = VEC ? 4 * (rs + RS * (r >> 2)) + (r & 3) : rs + RS * r;
@@ -461,14 +464,16 @@ forget_inputs_kernel(const T* __restrict__ pre, int row_width, const float* __re
   if (c < n_v) v[(size_t)t * n_v + c] = to_f32<T>(x[2 * n_qf + c]);
 }
 
-template <int RS, int ROWS, bool VEC>
+// KINDS 2: qf holds q and f, and the state takes in (1 - f) v^T.  KINDS 3: q, f and k (gated linear
+// attention), and it takes in k v^T.
+template <int RS, int ROWS, bool VEC, int KINDS>
 __global__ void __launch_bounds__(256)
 forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, float* __restrict__ state,
                    const int* __restrict__ cu_q, const int* __restrict__ slots, int num_slots, int H, int d, int dv,
                    int cols, int nbuf, float* __restrict__ out, int* err) {
   pdl_wait_block();
   pdl_launch_dependents();
-  // A ring of nbuf (2 or 4) buffers of: q [CHUNK][d], f [CHUNK][d], v [CHUNK][cols_pad].
+  // A ring of nbuf (2 or 4) buffers of: q [CHUNK][d], f [CHUNK][d], (k [CHUNK][d],) v [CHUNK][cols_pad].
   extern __shared__ __align__(16) float stage[];
   const int h = blockIdx.x, b = blockIdx.y, col0 = blockIdx.z * cols;
   const int rs = threadIdx.x % RS, col_local = threadIdx.x / RS;
@@ -480,8 +485,10 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
     if (threadIdx.x == 0) atomicOr(err, SB_ERR_BAD_SLOT);
     return;
   }
+  const int copies = rows_sharing_slot(slots, b, gridDim.y);
+  if (copies == 0) return;  // an earlier row of the slot does this row's work
   const int cols_pad = (cols + 3) & ~3;
-  const int buffer = FORGET_CHUNK * (2 * d + cols_pad);
+  const int buffer = FORGET_CHUNK * (KINDS * d + cols_pad);
   const int n_qf = H * d;
 
   auto issue = [&](int which, int base) {
@@ -489,19 +496,19 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
     const int count = min(FORGET_CHUNK, n - base);
     if (VEC) {
       const int d4 = d >> 2;
-      for (int idx = threadIdx.x; idx < count * 2 * d4; idx += blockDim.x) {
-        const int i = idx / (2 * d4), rem = idx - i * 2 * d4, kind = rem / d4, c = (rem - kind * d4) * 4;
+      for (int idx = threadIdx.x; idx < count * KINDS * d4; idx += blockDim.x) {
+        const int i = idx / (KINDS * d4), rem = idx - i * KINDS * d4, kind = rem / d4, c = (rem - kind * d4) * 4;
         scan_copy16(buf + (kind * FORGET_CHUNK + i) * d + c,
-                    qf + ((size_t)(first + base + i) * 2 + kind) * n_qf + h * d + c);
+                    qf + ((size_t)(first + base + i) * KINDS + kind) * n_qf + h * d + c);
       }
     } else {
-      for (int idx = threadIdx.x; idx < count * 2 * d; idx += blockDim.x) {
-        const int i = idx / (2 * d), rem = idx - i * 2 * d, kind = rem / d, c = rem - kind * d;
+      for (int idx = threadIdx.x; idx < count * KINDS * d; idx += blockDim.x) {
+        const int i = idx / (KINDS * d), rem = idx - i * KINDS * d, kind = rem / d, c = rem - kind * d;
         scan_copy4(buf + (kind * FORGET_CHUNK + i) * d + c,
-                   qf + ((size_t)(first + base + i) * 2 + kind) * n_qf + h * d + c);
+                   qf + ((size_t)(first + base + i) * KINDS + kind) * n_qf + h * d + c);
       }
     }
-    float* bv = buf + 2 * FORGET_CHUNK * d;
+    float* bv = buf + KINDS * FORGET_CHUNK * d;
     for (int idx = threadIdx.x; idx < count * cols; idx += blockDim.x) {
       const int i = idx / cols, c = idx - i * cols;
       scan_copy4(bv + i * cols_pad + c, v + ((size_t)(first + base + i) * H + h) * dv + min(col0 + c, dv - 1));
@@ -537,7 +544,7 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
       // Several tokens at a time: a row's state goes through their updates in one chain of
       // multiply-adds, the sums that read it are chains of their own, and their sums over lanes go
       // side by side, so that a token's latencies are paid once per group of tokens.
-      const float* vbuf = buf + 2 * FORGET_CHUNK * d + min(col_local, cols - 1);
+      const float* vbuf = buf + KINDS * FORGET_CHUNK * d + min(col_local, cols - 1);
       for (; i + FORGET_TOGETHER <= count; i += FORGET_TOGETHER) {
         float od4[FORGET_TOGETHER], vv4[FORGET_TOGETHER];
 #pragma unroll
@@ -553,10 +560,12 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
             for (int t = 0; t < FORGET_TOGETHER; ++t) {
               const float4 f4 = reinterpret_cast<const float4*>(buf + (FORGET_CHUNK + i + t) * d)[at];
               const float4 q4 = reinterpret_cast<const float4*>(buf + (i + t) * d)[at];
-              s[4 * r] = fmaf(f4.x, s[4 * r], (1.0f - f4.x) * vv4[t]);
-              s[4 * r + 1] = fmaf(f4.y, s[4 * r + 1], (1.0f - f4.y) * vv4[t]);
-              s[4 * r + 2] = fmaf(f4.z, s[4 * r + 2], (1.0f - f4.z) * vv4[t]);
-              s[4 * r + 3] = fmaf(f4.w, s[4 * r + 3], (1.0f - f4.w) * vv4[t]);
+              const float4 k4 = KINDS == 3 ? reinterpret_cast<const float4*>(buf + (2 * FORGET_CHUNK + i + t) * d)[at]
+                                           : make_float4(1.0f - f4.x, 1.0f - f4.y, 1.0f - f4.z, 1.0f - f4.w);
+              s[4 * r] = fmaf(f4.x, s[4 * r], k4.x * vv4[t]);
+              s[4 * r + 1] = fmaf(f4.y, s[4 * r + 1], k4.y * vv4[t]);
+              s[4 * r + 2] = fmaf(f4.z, s[4 * r + 2], k4.z * vv4[t]);
+              s[4 * r + 3] = fmaf(f4.w, s[4 * r + 3], k4.w * vv4[t]);
               od4[t] = fmaf(s[4 * r], q4.x, od4[t]);
               od4[t] = fmaf(s[4 * r + 1], q4.y, od4[t]);
               od4[t] = fmaf(s[4 * r + 2], q4.z, od4[t]);
@@ -570,7 +579,7 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
           for (int t = 0; t < FORGET_TOGETHER; ++t) od4[t] += __shfl_xor_sync(0xffffffffu, od4[t], o);
         }
         if (on && rs == 0) {
-          float* dst = out + ((size_t)(first + base + i) * H + h) * dv + col;
+          float* dst = out + ((size_t)(first + base + i) * H + h) * dv + col;  // (a row of eight tokens has no copy)
 #pragma unroll
           for (int t = 0; t < FORGET_TOGETHER; ++t) dst[(size_t)t * H * dv] = od4[t];
         }
@@ -579,7 +588,7 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
     for (; i < count; ++i) {
       const float* qq = buf + i * d;
       const float* ff = buf + (FORGET_CHUNK + i) * d;
-      const float vv = buf[2 * FORGET_CHUNK * d + i * cols_pad + min(col_local, cols - 1)];
+      const float vv = buf[KINDS * FORGET_CHUNK * d + i * cols_pad + min(col_local, cols - 1)];
       float od;
       if constexpr (VEC) {
         float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
@@ -589,10 +598,12 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
           if (4 * at < d) {
             const float4 f4 = reinterpret_cast<const float4*>(ff)[at];
             const float4 q4 = reinterpret_cast<const float4*>(qq)[at];
-            s[4 * r] = fmaf(f4.x, s[4 * r], (1.0f - f4.x) * vv); o0 = fmaf(s[4 * r], q4.x, o0);
-            s[4 * r + 1] = fmaf(f4.y, s[4 * r + 1], (1.0f - f4.y) * vv); o1 = fmaf(s[4 * r + 1], q4.y, o1);
-            s[4 * r + 2] = fmaf(f4.z, s[4 * r + 2], (1.0f - f4.z) * vv); o2 = fmaf(s[4 * r + 2], q4.z, o2);
-            s[4 * r + 3] = fmaf(f4.w, s[4 * r + 3], (1.0f - f4.w) * vv); o3 = fmaf(s[4 * r + 3], q4.w, o3);
+            const float4 k4 = KINDS == 3 ? reinterpret_cast<const float4*>(buf + (2 * FORGET_CHUNK + i) * d)[at]
+                                         : make_float4(1.0f - f4.x, 1.0f - f4.y, 1.0f - f4.z, 1.0f - f4.w);
+            s[4 * r] = fmaf(f4.x, s[4 * r], k4.x * vv); o0 = fmaf(s[4 * r], q4.x, o0);
+            s[4 * r + 1] = fmaf(f4.y, s[4 * r + 1], k4.y * vv); o1 = fmaf(s[4 * r + 1], q4.y, o1);
+            s[4 * r + 2] = fmaf(f4.z, s[4 * r + 2], k4.z * vv); o2 = fmaf(s[4 * r + 2], q4.z, o2);
+            s[4 * r + 3] = fmaf(f4.w, s[4 * r + 3], k4.w * vv); o3 = fmaf(s[4 * r + 3], q4.w, o3);
           }
         }
         od = (o0 + o1) + (o2 + o3);
@@ -603,19 +614,21 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
           const int row = rs + RS * r;
           if (row < d) {
             const float f = ff[row];
-            s[r] = fmaf(f, s[r], (1.0f - f) * vv);
+            const float take = KINDS == 3 ? buf[(2 * FORGET_CHUNK + i) * d + row] : 1.0f - f;
+            s[r] = fmaf(f, s[r], take * vv);
             od = fmaf(s[r], qq[row], od);
           }
         }
       }
 #pragma unroll
       for (int o = 1; o < RS; o <<= 1) od += __shfl_xor_sync(0xffffffffu, od, o);
-      if (on && rs == 0) out[((size_t)(first + base + i) * H + h) * dv + col] = od;
+      if (on && rs == 0)
+        for (int c = 0; c < copies; ++c) out[((size_t)(first + base + i + c) * H + h) * dv + col] = od;
     }
     __syncthreads();  // the buffer is filled again in the next round
   }
   asm volatile("cp.async.wait_group 0;\n" ::);
-  if (on && first_row_of_slot(slots, b)) {
+  if (on) {
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
       const int row = VEC ? 4 * (rs + RS * (r >> 2)) + (r & 3) : rs + RS * r;
@@ -624,24 +637,11 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
   }
 }
 
-// scratch: float32 [T, 2 H d + H dv] for the inputs.
-extern "C" int sb_forget_scan(const void* pre, int row_width, int dtype, const float* bias, const float* lower,
-                              float* state, const int* cu_q, const int* slots, int num_tokens, int num_seqs,
-                              int num_slots, int H, int d, int dv, int max_q_len, float* scratch, float* out,
-                              int* err, cudaStream_t stream) {
-  if (num_seqs == 0 || num_tokens == 0) return 0;
-  if (d <= 0 || d > 32 * 32 || dv <= 0 || H <= 0) return -13;
-  float* qf = scratch;
-  float* v = scratch + (size_t)num_tokens * 2 * H * d;
-  const int widest = H * d > H * dv ? H * d : H * dv;
-  const dim3 in_grid((unsigned)num_tokens, (unsigned)((widest + 255) / 256));
-  if (dtype == SB_DTYPE_F32)
-    sb_launch(forget_inputs_kernel<float>, in_grid, 256, 0, stream, (const float*)pre, row_width, bias, lower,
-              H * d, H * dv, qf, v);
-  else
-    sb_launch(forget_inputs_kernel<bf16>, in_grid, 256, 0, stream, (const bf16*)pre, row_width, bias, lower,
-              H * d, H * dv, qf, v);
-  SB_LAUNCH_CHECK();
+// The walk over float32 inputs qf [T, KINDS, H d] and v [T, H dv].
+template <int KINDS>
+static int launch_forget_scan(const float* qf, const float* v, float* state, const int* cu_q, const int* slots,
+                              int num_seqs, int num_slots, int H, int d, int dv, int max_q_len, float* out, int* err,
+                              cudaStream_t stream) {
   const bool vec = d % 4 == 0;
   const int rows = (vec && d <= 8 * 32) ? 8 : 32;
   int rs = 1;
@@ -655,21 +655,21 @@ extern "C" int sb_forget_scan(const void* pre, int row_width, int dtype, const f
   if (cols > dv) cols = dv;
   const int block = ((cols * rs + 31) / 32) * 32;
   const dim3 grid(H, num_seqs, (dv + cols - 1) / cols);
-  const size_t one = (size_t)FORGET_CHUNK * (2 * d + ((cols + 3) & ~3)) * sizeof(float);
+  const size_t one = (size_t)FORGET_CHUNK * (KINDS * d + ((cols + 3) & ~3)) * sizeof(float);
   const int nbuf = (max_q_len > 2 * FORGET_CHUNK && 4 * one <= 100 * 1024) ? 4 : 2;
   const size_t smem = nbuf * one;
   if (smem > 200 * 1024) return -13;
-#define SB_FORGET_V(RS_, ROWS_, VEC_)                                                                          \
-  do {                                                                                                         \
-    if (smem > 48 * 1024)                                                                                      \
-      cudaFuncSetAttribute(forget_scan_kernel<RS_, ROWS_, VEC_>, cudaFuncAttributeMaxDynamicSharedMemorySize,  \
-                           (int)smem);                                                                         \
-    if (max_q_len >= 64)                                                                                       \
-      sb_launch_plain(forget_scan_kernel<RS_, ROWS_, VEC_>, grid, block, smem, stream, (const float*)qf,       \
-                      (const float*)v, state, cu_q, slots, num_slots, H, d, dv, cols, nbuf, out, err);         \
-    else                                                                                                       \
-      sb_launch(forget_scan_kernel<RS_, ROWS_, VEC_>, grid, block, smem, stream, (const float*)qf,             \
-                (const float*)v, state, cu_q, slots, num_slots, H, d, dv, cols, nbuf, out, err);               \
+#define SB_FORGET_V(RS_, ROWS_, VEC_)                                                                                 \
+  do {                                                                                                                \
+    if (smem > 48 * 1024)                                                                                             \
+      cudaFuncSetAttribute(forget_scan_kernel<RS_, ROWS_, VEC_, KINDS>, cudaFuncAttributeMaxDynamicSharedMemorySize,  \
+                           (int)smem);                                                                                \
+    if (max_q_len >= 64)                                                                                              \
+      sb_launch_plain(forget_scan_kernel<RS_, ROWS_, VEC_, KINDS>, grid, block, smem, stream, qf, v, state, cu_q,     \
+                      slots, num_slots, H, d, dv, cols, nbuf, out, err);                                              \
+    else                                                                                                              \
+      sb_launch(forget_scan_kernel<RS_, ROWS_, VEC_, KINDS>, grid, block, smem, stream, qf, v, state, cu_q, slots,    \
+                num_slots, H, d, dv, cols, nbuf, out, err);                                                           \
   } while (0)
 #define SB_FORGET(RS_)                                \
   do {                                                \
@@ -691,14 +691,113 @@ extern "C" int sb_forget_scan(const void* pre, int row_width, int dtype, const f
   return 0;
 }
 
+// scratch: float32 [T, 2 H d + H dv] for the inputs.
+extern "C" int sb_forget_scan(const void* pre, int row_width, int dtype, const float* bias, const float* lower,
+                              float* state, const int* cu_q, const int* slots, int num_tokens, int num_seqs,
+                              int num_slots, int H, int d, int dv, int max_q_len, float* scratch, float* out,
+                              int* err, cudaStream_t stream) {
+  if (num_seqs == 0 || num_tokens == 0) return 0;
+  if (d <= 0 || d > 32 * 32 || dv <= 0 || H <= 0) return -13;
+  float* qf = scratch;
+  float* v = scratch + (size_t)num_tokens * 2 * H * d;
+  const int widest = H * d > H * dv ? H * d : H * dv;
+  const dim3 in_grid((unsigned)num_tokens, (unsigned)((widest + 255) / 256));
+  if (dtype == SB_DTYPE_F32)
+    sb_launch(forget_inputs_kernel<float>, in_grid, 256, 0, stream, (const float*)pre, row_width, bias, lower,
+              H * d, H * dv, qf, v);
+  else
+    sb_launch(forget_inputs_kernel<bf16>, in_grid, 256, 0, stream, (const bf16*)pre, row_width, bias, lower,
+              H * d, H * dv, qf, v);
+  SB_LAUNCH_CHECK();
+  return launch_forget_scan<2>(qf, v, state, cu_q, slots, num_seqs, num_slots, H, d, dv, max_q_len, out, err, stream);
+}
+
+// ---------------------------------------------------------------------------
+// Gated linear attention: S <- diag(f) S + k v^T, o = S^T q with
+//   q = pq * d^(-1/2),  f = sigmoid(z)^(1 / tau),  z = low . W + b
+// `pre` [T, row_width] holds pq (H d) | k (H d) | v (H dv) as the projection left them and at
+// low_offset `rank` numbers of a low rank's first half; w [rank, H d] float32 is its second half,
+// multiplied here in float32.  Inputs once per token (float32: qf [T, 3, H d] = q, f, k and v [T, H dv]),
+// then the walk above.  A block makes the inputs of GLA_TOKENS tokens for 256 channels, so that a
+// fetched weight serves all of them.
+// ---------------------------------------------------------------------------
+template <typename T, int TOKENS>
+__global__ void __launch_bounds__(256)
+gated_linear_inputs_kernel(const T* __restrict__ pre, int row_width, int low_offset, int rank,
+                           const float* __restrict__ w, const float* __restrict__ bias, float inv_tau, float q_scale,
+                           int n_qf, int n_v, int num_tokens, float* __restrict__ qf, float* __restrict__ v) {
+  extern __shared__ float low[];  // [rank][TOKENS]
+  pdl_wait_block();
+  pdl_launch_dependents();
+  const int t0 = blockIdx.x * TOKENS, c = blockIdx.y * blockDim.x + threadIdx.x;
+  for (int idx = threadIdx.x; idx < rank * TOKENS; idx += blockDim.x) {
+    const int i = idx / rank, r = idx - i * rank;
+    low[r * TOKENS + i] = t0 + i < num_tokens ? to_f32<T>(pre[(size_t)(t0 + i) * row_width + low_offset + r]) : 0.f;
+  }
+  __syncthreads();
+  if (c < n_qf) {
+    float z[TOKENS];
+#pragma unroll
+    for (int i = 0; i < TOKENS; ++i) z[i] = bias[c];
+    for (int r = 0; r < rank; ++r) {
+      const float wr = w[(size_t)r * n_qf + c];
+#pragma unroll
+      for (int i = 0; i < TOKENS; ++i) z[i] = fmaf(low[r * TOKENS + i], wr, z[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < TOKENS; ++i) {
+      if (t0 + i >= num_tokens) break;
+      const T* x = pre + (size_t)(t0 + i) * row_width;
+      float* out = qf + (size_t)(t0 + i) * 3 * n_qf;
+      out[c] = to_f32<T>(x[c]) * q_scale;
+      // log sigmoid(z) = min(z, 0) - log(1 + e^(-|z|))
+      out[n_qf + c] = expf((fminf(z[i], 0.f) - log1pf(expf(-fabsf(z[i])))) * inv_tau);
+      out[2 * n_qf + c] = to_f32<T>(x[n_qf + c]);
+    }
+  }
+  if (c < n_v) {
+#pragma unroll
+    for (int i = 0; i < TOKENS; ++i)
+      if (t0 + i < num_tokens)
+        v[(size_t)(t0 + i) * n_v + c] = to_f32<T>(pre[(size_t)(t0 + i) * row_width + 2 * n_qf + c]);
+  }
+}
+
+// scratch: float32 [T, 3 H d + H dv] for the inputs.
+extern "C" int sb_gated_linear_scan(const void* pre, int row_width, int low_offset, int dtype, const float* w, int rank,
+                                    const float* bias, float tau, float* state, const int* cu_q, const int* slots,
+                                    int num_tokens, int num_seqs, int num_slots, int H, int d, int dv, int max_q_len,
+                                    float* scratch, float* out, int* err, cudaStream_t stream) {
+  if (num_seqs == 0 || num_tokens == 0) return 0;
+  if (d <= 0 || d > 32 * 32 || dv <= 0 || H <= 0 || rank <= 0 || rank > 1024 || !(tau > 0.f)) return -13;
+  float* qf = scratch;
+  float* v = scratch + (size_t)num_tokens * 3 * H * d;
+  const int widest = H * d > H * dv ? H * d : H * dv;
+  const unsigned slices = (unsigned)((widest + 255) / 256);
+  const float q_scale = (float)(1.0 / sqrt((double)d)), inv_tau = 1.0f / tau;
+#define SB_GLA_INPUTS(T_, N_)                                                                                         \
+  sb_launch(gated_linear_inputs_kernel<T_, N_>, dim3((unsigned)((num_tokens + N_ - 1) / N_), slices), 256,            \
+            (size_t)rank * N_ * sizeof(float), stream, (const T_*)pre, row_width, low_offset, rank, w, bias, inv_tau, \
+            q_scale, H * d, H * dv, num_tokens, qf, v)
+  const bool many = num_tokens >= 256;
+  if (dtype == SB_DTYPE_F32) {
+    if (many) SB_GLA_INPUTS(float, 8); else SB_GLA_INPUTS(float, 1);
+  } else {
+    if (many) SB_GLA_INPUTS(bf16, 8); else SB_GLA_INPUTS(bf16, 1);
+  }
+#undef SB_GLA_INPUTS
+  SB_LAUNCH_CHECK();
+  return launch_forget_scan<3>(qf, v, state, cu_q, slots, num_seqs, num_slots, H, d, dv, max_q_len, out, err, stream);
+}
+
 // ---------------------------------------------------------------------------
 // Output of a recurrent mixer: per head RMS norm, channel scale, and (gate_offset >= 0) a gate read
-// from `low`.  One block per token, a warp per head.
+// from `low`: sigmoid(g), or g sigmoid(g) with `silu`.  One block per token, a warp per head.
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_head_norm_kernel(const float* __restrict__ o, const T* __restrict__ low, int low_width, int gate_offset,
-                       const float* __restrict__ w, float eps, int H, int dv, T* __restrict__ out) {
+                       int silu, const float* __restrict__ w, float eps, int H, int dv, T* __restrict__ out) {
   pdl_wait_block();
   pdl_launch_dependents();
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -709,23 +808,26 @@ gated_head_norm_kernel(const float* __restrict__ o, const T* __restrict__ low, i
     ss = warp_sum(ss);
     const float rstd = 1.0f / sqrtf(ss / (float)dv + eps);
     for (int c = lane; c < dv; c += 32) {
-      const float gate = gate_offset < 0 ? 1.0f
-          : sigmoid_f32(to_f32<T>(low[(size_t)t * low_width + gate_offset + h * dv + c]));
+      float gate = 1.0f;
+      if (gate_offset >= 0) {
+        const float g = to_f32<T>(low[(size_t)t * low_width + gate_offset + h * dv + c]);
+        gate = sigmoid_f32(g) * (silu ? g : 1.0f);
+      }
       out[((size_t)t * H + h) * dv + c] = from_f32<T>(src[c] * rstd * w[c] * gate);
     }
   }
 }
 
-extern "C" int sb_gated_head_norm(const float* o, const void* low, int low_width, int gate_offset, int dtype,
+extern "C" int sb_gated_head_norm(const float* o, const void* low, int low_width, int gate_offset, int silu, int dtype,
                                   const float* w, float eps, int num_tokens, int H, int dv, void* out,
                                   cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (dtype == SB_DTYPE_F32)
     sb_launch(gated_head_norm_kernel<float>, num_tokens, 256, 0, stream, o, (const float*)low, low_width,
-              gate_offset, w, eps, H, dv, (float*)out);
+              gate_offset, silu, w, eps, H, dv, (float*)out);
   else
     sb_launch(gated_head_norm_kernel<bf16>, num_tokens, 256, 0, stream, o, (const bf16*)low, low_width,
-              gate_offset, w, eps, H, dv, (bf16*)out);
+              gate_offset, silu, w, eps, H, dv, (bf16*)out);
   SB_LAUNCH_CHECK();
   return 0;
 }

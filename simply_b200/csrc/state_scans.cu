@@ -112,6 +112,8 @@ general_delta_scan_kernel(const float* __restrict__ vecs, const float* __restric
     if (threadIdx.x == 0) atomicOr(err, SB_ERR_BAD_SLOT);
     return;
   }
+  const int copies = rows_sharing_slot(slots, b, gridDim.y);
+  if (copies == 0) return;  // an earlier row of the slot does this row's work
   const int cols_pad = (cols + 3) & ~3;
   const int per_token = 5 * d + cols_pad + 4;
   const bool wide = (d & 3) == 0;
@@ -232,7 +234,9 @@ general_delta_scan_kernel(const float* __restrict__ vecs, const float* __restric
         const int row = rs + RS * r;
         if (row < d) s[r] = fmaf(AHEAD ? ck[r] : here[3 * d + row], cv, fmaf(-(AHEAD ? ca[r] : here[2 * d + row]), p, s[r]));
       }
-      if (on && rs == 0) out[((size_t)(first + base + i) * H + h) * d + col] = fmaf(cv, crk, fmaf(-p, cra, od));
+      if (on && rs == 0)
+        for (int c = 0; c < copies; ++c)
+          out[((size_t)(first + base + i + c) * H + h) * d + col] = fmaf(cv, crk, fmaf(-p, cra, od));
       if constexpr (AHEAD) {
 #pragma unroll
         for (int r = 0; r < ROWS; ++r) {
@@ -243,7 +247,7 @@ general_delta_scan_kernel(const float* __restrict__ vecs, const float* __restric
     }
     __syncthreads();  // the buffer is filled again two chunks on
   }
-  if (on && owns_slot(slots, b)) {
+  if (on) {
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
       const int row = rs + RS * r;
@@ -516,6 +520,8 @@ state_space_scan_kernel(const float* __restrict__ xbc, int C, const float* __res
     if (threadIdx.x == 0) atomicOr(err, SB_ERR_BAD_SLOT);
     return;
   }
+  const int copies = rows_sharing_slot(slots, b, gridDim.y);
+  if (copies == 0) return;  // an earlier row of the slot does this row's work
   const int g = h / (H / G);
   const int inner = H * dv;
   const int cols_pad = (cols + 3) & ~3;
@@ -579,11 +585,13 @@ state_space_scan_kernel(const float* __restrict__ xbc, int C, const float* __res
       }
 #pragma unroll
       for (int o = 1; o < RS; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (on && rs == 0) out[((size_t)(first + base + i) * H + h) * dv + col] = fmaf(d_skip, xj, y);
+      if (on && rs == 0)
+        for (int c = 0; c < copies; ++c)
+          out[((size_t)(first + base + i + c) * H + h) * dv + col] = fmaf(d_skip, xj, y);
     }
     __syncthreads();
   }
-  if (on && owns_slot(slots, b)) {
+  if (on) {
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
       const int row = rs + RS * r;

@@ -228,3 +228,38 @@ extern "C" int sb_scale_values(float* x, float c, long long n, cudaStream_t stre
   SB_LAUNCH_CHECK();
   return 0;
 }
+
+// ---------------------------------------------------------------------------
+// max(z, 0)^2 in place, 16 bytes per thread and turn.
+template <typename T>
+__global__ void __launch_bounds__(256)
+relu_squared_kernel(T* __restrict__ z, long long n) {
+  pdl_wait_block();
+  pdl_launch_dependents();
+  constexpr int N = Vec<T>::N;
+  const long long groups = n / N, step = (long long)gridDim.x * blockDim.x;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < groups; i += step) {
+    float a[N];
+    Vec<T>::load(z + i * N, a);
+#pragma unroll
+    for (int e = 0; e < N; ++e) {
+      const float r = fmaxf(a[e], 0.f);
+      a[e] = r * r;
+    }
+    Vec<T>::store(z + i * N, a);
+  }
+  for (long long i = groups * N + (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += step) {
+    const float r = fmaxf(to_f32<T>(z[i]), 0.f);
+    z[i] = from_f32<T>(r * r);
+  }
+}
+
+extern "C" int sb_relu_squared(void* z, int dtype, long long n, cudaStream_t stream) {
+  if (n == 0) return 0;
+  const long long per = 256 * (dtype == SB_DTYPE_F32 ? 4 : 8);
+  const unsigned blocks = (unsigned)min((n + per - 1) / per, (long long)148 * 16);
+  if (dtype == SB_DTYPE_F32) sb_launch(relu_squared_kernel<float>, blocks, 256, 0, stream, (float*)z, n);
+  else sb_launch(relu_squared_kernel<bf16>, blocks, 256, 0, stream, (bf16*)z, n);
+  SB_LAUNCH_CHECK();
+  return 0;
+}

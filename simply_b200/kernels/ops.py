@@ -215,6 +215,7 @@ class CudaOps:
       for item in env.split(","):
         name, _, rows = item.partition(":")
         self.mid_rows[name] = int(rows or 128)
+    self.two_norms_rows = 0  # tokens per block of the two-norms kernel; 0: the launch chooses (tests)
     self.mid_split = 0
     self.mid_stages = 0  # 0: the launch chooses the depth of the ring of stages; 8 deep, 4 shallow (tests)
     # The true 32-bit path must not be routed through a reduced-precision matrix mode.
@@ -251,7 +252,14 @@ class CudaOps:
                                        c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void, c_void],
         "sb_paged_attention_general": [c_void, c_int, c_void, c_void, c_int, c_void, c_void, c_void, c_int,
                                        c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void, c_void,
-                                       c_int, c_int, c_int, c_int, c_void, c_void, c_void, c_void],
+                                       c_int, c_int, c_int, c_int, c_void, c_void, c_int, c_int, c_void, c_void],
+        "sb_residual_two_norms": [c_void, c_void, c_void, c_void, c_int, c_void, c_int, c_float, c_int, c_void, c_int,
+                                  c_float, c_int, c_void, c_void, c_int, c_void, c_void, c_void, c_int, c_int, c_int,
+                                  c_void, c_void, c_int, c_void, c_void],
+        "sb_gated_linear_scan": [c_void, c_int, c_int, c_int, c_void, c_int, c_void, c_float, c_void, c_void, c_void,
+                                 c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void, c_void, c_void, c_void],
+        "sb_gemm_skinny_bf16_relu_squared": [c_void, c_void, c_void, c_int, c_int, c_int, c_int, c_void],
+        "sb_relu_squared": [c_void, c_int, c_ll, c_void],
         "sb_qk_norm_rotate_store": [c_void, c_int, c_int, c_void, c_void, c_float, c_void, c_void, c_int, c_void,
                                     c_void, c_void, c_void, c_int, c_void, c_void, c_int, c_int, c_int, c_int, c_int,
                                     c_int, c_int, c_int, c_void, c_void],
@@ -263,7 +271,7 @@ class CudaOps:
                             c_void, c_void, c_void, c_void],
         "sb_delta_scan": [c_void, c_void, c_void, c_void, c_void, c_void, c_void, c_void, c_int, c_int, c_int,
                           c_int, c_int, c_int, c_int, c_void, c_void, c_void],
-        "sb_gated_head_norm": [c_void, c_void, c_int, c_int, c_int, c_void, c_float, c_int, c_int, c_int, c_void,
+        "sb_gated_head_norm": [c_void, c_void, c_int, c_int, c_int, c_int, c_void, c_float, c_int, c_int, c_int, c_void,
                                c_void],
         "sb_normed_mean": [c_void, c_void, c_void, c_void, c_void, c_void, c_void, c_void, c_int, c_int, c_float,
                            c_int, c_int, c_void, c_void],
@@ -284,9 +292,9 @@ class CudaOps:
         "sb_table_route": [c_void, c_void, c_int, c_int, c_int, c_void, c_void, c_int, c_void, c_void],
         "sb_head_linear": [c_void, c_int, c_int, c_int, c_void, c_int, c_int, c_int, c_int, c_void, c_int, c_int,
                            c_float, c_int, c_void],
-        "sb_latent_prepare": [c_void, c_int, c_int, c_void, c_void, c_float, c_void, c_int, c_int, c_int, c_int,
+        "sb_latent_prepare": [c_void, c_int, c_int, c_void, c_void, c_float, c_void, c_int, c_int, c_float, c_int, c_int, c_int,
                               c_void, c_void, c_void, c_int, c_int, c_int, c_void, c_void, c_int, c_void, c_void],
-        "sb_turn_query_part": [c_void, c_int, c_int, c_void, c_int, c_int, c_int, c_void, c_int, c_int, c_float,
+        "sb_turn_query_part": [c_void, c_int, c_int, c_void, c_int, c_int, c_int, c_void, c_int, c_int, c_float, c_int, c_float,
                                c_void, c_int, c_int, c_void],
         "sb_general_delta_scan": [c_void, c_int, c_void, c_int, c_int, c_void, c_void, c_void, c_void, c_void, c_int,
                                   c_int, c_int, c_int, c_int, c_int, c_void, c_void, c_void, c_void],
@@ -397,8 +405,10 @@ class CudaOps:
       raise KernelError("a kernel skipped an invalid access: " + "; ".join(reasons))
 
   # ---- checks ---------------------------------------------------------------
-  def check_attention(self, head_dim: int, num_heads: int, num_kv_heads: int) -> None:
+  def check_attention(self, head_dim: int, num_heads: int, num_kv_heads: int, value_dim: int | None = None) -> None:
     """Refuses shapes no kernel takes; compiles the tensor-core kernels of this head size."""
+    if value_dim is not None and value_dim != head_dim:
+      return
     if head_dim <= 0 or head_dim % 2 or head_dim > 512:
       raise KernelError(f"attention kernels take even head sizes up to 512, got {head_dim}")
     if num_heads % num_kv_heads:
@@ -573,11 +583,12 @@ class CudaOps:
     return ("attention_plan", window, group, num_kv_heads, head_dim, self._prefill_rows(head_dim, group, page_size))
 
   def attention_graph_plan(self, *, window: int | None, num_heads: int, num_kv_heads: int, head_dim: int,
-                           batch: int, bucket: int, max_burst: int, page_size: int):
+                           batch: int, bucket: int, max_burst: int, page_size: int, key_chunk: int | None = None,
+                           value_dim: int | None = None):
     """The static work list a decode graph needs for one kind of attention layer, or None when
     the kernel that serves it reads no list (the general kernel)."""
     group = num_heads // num_kv_heads
-    if not self._uses_tensor_core_attention(head_dim, group):
+    if not self._uses_tensor_core_attention(head_dim, group) or value_dim is not None or key_chunk is not None:
       return None
     return AttentionGraphPlan(self, window, group, num_kv_heads, head_dim, batch, bucket, max_burst, page_size)
 
@@ -826,6 +837,29 @@ class CudaOps:
         _ptr(rows), _ptr(y), num_rows, width, h.shape[0], _ptr(self.err))
     return y
 
+  def residual_two_norms(self, h: torch.Tensor, branch: torch.Tensor | None, branch2: torch.Tensor | None, norm: Any,
+                         norm2: Any, shift: torch.Tensor | None, state: torch.Tensor | None, ctx: Any):
+    """(h + branch + branch2, y, y2): y = norm(h + ...), with `shift` (float32 [width]) moved towards the
+    previous token's y, and y2 = norm2(h + ...) (None without `norm2`), in the activation dtype.
+    `state` [slots, width] float32 keeps every request's last y (csrc/two_norms.cu)."""
+    t, width = h.shape
+    as_own = lambda b: b if b is None or b.dtype == self.dtype else self.cast(b, self.dtype)
+    branch, branch2 = as_own(branch), as_own(branch2)
+    if branch is None:
+      branch, branch2 = branch2, None
+    h_out = self._new(t, width, dtype=torch.float32) if branch is not None else None
+    y = self._new(t, width)
+    y2 = self._new(t, width) if norm2 is not None else None
+    w1, w2 = norm.weight, norm2.weight if norm2 is not None else None
+    self._call("sb_residual_two_norms", _ptr(h), _ptr(h_out), _ptr(branch), _ptr(branch2), _code(y), _ptr(w1), int(w1.dtype == torch.float32),
+               float(norm.eps), int(norm.plus_one), _ptr(w2),
+               int(w2 is not None and w2.dtype == torch.float32),
+               float(norm2.eps) if norm2 is not None else float(norm.eps),
+               int(norm2.plus_one) if norm2 is not None else 0, _ptr(shift), _ptr(state),
+               state.shape[0] if state is not None else 0, _ptr(ctx.token_seq), _ptr(ctx.cu_q), _ptr(ctx.slots),
+               ctx.num_seqs, t, width, _ptr(y), _ptr(y2), self.two_norms_rows, _ptr(self.err))
+    return (h_out if h_out is not None else h), y, y2
+
   def gather_rows(self, x: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
     out = self._new(rows.numel(), x.shape[1], dtype=x.dtype)
     self._call("sb_gather_rows", _ptr(x), _code(x), _ptr(rows), _ptr(out), rows.numel(), x.shape[1],
@@ -897,6 +931,18 @@ class CudaOps:
     self._call("sb_xielu", _ptr(z), _ptr(act), _ptr(z), _code(z), z.numel())
     return z
 
+  def linear_relu_squared(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """max(x . w^T, 0)^2; a step of few tokens activates on the product's sums."""
+    m, k = x.shape
+    if w.dtype == torch.bfloat16 and x.dtype == torch.bfloat16 and m <= self.skinny_max_rows:
+      out = self._new(m, w.shape[0], dtype=torch.bfloat16)
+      if self._call("sb_gemm_skinny_bf16_relu_squared", _ptr(x), _ptr(w), _ptr(out), m, w.shape[0], k,
+                    self.skinny_warps) == 0:
+        return out
+    z = self.linear(x, w)
+    self._call("sb_relu_squared", _ptr(z), _code(z), z.numel())
+    return z
+
   # ---- positions ------------------------------------------------------------
   def rotation_tables(self, positions: torch.Tensor, timescale: torch.Tensor, scale_factor: float):
     t, half = positions.numel(), timescale.numel()
@@ -966,14 +1012,15 @@ class CudaOps:
                       num_heads: int, num_kv_heads: int, head_dim: int, logit_softcap: float,
                       window: int | None, value_dim: int | None = None, pooled: tuple | None = None,
                       values_in_keys: bool = False, sink: torch.Tensor | None = None,
-                      distance_bias: torch.Tensor | None = None) -> torch.Tensor:
+                      distance_bias: torch.Tensor | None = None, key_chunk: int | None = None) -> torch.Tensor:
     """`value_dim`: size of a value head where it is not the key heads'.  `pooled`: (storage of block
     entries, its block table, block length): with a window, one key and value per whole block that
     has left the window, under the same softmax.  `values_in_keys`: an entry's value is the first
     `value_dim` numbers of its key row (a cache of latents).  `sink`: float32 [heads], a number per
     head whose exponential joins the softmax's denominator (csrc/attention_generic.cu).
     `distance_bias`: float32 [2, heads], r1 and r2 per head: the score of query i and key j loses
-    r1 log(1 + r2 (i - j))."""
+    r1 log(1 + r2 (i - j)); float32 [1, heads]: it loses r1 (i - j).  `key_chunk` C (without a
+    window): a query sees its own chunk's keys, from (i // C) * C on."""
     t = q.shape[0]
     value_dim = head_dim if value_dim is None else value_dim
     out = self._new(t, num_heads * value_dim, dtype=q.dtype)
@@ -982,10 +1029,13 @@ class CudaOps:
       raise KernelError("latent rows and sinks go with neither a score cap nor pooled blocks")
     if distance_bias is not None and (pooled is not None or values_in_keys):
       raise KernelError("a distance bias goes with neither pooled blocks nor latent rows")
+    if key_chunk is not None and (window or pooled is not None or values_in_keys):
+      raise KernelError("chunks of keys go with neither a window, pooled blocks nor latent rows")
+    linear_bias = int(distance_bias is not None and distance_bias.shape[0] == 1)
     # (a distance bias with key size = value size in bfloat16: the mma.sync tile kernels below)
     biased_on_tensor_cores = (distance_bias is not None and value_dim == head_dim and q.dtype == torch.bfloat16
                               and self._uses_tensor_core_attention(head_dim, group))
-    if (pooled is not None or value_dim != head_dim or values_in_keys or sink is not None
+    if (pooled is not None or value_dim != head_dim or values_in_keys or sink is not None or key_chunk is not None or linear_bias
         or (distance_bias is not None and not biased_on_tensor_cores)):
       pool, pool_table, pool_len = pooled if pooled is not None else (None, None, 0)
       if pool is not None and pool.dtype != storage.dtype:
@@ -997,7 +1047,8 @@ class CudaOps:
         self._call("sb_paged_attention_general", _ptr(q), _code(q), _ptr(storage), _ptr(block_table),
                    block_table.shape[1], _ptr(ctx.token_seq), _ptr(ctx.positions), _ptr(out), t, num_heads,
                    num_kv_heads, head_dim, value_dim, ctx.page_size, storage.shape[0], float(logit_softcap),
-                   int(window or 0), *pool_args, int(values_in_keys), _ptr(sink), _ptr(distance_bias), _ptr(self.err))
+                   int(window or 0), *pool_args, int(values_in_keys), _ptr(sink), _ptr(distance_bias), linear_bias,
+                   int(key_chunk or 0), _ptr(self.err))
 
       # bfloat16 with key size = value size: the tensor-core tile kernel (mma.sync tiles of 64 rows,
       # the block entries in tiles of their own ahead of the tokens) for prompt portions and single
@@ -1254,21 +1305,25 @@ class CudaOps:
   # ---- attention over latents ---------------------------------------------------------------------
   def latent_prepare(self, down: torch.Tensor, query_norm: torch.Tensor, kv_norm: torch.Tensor, eps: float,
                      freq: torch.Tensor | None, *, query_rank: int, kv_rank: int, rotated_dim: int,
-                     storage: torch.Tensor | None, block_table: torch.Tensor, ctx: Any) -> torch.Tensor:
+                     storage: torch.Tensor | None, block_table: torch.Tensor, ctx: Any, interleaved: bool = False,
+                     amplitude: float = 1.0) -> torch.Tensor:
     """Norms of both latents, the shared key part turned, the token's row [c | k_r] into its page;
-    returns the queries' latent [T, query_rank] (csrc/latent_attention.cu)."""
+    returns the queries' latent [T, query_rank] (csrc/latent_attention.cu).  `interleaved`: neighbours pair
+    up (else halves); `amplitude`: the factor on cosines and sines."""
     t = down.shape[0]
     cq = self._new(t, query_rank, dtype=down.dtype)
     if storage is not None and storage.dtype != down.dtype:
       raise KernelError("the cache of latents is kept in the activation dtype")
     self._call("sb_latent_prepare", _ptr(down), down.shape[1], _code(down), _ptr(query_norm), _ptr(kv_norm),
-               float(eps), _ptr(freq), freq.numel() if freq is not None else 0, query_rank, kv_rank, rotated_dim,
+               float(eps), _ptr(freq), freq.numel() if freq is not None else 0, int(interleaved), float(amplitude),
+               query_rank, kv_rank, rotated_dim,
                _ptr(ctx.positions), _ptr(ctx.token_seq), _ptr(block_table), block_table.shape[1], ctx.page_size,
                storage.shape[0] if storage is not None else 0, _ptr(storage), _ptr(cq), t, _ptr(self.err))
     return cq
 
   def latent_queries(self, q: torch.Tensor, key_up_t: torch.Tensor, freq: torch.Tensor | None, scale: float,
-                     ctx: Any, *, num_heads: int, head_dim: int, rotated_dim: int) -> torch.Tensor:
+                     ctx: Any, *, num_heads: int, head_dim: int, rotated_dim: int, interleaved: bool = False,
+                     amplitude: float = 1.0) -> torch.Tensor:
     """Per head [W_uk^T q_plain | turn(q_rot)] * scale: q [T, H (head_dim + rotated_dim)], key_up_t
     [H, kv_rank, head_dim] -> [T, H (kv_rank + rotated_dim)]."""
     t = q.shape[0]
@@ -1279,7 +1334,8 @@ class CudaOps:
       self._call("sb_head_linear", _ptr(q), num_heads * row_in, row_in, 0, _ptr(key_up_t), _code(q), num_heads, head_dim,
                  rank, _ptr(out), num_heads * row_out, row_out, float(scale), t)
     self._call("sb_turn_query_part", _ptr(q), row_in, head_dim, _ptr(out), row_out, rank, _code(q), _ptr(freq),
-               freq.numel() if freq is not None else 0, rotated_dim, float(scale), _ptr(ctx.positions), t, num_heads)
+               freq.numel() if freq is not None else 0, int(interleaved), float(amplitude), rotated_dim, float(scale),
+               _ptr(ctx.positions), t, num_heads)
     return out
 
   # ---- recurrent mixers with a matrix per head ------------------------------------------------------
@@ -1323,6 +1379,22 @@ class CudaOps:
     self._call("sb_forget_scan", _ptr(pre), pre.shape[1], _code(pre), _ptr(bias), _ptr(lower), _ptr(state),
                _ptr(ctx.cu_q), _ptr(ctx.slots), t, ctx.num_seqs, state.shape[0], num_heads, head_dim, value_dim,
                ctx.max_q_len, _ptr(scratch), _ptr(out), _ptr(self.err))
+    self.launches += 1
+    return out
+
+  def gated_linear_scan(self, pre: torch.Tensor, low_offset: int, decay_out_t: torch.Tensor, decay_bias: torch.Tensor,
+                        tau: float, state: torch.Tensor, ctx: Any, *, num_heads: int, head_dim: int,
+                        value_dim: int) -> torch.Tensor:
+    """pre [T, q | k | v | ... | low rank at low_offset] as projected, decay_out_t float32 [rank, heads * head_dim]
+    -> float32 o [T, heads, value_dim]; walks every sequence's tokens through its state [slots, heads,
+    head_dim, value_dim] (csrc/recurrent_mix.cu)."""
+    t = pre.shape[0]
+    out = self._new(t, num_heads, value_dim, dtype=torch.float32)
+    scratch = self._new(t, num_heads * (3 * head_dim + value_dim), dtype=torch.float32)
+    self._call("sb_gated_linear_scan", _ptr(pre), pre.shape[1], low_offset, _code(pre), _ptr(decay_out_t),
+               decay_out_t.shape[0], _ptr(decay_bias), float(tau), _ptr(state), _ptr(ctx.cu_q), _ptr(ctx.slots), t,
+               ctx.num_seqs, state.shape[0], num_heads, head_dim, value_dim, ctx.max_q_len, _ptr(scratch), _ptr(out),
+               _ptr(self.err))
     self.launches += 1
     return out
 
@@ -1476,15 +1548,16 @@ class CudaOps:
     return out
 
   def gated_head_norm(self, o: torch.Tensor, low: torch.Tensor | None, gate_offset: int, weight: torch.Tensor,
-                      eps: float, num_heads: int, value_dim: int) -> torch.Tensor:
-    """Per head o / rms(o) * weight, times sigmoid(low[:, gate_offset + ...]); `low` None: no gate."""
+                      eps: float, num_heads: int, value_dim: int, gate: str = "sigmoid") -> torch.Tensor:
+    """Per head o / rms(o) * weight, times sigmoid(g) (`gate` "silu": g sigmoid(g)) with g = low[:, gate_offset
+    + ...]; `low` None: no gate."""
     if low is None:
       out = self._new(o.shape[0], num_heads * value_dim)
-      self._call("sb_gated_head_norm", _ptr(o), None, 0, -1, _code(out), _ptr(weight),
+      self._call("sb_gated_head_norm", _ptr(o), None, 0, -1, 0, _code(out), _ptr(weight),
                  float(eps), o.shape[0], num_heads, value_dim, _ptr(out))
       return out
     out = self._new(o.shape[0], num_heads * value_dim, dtype=low.dtype)
-    self._call("sb_gated_head_norm", _ptr(o), _ptr(low), low.shape[1], gate_offset, _code(low), _ptr(weight),
+    self._call("sb_gated_head_norm", _ptr(o), _ptr(low), low.shape[1], gate_offset, int(gate == "silu"), _code(low), _ptr(weight),
                float(eps), o.shape[0], num_heads, value_dim, _ptr(out))
     return out
 
