@@ -295,7 +295,10 @@ __global__ void __launch_bounds__(WM * WN * NS * 32) latent_attention_kernel(con
                     vs * VDS, need_mask);
     __syncthreads();
   }
-  cp_async_wait<0>();  // (a block without tiles of its own still has its query rows under way)
+  // A block without tiles of its own still has its query rows under way, every thread's, and the merge
+  // below writes where they land.
+  cp_async_wait<0>();
+  __syncthreads();
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 1);
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
