@@ -1,5 +1,6 @@
 // Ragged paged attention on tensor cores (bfloat16 in, float32 softmax and accumulate),
-// compiled once per head size (-DSB_HEAD_DIM=N, N a multiple of 16 up to 256).
+// compiled once per head size (-DSB_HEAD_DIM=N, N a multiple of 16 up to 256) and, where value heads
+// have another size than key heads, per pair of sizes (-DSB_VALUE_DIM=M, likewise).
 //
 //   s = q . k                 (q is already rotated and scaled)
 //   s = cap * tanh(s / cap)   if cap > 0          simply/model_lib.py:621-626
@@ -7,6 +8,10 @@
 //                                                 simply/model_lib.py:469-515
 //   p = softmax(s) in float32, o = p . v          simply/model_lib.py:633-637
 //   query head n reads kv head n / G              simply/model_lib.py:2306-2310
+//
+// Options: a distance term is taken off the scores (r1 log(1 + r2 d), or r1 d); in place of a window,
+// chunks of C keys counted from position 0, of which a query sees its own; a number per head (a sink)
+// whose exponential joins the softmax's denominator.
 //
 // Two kernels share the tile code.
 //  * prefill: a block owns 64 query rows of one (sequence, kv head): the G query heads
@@ -29,35 +34,46 @@
 #ifndef SB_HEAD_DIM
 #define SB_HEAD_DIM 256
 #endif
+#ifndef SB_VALUE_DIM
+#define SB_VALUE_DIM SB_HEAD_DIM
+#endif
 
 namespace {
 
-constexpr int DH = SB_HEAD_DIM;
+constexpr int DH = SB_HEAD_DIM, DV = SB_VALUE_DIM;
+constexpr bool ONE_SIZE = DH == DV;
 constexpr int PITCH = DH + 8;  // elements; the 16-byte pad spreads 8 consecutive rows over all banks
+constexpr int VPITCH = DV + 8;
 constexpr int BN = 64;         // keys per tile
 constexpr int CPR = DH / 8;    // 16-byte chunks per row
+constexpr int VCPR = DV / 8;
+constexpr int SRC = ONE_SIZE ? 1 : 2;  // places per row of a tile: the key's, and the value's where it is not at a fixed distance
 constexpr int NT = 128;        // threads per block
 constexpr float LOG2E = 1.4426950408889634f;
 
 static_assert(DH % 16 == 0 && DH >= 16 && DH <= 256, "head size must be a multiple of 16 up to 256");
+static_assert(DV % 16 == 0 && DV >= 16 && DV <= 256, "value size must be a multiple of 16 up to 256");
 
 struct AttnParams {
   const bf16* q;      // [T, Hq, DH]
-  const bf16* cache;  // [P, 2, Hkv, page, DH]
+  const bf16* cache;  // [P, 2, Hkv, page, DH]; with two sizes per page [Hkv, page, DH], then [Hkv, page, DV]
   const int* block_table;
   int max_pages;
   const int* cu_q;     // [B + 1]
   const int* q_start;  // [B]
-  bf16* out;           // [T, Hq * DH]
+  bf16* out;           // [T, Hq * DV]
   int num_q_heads, num_kv_heads, page_size, num_pages;
   float cap;
   int window;
   // optional, float32 [2, Hq]: r1 and r2 per query head; the score of query i and key j loses
-  // r1 log(1 + r2 (i - j))
+  // r1 log(1 + r2 (i - j)).  With `linear`, float32 [Hq]: it loses r1 (i - j).
   const float* distance;
+  int linear;
+  int key_chunk;      // > 0 (without a window): position i sees the keys from (i / C) * C on
+  const float* sink;  // optional, float32 [Hq]: exp(sink) joins the denominator
   const int* items;  // prefill: (sequence, first token of the tile); decode: (sequence, chunk)
   int chunk;         // decode: keys per chunk (a multiple of BN)
-  float* part_o;     // decode: [items, Hkv, rows_max, DH]
+  float* part_o;     // decode: [items, Hkv, rows_max, DV]
   float* part_ml;    // decode: [items, Hkv, rows_max, 2]
   int rows_max;
   int older_keys_settled;  // decode: keys below q_start were written before the kernel just before this one
@@ -68,6 +84,12 @@ struct AttnParams {
   const int* pool_table;
   int pool_max_pages, pool_len, pool_entries, pool_pages;
 };
+
+// The lowest key that the query at `pos` sees.
+__device__ __forceinline__ int lowest_key(const AttnParams& p, int pos) {
+  if (p.window > 0) return max(pos - p.window + 1, 0);
+  return p.key_chunk > 0 ? max(pos, 0) / p.key_chunk * p.key_chunk : 0;
+}
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
   const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
@@ -121,30 +143,47 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 template <int TILE, int THREADS>
 __device__ __forceinline__ void load_kv_tile(const AttnParams& p, bf16* sk, bf16* sv, long long* row_src,
                                              int tile, int kv_lo, int kv_hi, int b, int m) {
-  const size_t head_stride = (size_t)p.page_size * DH;
-  const size_t v_offset = (size_t)p.num_kv_heads * head_stride;
+  const size_t rows = (size_t)p.num_kv_heads * p.page_size;  // key rows of a page, and value rows
   for (int row = threadIdx.x; row < TILE; row += THREADS) {
     const int j = tile + row;
-    long long src = -1;
+    long long src = -1, vsrc = -1;
     if (j >= kv_lo && j < kv_hi) {
       const int page_index = j / p.page_size;
       const long long page = p.block_table[(size_t)b * p.max_pages + page_index];
-      if (page < 0 || page >= p.num_pages)
+      if (page < 0 || page >= p.num_pages) {
         atomicOr(p.err, SB_ERR_BAD_PAGE);
-      else
-        src = (long long)(((size_t)page * 2 * p.num_kv_heads + m) * head_stride +
-                          (size_t)(j - page_index * p.page_size) * DH);
+      } else {
+        const size_t base = (size_t)page * rows * (DH + DV);
+        const size_t at = (size_t)m * p.page_size + (j - page_index * p.page_size);
+        src = (long long)(base + at * DH);
+        vsrc = (long long)(base + rows * DH + at * DV);
+      }
     }
     row_src[row] = src;
+    if constexpr (!ONE_SIZE) row_src[TILE + row] = vsrc;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < TILE * CPR; i += THREADS) {
-    const int row = i / CPR, c = i - row * CPR;
-    const long long src = row_src[row];
-    const bool valid = src >= 0;
-    const bf16* g = p.cache + (valid ? src : 0) + c * 8;
-    cp_async16(sk + row * PITCH + c * 8, g, valid);
-    cp_async16(sv + row * PITCH + c * 8, g + v_offset, valid);
+  if constexpr (ONE_SIZE) {
+    const size_t v_offset = rows * DH;
+    for (int i = threadIdx.x; i < TILE * CPR; i += THREADS) {
+      const int row = i / CPR, c = i - row * CPR;
+      const long long src = row_src[row];
+      const bool valid = src >= 0;
+      const bf16* g = p.cache + (valid ? src : 0) + c * 8;
+      cp_async16(sk + row * PITCH + c * 8, g, valid);
+      cp_async16(sv + row * VPITCH + c * 8, g + v_offset, valid);
+    }
+  } else {
+    for (int i = threadIdx.x; i < TILE * CPR; i += THREADS) {
+      const int row = i / CPR, c = i - row * CPR;
+      const long long src = row_src[row];
+      cp_async16(sk + row * PITCH + c * 8, p.cache + (src >= 0 ? src : 0) + c * 8, src >= 0);
+    }
+    for (int i = threadIdx.x; i < TILE * VCPR; i += THREADS) {
+      const int row = i / VCPR, c = i - row * VCPR;
+      const long long src = row_src[TILE + row];
+      cp_async16(sv + row * VPITCH + c * 8, p.cache + (src >= 0 ? src : 0) + c * 8, src >= 0);
+    }
   }
 }
 
@@ -176,7 +215,7 @@ __device__ __forceinline__ void load_pool_tile(const AttnParams& p, bf16* sk, bf
     const bool valid = src >= 0;
     const bf16* g = p.pool + (valid ? src : 0) + c * 8;
     cp_async16(sk + row * PITCH + c * 8, g, valid);
-    cp_async16(sv + row * PITCH + c * 8, g + v_offset, valid);
+    cp_async16(sv + row * VPITCH + c * 8, g + v_offset, valid);
   }
 }
 
@@ -205,30 +244,38 @@ __device__ __forceinline__ void scores(float (&s)[NKT][4], const bf16* sq_rows, 
 // Soft cap, mask, online softmax update and P.V for one warp.  `pos_a`, `pos_b`: positions of
 // the thread's two query rows (-1 for a padding row).  `j0`: position of the first of the
 // NKT * 8 keys.  m_* are kept in log2 units.
-// The distance bias of one query row: r1 ln 2 and r2 of its head (zeros: none).
+// The distance bias of one query row: r1 ln 2 and r2 of its head, or (`linear`) r1 and 0.
 struct RowBias {
   float r1, r2;
 };
-__device__ __forceinline__ RowBias row_bias(const float* distance, int num_q_heads, int head) {
+enum { NO_BIAS = 0, LOG_BIAS = 1, LINEAR_BIAS = 2 };
+__device__ __forceinline__ int bias_kind(const AttnParams& p) {
+  return p.distance == nullptr ? NO_BIAS : (p.linear ? LINEAR_BIAS : LOG_BIAS);
+}
+__device__ __forceinline__ RowBias row_bias(const AttnParams& p, int head) {
   RowBias b{0.f, 0.f};
-  if (distance != nullptr) {
-    b.r1 = distance[head] * 0.6931471805599453f;
-    b.r2 = distance[num_q_heads + head];
+  if (p.distance != nullptr) {
+    b.r1 = p.distance[head];
+    if (!p.linear) {
+      b.r1 *= 0.6931471805599453f;
+      b.r2 = p.distance[p.num_q_heads + head];
+    }
   }
   return b;
 }
-// r1 ln(1 + r2 d) for d >= 0 keys between the query and the key.
-__device__ __forceinline__ float distance_loss(const RowBias& b, int d) {
-  return b.r1 * __log2f(fmaf(b.r2, (float)max(d, 0), 1.0f));
+// What a score loses for d >= 0 keys between the query and the key: r1 ln(1 + r2 d), or r1 d.
+__device__ __forceinline__ float distance_loss(const RowBias& b, int d, int kind) {
+  const float x = (float)max(d, 0);
+  return b.r1 * (kind == LINEAR_BIAS ? x : __log2f(fmaf(b.r2, x, 1.0f)));
 }
 
 template <int NKT>
-__device__ __forceinline__ void softmax_pv(float (&s)[NKT][4], float (&o)[DH / 8][4], float& m_a, float& m_b,
-                                           float& l_a, float& l_b, int pos_a, int pos_b, int j0, float cap,
-                                           int window, const bf16* sv, int key0, bool need_mask = true,
-                                           int pool_len = 0, bool biased = false, RowBias bias_a = RowBias{0.f, 0.f},
+__device__ __forceinline__ void softmax_pv(float (&s)[NKT][4], float (&o)[DV / 8][4], float& m_a, float& m_b,
+                                           float& l_a, float& l_b, int pos_a, int pos_b, int lo_a, int lo_b, int j0,
+                                           float cap, int window, const bf16* sv, int key0, bool need_mask = true,
+                                           int pool_len = 0, int biased = NO_BIAS, RowBias bias_a = RowBias{0.f, 0.f},
                                            RowBias bias_b = RowBias{0.f, 0.f}) {
-  // pool_len > 0: the keys are block entries j0, j0 + 1, ...; a row at `pos` sees the blocks that
+  // lo_a, lo_b: the lowest keys the two rows see.  pool_len > 0: the keys are block entries j0, j0 + 1, ...; a row at `pos` sees the blocks that
   // lie wholly before its window, j < (pos - window + 1) / pool_len.
   const int lane = threadIdx.x & 31, t = lane & 3;
   const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f;
@@ -241,10 +288,10 @@ __device__ __forceinline__ void softmax_pv(float (&s)[NKT][4], float (&o)[DH / 8
       const int pos = e < 2 ? pos_a : pos_b;
       float v = s[i][e];
       if (cap > 0.f) v = cap * fast_tanh(v * inv_cap);
-      if (biased) v -= distance_loss(e < 2 ? bias_a : bias_b, pos - j);
+      if (biased) v -= distance_loss(e < 2 ? bias_a : bias_b, pos - j, biased);
       // need_mask is false (for the whole warp) when every key of the tile is visible to every row.
       const bool keep = pool_len > 0 ? (pos - window + 1 > 0 && j < (pos - window + 1) / pool_len)
-                                     : (!need_mask || (j <= pos && (window <= 0 || pos - j < window)));
+                                     : (!need_mask || (j <= pos && j >= (e < 2 ? lo_a : lo_b)));
       v = keep ? v * LOG2E : -INFINITY;
       s[i][e] = v;
       if (e < 2) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
@@ -272,7 +319,7 @@ __device__ __forceinline__ void softmax_pv(float (&s)[NKT][4], float (&o)[DH / 8
   l_b = l_b * alpha_b + sum_b;
   if (__any_sync(0xffffffffu, alpha_a != 1.f || alpha_b != 1.f)) {  // the running maxima rarely move
 #pragma unroll
-    for (int d = 0; d < DH / 8; ++d) {
+    for (int d = 0; d < DV / 8; ++d) {
       o[d][0] *= alpha_a;
       o[d][1] *= alpha_a;
       o[d][2] *= alpha_b;
@@ -287,9 +334,9 @@ __device__ __forceinline__ void softmax_pv(float (&s)[NKT][4], float (&o)[DH / 8
     a[2] = pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]);
     a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
-    for (int dp = 0; dp < DH / 16; ++dp) {
+    for (int dp = 0; dp < DV / 16; ++dp) {
       uint32_t r[4];
-      ldmatrix_x4_trans(r, sv + (key0 + kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * PITCH + dp * 16 + (lane >> 4) * 8);
+      ldmatrix_x4_trans(r, sv + (key0 + kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * VPITCH + dp * 16 + (lane >> 4) * 8);
       mma16816(o[2 * dp], a, r[0], r[1]);
       mma16816(o[2 * dp + 1], a, r[2], r[3]);
     }
@@ -310,8 +357,8 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* sq = reinterpret_cast<bf16*>(smem_raw);  // [BM][PITCH]
   bf16* sk = sq + BM * PITCH;                    // [2][BN][PITCH]
-  bf16* sv = sk + 2 * BN * PITCH;                // [2][BN][PITCH]
-  __shared__ long long row_src[2][BN];
+  bf16* sv = sk + 2 * BN * PITCH;                // [2][BN][VPITCH]
+  __shared__ long long row_src[2][SRC * BN];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
   const int wm = warp % WM, wn = warp / WM;
   const int b = p.items[2 * blockIdx.x], i0 = p.items[2 * blockIdx.x + 1], m = blockIdx.y;
@@ -328,8 +375,8 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
     cp_async16(sq + row * PITCH + c * 8, p.q + ((size_t)(row0 + tok) * p.num_q_heads + h) * DH + c * 8, valid);
   }
   const int p0 = qs + i0, p1 = qs + i0 + ntok - 1;
-  const int kv_lo = p.window > 0 ? max(qs - p.window + 1, 0) : 0;  // lowest key the request still holds
-  const int lo = p.window > 0 ? max(p0 - p.window + 1, 0) : 0;     // lowest key this tile can see
+  const int kv_lo = lowest_key(p, qs);  // lowest key the request still holds
+  const int lo = lowest_key(p, p0);     // lowest key this tile can see
   const int kv_hi = p1 + 1;
   const int tile0 = (lo / BN) * BN;
   const int n_tiles = (kv_hi - tile0 + BN - 1) / BN;
@@ -337,10 +384,10 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
   const int n_blocks = (p.pool != nullptr && p.window > 0 && p1 - p.window + 1 > 0) ? (p1 - p.window + 1) / p.pool_len : 0;
   const int n_pool_tiles = (n_blocks + BN - 1) / BN;
   auto load_tile = [&](int it, int stage) {
-    if (it < n_pool_tiles)
-      load_pool_tile<BN, THREADS>(p, sk + stage * BN * PITCH, sv + stage * BN * PITCH, row_src[stage], it * BN, n_blocks, b, m);
+    if (ONE_SIZE && it < n_pool_tiles)
+      load_pool_tile<BN, THREADS>(p, sk + stage * BN * PITCH, sv + stage * BN * VPITCH, row_src[stage], it * BN, n_blocks, b, m);
     else
-      load_kv_tile<BN, THREADS>(p, sk + stage * BN * PITCH, sv + stage * BN * PITCH, row_src[stage],
+      load_kv_tile<BN, THREADS>(p, sk + stage * BN * PITCH, sv + stage * BN * VPITCH, row_src[stage],
                                 tile0 + (it - n_pool_tiles) * BN, kv_lo, kv_hi, b, m);
   };
   load_tile(0, 0);
@@ -350,15 +397,17 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
   const int pos_a = ra < rows_valid ? p0 + ra / group : -1;
   const int pos_b = rb < rows_valid ? p0 + rb / group : -1;
   // Positions of this warp's first and last row, for deciding whether a tile needs masking.
-  const bool biased = p.distance != nullptr;
-  const RowBias bias_a = row_bias(p.distance, p.num_q_heads, m * group + ra % group);
-  const RowBias bias_b = row_bias(p.distance, p.num_q_heads, m * group + rb % group);
+  const int biased = bias_kind(p);
+  const RowBias bias_a = row_bias(p, m * group + ra % group);
+  const RowBias bias_b = row_bias(p, m * group + rb % group);
+  const int lo_a = lowest_key(p, pos_a), lo_b = lowest_key(p, pos_b);
   const bool rows_full = wm * 16 + 15 < rows_valid;
   const int warp_pos_lo = p0 + (wm * 16) / group, warp_pos_hi = p0 + (wm * 16 + 15) / group;
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
-  float o[DH / 8][4];
+  const int warp_lo = lowest_key(p, warp_pos_hi);
+  float o[DV / 8][4];
 #pragma unroll
-  for (int d = 0; d < DH / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
+  for (int d = 0; d < DV / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
 
   for (int it = 0; it < n_pool_tiles + n_tiles; ++it) {
     const int stage = it & 1;
@@ -374,12 +423,12 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
     // this warp's first key of the tile (its first block entry, in a tile of those)
     const int j0 = (pooled ? it * BN : tile0 + (it - n_pool_tiles) * BN) + wn * KEYS;
     // Every key visible to every row of the warp: below the lowest row's position, inside the
-    // highest row's window.
-    const bool need_mask = !rows_full || j0 + KEYS - 1 > warp_pos_lo || (p.window > 0 && warp_pos_hi - j0 >= p.window);
+    // highest row's window or chunk.
+    const bool need_mask = !rows_full || j0 + KEYS - 1 > warp_pos_lo || j0 < warp_lo;
     float s[KEYS / 8][4];
     scores<KEYS / 8>(s, sq + wm * 16 * PITCH, sk + stage * BN * PITCH, wn * KEYS);
-    softmax_pv<KEYS / 8>(s, o, m_a, m_b, l_a, l_b, pos_a, pos_b, j0, p.cap, p.window, sv + stage * BN * PITCH,
-                         wn * KEYS, need_mask, pooled ? p.pool_len : 0, biased && !pooled, bias_a, bias_b);
+    softmax_pv<KEYS / 8>(s, o, m_a, m_b, l_a, l_b, pos_a, pos_b, lo_a, lo_b, j0, p.cap, p.window, sv + stage * BN * VPITCH,
+                         wn * KEYS, need_mask, pooled ? p.pool_len : 0, pooled ? NO_BIAS : biased, bias_a, bias_b);
     __syncthreads();
   }
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 1);
@@ -388,7 +437,7 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
   if (WN > 1) {
     // The key groups of a row group merge: warps of group 1 hand (max, sum, output) to group 0.
-    float* xm = reinterpret_cast<float*>(sk);  // [BM] max, [BM] sum, then [BM][DH] (the tiles are no longer needed)
+    float* xm = reinterpret_cast<float*>(sk);  // [BM] max, [BM] sum, then [BM][DV] (the tiles are no longer needed)
     float* xl = xm + BM;
     float* xo = xl + BM;
     if (wn == 1) {
@@ -397,9 +446,9 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
         xl[ra] = l_a; xl[rb] = l_b;
       }
 #pragma unroll
-      for (int d = 0; d < DH / 8; ++d) {
-        *reinterpret_cast<float2*>(xo + (size_t)ra * DH + d * 8 + 2 * t) = make_float2(o[d][0], o[d][1]);
-        *reinterpret_cast<float2*>(xo + (size_t)rb * DH + d * 8 + 2 * t) = make_float2(o[d][2], o[d][3]);
+      for (int d = 0; d < DV / 8; ++d) {
+        *reinterpret_cast<float2*>(xo + (size_t)ra * DV + d * 8 + 2 * t) = make_float2(o[d][0], o[d][1]);
+        *reinterpret_cast<float2*>(xo + (size_t)rb * DV + d * 8 + 2 * t) = make_float2(o[d][2], o[d][3]);
       }
     }
     __syncthreads();
@@ -411,27 +460,33 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
     const float ta = fast_exp2(om_a - ua), tb = fast_exp2(om_b - ub);   // scale of the other's
     l_a = l_a * sa + xl[ra] * ta;
     l_b = l_b * sb + xl[rb] * tb;
+    m_a = nm_a;
+    m_b = nm_b;
 #pragma unroll
-    for (int d = 0; d < DH / 8; ++d) {
-      const float2 oa = *reinterpret_cast<const float2*>(xo + (size_t)ra * DH + d * 8 + 2 * t);
-      const float2 ob = *reinterpret_cast<const float2*>(xo + (size_t)rb * DH + d * 8 + 2 * t);
+    for (int d = 0; d < DV / 8; ++d) {
+      const float2 oa = *reinterpret_cast<const float2*>(xo + (size_t)ra * DV + d * 8 + 2 * t);
+      const float2 ob = *reinterpret_cast<const float2*>(xo + (size_t)rb * DV + d * 8 + 2 * t);
       o[d][0] = o[d][0] * sa + oa.x * ta;
       o[d][1] = o[d][1] * sa + oa.y * ta;
       o[d][2] = o[d][2] * sb + ob.x * tb;
       o[d][3] = o[d][3] * sb + ob.y * tb;
     }
   }
+  if (p.sink != nullptr) {  // exp(sink) has no value: it only joins the sums (relative to the rows' maxima)
+    l_a += fast_exp2(p.sink[m * group + ra % group] * LOG2E - m_a);
+    l_b += fast_exp2(p.sink[m * group + rb % group] * LOG2E - m_b);
+  }
   const float inv_a = l_a > 0.f ? 1.0f / l_a : 0.f, inv_b = l_b > 0.f ? 1.0f / l_b : 0.f;
   if (ra < rows_valid) {
-    bf16* op = p.out + ((size_t)(row0 + i0 + ra / group) * p.num_q_heads + m * group + ra % group) * DH;
+    bf16* op = p.out + ((size_t)(row0 + i0 + ra / group) * p.num_q_heads + m * group + ra % group) * DV;
 #pragma unroll
-    for (int d = 0; d < DH / 8; ++d)
+    for (int d = 0; d < DV / 8; ++d)
       *reinterpret_cast<uint32_t*>(op + d * 8 + 2 * t) = pack_bf16(o[d][0] * inv_a, o[d][1] * inv_a);
   }
   if (rb < rows_valid) {
-    bf16* op = p.out + ((size_t)(row0 + i0 + rb / group) * p.num_q_heads + m * group + rb % group) * DH;
+    bf16* op = p.out + ((size_t)(row0 + i0 + rb / group) * p.num_q_heads + m * group + rb % group) * DV;
 #pragma unroll
-    for (int d = 0; d < DH / 8; ++d)
+    for (int d = 0; d < DV / 8; ++d)
       *reinterpret_cast<uint32_t*>(op + d * 8 + 2 * t) = pack_bf16(o[d][2] * inv_b, o[d][3] * inv_b);
   }
 }
@@ -454,9 +509,9 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* sq = reinterpret_cast<bf16*>(smem_raw);  // [16][PITCH]
   bf16* sk = sq + 16 * PITCH;                    // [STAGES][DEC_BN][PITCH]
-  bf16* sv = sk + DEC_STAGES * DEC_BN * PITCH;   // [STAGES][DEC_BN][PITCH]
+  bf16* sv = sk + DEC_STAGES * DEC_BN * PITCH;   // [STAGES][DEC_BN][VPITCH]
   __shared__ int s_work;
-  __shared__ long long row_src[DEC_STAGES][DEC_BN];
+  __shared__ long long row_src[DEC_STAGES][SRC * DEC_BN];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
   const int group = p.num_q_heads / p.num_kv_heads;
   for (;;) {
@@ -470,7 +525,7 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
     if (b < 0) continue;  // filler item of a fixed-size work list
     const int row0 = p.cu_q[b], q_len = p.cu_q[b + 1] - row0, qs = p.q_start[b];
     const int rows_valid = q_len * group;  // <= 16 by the host's routing
-    const int kv_lo = p.window > 0 ? max(qs - p.window + 1, 0) : 0;
+    const int kv_lo = lowest_key(p, qs);
     const int kv_hi = qs + q_len;
     const int begin = max(chunk_index * p.chunk, (kv_lo / 64) * 64);
     const int end = min((chunk_index + 1) * p.chunk, kv_hi);
@@ -485,18 +540,19 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
 #pragma unroll
     for (int st = 0; st < DEC_STAGES - 1; ++st) {
       if (st < n_tiles)  // uniform over the block
-        load_kv_tile<DEC_BN, DEC_NT>(p, sk + st * DEC_BN * PITCH, sv + st * DEC_BN * PITCH, row_src[st],
+        load_kv_tile<DEC_BN, DEC_NT>(p, sk + st * DEC_BN * PITCH, sv + st * DEC_BN * VPITCH, row_src[st],
                                      begin + st * DEC_BN, kv_lo, end, b, m);
       cp_async_commit();
     }
     const int pos_a = g < rows_valid ? qs + g / group : -1;
     const int pos_b = g + 8 < rows_valid ? qs + (g + 8) / group : -1;
-    const RowBias bias_a = row_bias(p.distance, p.num_q_heads, m * group + g % group);
-    const RowBias bias_b = row_bias(p.distance, p.num_q_heads, m * group + (g + 8) % group);
+    const RowBias bias_a = row_bias(p, m * group + g % group);
+    const RowBias bias_b = row_bias(p, m * group + (g + 8) % group);
+    const int lo_a = lowest_key(p, pos_a), lo_b = lowest_key(p, pos_b);
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
-    float o[DH / 8][4];
+    float o[DV / 8][4];
 #pragma unroll
-    for (int d = 0; d < DH / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
+    for (int d = 0; d < DV / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
 
     for (int it = 0; it < n_tiles; ++it) {
       const int stage = it % DEC_STAGES;
@@ -504,14 +560,14 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
       __syncthreads();  // tile `it` has landed; everyone is done with tile it - 1
       if (it + DEC_STAGES - 1 < n_tiles) {
         const int st = (it + DEC_STAGES - 1) % DEC_STAGES;
-        load_kv_tile<DEC_BN, DEC_NT>(p, sk + st * DEC_BN * PITCH, sv + st * DEC_BN * PITCH, row_src[st],
+        load_kv_tile<DEC_BN, DEC_NT>(p, sk + st * DEC_BN * PITCH, sv + st * DEC_BN * VPITCH, row_src[st],
                                      begin + (it + DEC_STAGES - 1) * DEC_BN, kv_lo, end, b, m);
       }
       cp_async_commit();
       float s[2][4];
       scores<2>(s, sq, sk + stage * DEC_BN * PITCH, warp * 16);
-      softmax_pv<2>(s, o, m_a, m_b, l_a, l_b, pos_a, pos_b, begin + it * DEC_BN + warp * 16, p.cap, p.window,
-                    sv + stage * DEC_BN * PITCH, warp * 16, true, 0, p.distance != nullptr, bias_a, bias_b);
+      softmax_pv<2>(s, o, m_a, m_b, l_a, l_b, pos_a, pos_b, lo_a, lo_b, begin + it * DEC_BN + warp * 16, p.cap, p.window,
+                    sv + stage * DEC_BN * VPITCH, warp * 16, true, 0, bias_kind(p), bias_a, bias_b);
     }
     cp_async_wait<0>();
     __syncthreads();
@@ -521,7 +577,7 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
 
     // Merge the warps (each saw its share of every tile) through shared memory.
-    float* wm = reinterpret_cast<float*>(sk);  // [W][16] max, [W][16] sum, then [W][rows_valid][DH]
+    float* wm = reinterpret_cast<float*>(sk);  // [W][16] max, [W][16] sum, then [W][rows_valid][DV]
     float* wl = wm + DEC_WARPS * 16;
     float* wo = wl + DEC_WARPS * 16;
     if (t == 0) {
@@ -532,22 +588,22 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
     }
     if (g < rows_valid) {
 #pragma unroll
-      for (int d = 0; d < DH / 8; ++d) {
-        wo[((size_t)warp * rows_valid + g) * DH + d * 8 + 2 * t] = o[d][0];
-        wo[((size_t)warp * rows_valid + g) * DH + d * 8 + 2 * t + 1] = o[d][1];
+      for (int d = 0; d < DV / 8; ++d) {
+        wo[((size_t)warp * rows_valid + g) * DV + d * 8 + 2 * t] = o[d][0];
+        wo[((size_t)warp * rows_valid + g) * DV + d * 8 + 2 * t + 1] = o[d][1];
       }
     }
     if (g + 8 < rows_valid) {
 #pragma unroll
-      for (int d = 0; d < DH / 8; ++d) {
-        wo[((size_t)warp * rows_valid + g + 8) * DH + d * 8 + 2 * t] = o[d][2];
-        wo[((size_t)warp * rows_valid + g + 8) * DH + d * 8 + 2 * t + 1] = o[d][3];
+      for (int d = 0; d < DV / 8; ++d) {
+        wo[((size_t)warp * rows_valid + g + 8) * DV + d * 8 + 2 * t] = o[d][2];
+        wo[((size_t)warp * rows_valid + g + 8) * DV + d * 8 + 2 * t + 1] = o[d][3];
       }
     }
     __syncthreads();
     const size_t pidx = (size_t)item * p.num_kv_heads + m;
-    for (int i = threadIdx.x; i < rows_valid * DH; i += DEC_NT) {
-      const int r = i / DH, d = i - r * DH;
+    for (int i = threadIdx.x; i < rows_valid * DV; i += DEC_NT) {
+      const int r = i / DV, d = i - r * DV;
       float mx = -INFINITY;
 #pragma unroll
       for (int w = 0; w < DEC_WARPS; ++w) mx = fmaxf(mx, wm[w * 16 + r]);
@@ -556,11 +612,11 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
 #pragma unroll
         for (int w = 0; w < DEC_WARPS; ++w) {
           const float sc = fast_exp2(wm[w * 16 + r] - mx);
-          num += sc * wo[((size_t)w * rows_valid + r) * DH + d];
+          num += sc * wo[((size_t)w * rows_valid + r) * DV + d];
           den += sc * wl[w * 16 + r];
         }
       }
-      p.part_o[(pidx * p.rows_max + r) * DH + d] = den > 0.f ? num / den : 0.f;
+      p.part_o[(pidx * p.rows_max + r) * DV + d] = den > 0.f ? num / den : 0.f;
       if (d == 0) {
         p.part_ml[(pidx * p.rows_max + r) * 2] = mx;
         p.part_ml[(pidx * p.rows_max + r) * 2 + 1] = den;
@@ -642,16 +698,16 @@ constexpr int D8_BN = DH > 128 ? 32 : 64;  // keys per tile
 constexpr int D8_WARPS = D8_BN / 16;
 constexpr int D8_NT = D8_WARPS * 32;
 constexpr int D8_STAGES = 2;
-constexpr bool TMA_OK = DH % 64 == 0;        // 128-byte swizzled boxes of 64 columns
+constexpr bool TMA_OK = ONE_SIZE && DH % 64 == 0;  // 128-byte swizzled boxes of 64 columns
 constexpr int SLABS = TMA_OK ? DH / 64 : 1;  // 64-column slabs of a tile in the swizzled layout
 constexpr int SLAB_ELEMS = D8_BN * 64;       // elements of one slab of one tile
 
 // Element (row, dim) of a tile.  Swizzled layout: [slab][row][64 columns], the 16-byte chunks of
 // a 128-byte row XOR-ed with the row's low three bits (what the TMA's 128-byte swizzle writes).
-template <bool USE_TMA>
+template <bool USE_TMA, int ROW_PITCH = PITCH>
 __device__ __forceinline__ const bf16* tile_at(const bf16* tile, int row, int dim) {
   if (USE_TMA) return tile + (dim >> 6) * SLAB_ELEMS + row * 64 + ((((dim & 63) >> 3) ^ (row & 7)) << 3) + (dim & 7);
-  return tile + row * PITCH + dim;
+  return tile + row * ROW_PITCH + dim;
 }
 
 template <bool USE_TMA>
@@ -660,7 +716,7 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
                     int box_rows) {
   pdl_wait();
   pdl_launch_dependents();
-  constexpr int TILE_ELEMS = USE_TMA ? D8_BN * DH : D8_BN * PITCH;
+  constexpr int TILE_ELEMS = USE_TMA ? D8_BN * DH : D8_BN * PITCH, VTILE_ELEMS = USE_TMA ? D8_BN * DV : D8_BN * VPITCH;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   // The swizzle pattern is a function of the address: tiles start on a 1024-byte boundary
   // (the launch adds 1024 bytes of slack for this).
@@ -668,7 +724,7 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
   bf16* sk = reinterpret_cast<bf16*>(aligned);  // [STAGES] key tiles
   bf16* sv = sk + D8_STAGES * TILE_ELEMS;        // [STAGES] value tiles
   __shared__ __align__(8) uint64_t full[D8_STAGES];
-  __shared__ long long row_src[D8_STAGES][D8_BN];
+  __shared__ long long row_src[D8_STAGES][SRC * D8_BN];
   __shared__ int s_work;
   __shared__ int s_failed;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
@@ -693,7 +749,7 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
     if (b < 0) continue;  // filler item of a fixed-size work list
     const int row0 = p.cu_q[b], q_len = p.cu_q[b + 1] - row0, qs = p.q_start[b];
     const int rows_valid = q_len * group;  // <= 8 by the host's routing
-    const int kv_lo = p.window > 0 ? max(qs - p.window + 1, 0) : 0;
+    const int kv_lo = lowest_key(p, qs);
     const int kv_hi = qs + q_len;
     const int begin = max(chunk_index * p.chunk, (kv_lo / 64) * 64);
     const int end = min((chunk_index + 1) * p.chunk, kv_hi);
@@ -728,11 +784,11 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
 #pragma unroll
           for (int sl = 0; sl < SLABS; ++sl) {
             tma_load_box(sk + (size_t)stage * TILE_ELEMS + sl * SLAB_ELEMS + r * 64, &tmap, sl * 64, (int)krow, &full[stage]);
-            tma_load_box(sv + (size_t)stage * TILE_ELEMS + sl * SLAB_ELEMS + r * 64, &tmap, sl * 64, (int)vrow, &full[stage]);
+            tma_load_box(sv + (size_t)stage * VTILE_ELEMS + sl * SLAB_ELEMS + r * 64, &tmap, sl * 64, (int)vrow, &full[stage]);
           }
         }
       } else {
-        load_kv_tile<D8_BN, D8_NT>(p, sk + (size_t)stage * TILE_ELEMS, sv + (size_t)stage * TILE_ELEMS, row_src[stage],
+        load_kv_tile<D8_BN, D8_NT>(p, sk + (size_t)stage * TILE_ELEMS, sv + (size_t)stage * VTILE_ELEMS, row_src[stage],
                                    j0, kv_lo, end, b, m);
       }
     };
@@ -758,13 +814,14 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
     const int pos0 = 2 * t < rows_valid ? qs + (2 * t) / group : -1;
     const int pos1 = 2 * t + 1 < rows_valid ? qs + (2 * t + 1) / group : -1;
     const float inv_cap = p.cap > 0.f ? 1.0f / p.cap : 0.f;
-    const bool biased = p.distance != nullptr;
-    const RowBias bias0 = row_bias(p.distance, p.num_q_heads, m * group + (2 * t) % group);
-    const RowBias bias1 = row_bias(p.distance, p.num_q_heads, m * group + (2 * t + 1) % group);
+    const int biased = bias_kind(p);
+    const RowBias bias0 = row_bias(p, m * group + (2 * t) % group);
+    const RowBias bias1 = row_bias(p, m * group + (2 * t + 1) % group);
+    const int lo0 = lowest_key(p, pos0), lo1 = lowest_key(p, pos1);
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-    float o[DH / 16][4];  // out^T: [dims 16 blk + g | g + 8][rows 2t | 2t + 1]
+    float o[DV / 16][4];  // out^T: [dims 16 blk + g | g + 8][rows 2t | 2t + 1]
 #pragma unroll
-    for (int d = 0; d < DH / 16; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
+    for (int d = 0; d < DV / 16; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
 
     bool ok = true;
     for (int it = 0; it < n_tiles; ++it) {
@@ -784,14 +841,14 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
       }
       if (landed) {
         const bf16* kt = sk + (size_t)stage * TILE_ELEMS;
-        const bf16* vt = sv + (size_t)stage * TILE_ELEMS;
+        const bf16* vt = sv + (size_t)stage * VTILE_ELEMS;
         const int key0 = warp * 16;  // this warp's keys of the tile
         const int j_first = begin + it * D8_BN + key0;
         if (USE_TMA && (j_first < kv_lo || j_first + 16 > end)) {
           // Some of this warp's 16 keys are not the request's: their value rows must read as zeros
           // (0 * garbage could be NaN).  Only this warp reads these rows.
-          for (int i = lane; i < 16 * (DH / 8); i += 32) {
-            const int r = i / (DH / 8), c = i - r * (DH / 8);
+          for (int i = lane; i < 16 * (DV / 8); i += 32) {
+            const int r = i / (DV / 8), c = i - r * (DV / 8);
             const int j = j_first + r;
             if (j < kv_lo || j >= end)
               *reinterpret_cast<uint4*>(const_cast<bf16*>(tile_at<true>(vt, key0 + r, c * 8))) = make_uint4(0, 0, 0, 0);
@@ -819,8 +876,8 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
           if (p.cap > 0.f) v = p.cap * fast_tanh(v * inv_cap);
           const int j = j_first + g + (e >> 1) * 8;
           const int pos = (e & 1) ? pos1 : pos0;
-          if (biased) v -= distance_loss((e & 1) ? bias1 : bias0, pos - j);
-          const bool keep = j <= pos && (p.window <= 0 || pos - j < p.window);
+          if (biased) v -= distance_loss((e & 1) ? bias1 : bias0, pos - j, biased);
+          const bool keep = j <= pos && j >= ((e & 1) ? lo1 : lo0);
           sc[e] = keep ? v * LOG2E : -INFINITY;
         }
         float mx0 = fmaxf(sc[0], sc[2]), mx1 = fmaxf(sc[1], sc[3]);
@@ -840,7 +897,7 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
         l1 = l1 * alpha1 + p1 + p3;
         if (__any_sync(0xffffffffu, alpha0 != 1.f || alpha1 != 1.f)) {
 #pragma unroll
-          for (int d = 0; d < DH / 16; ++d) {
+          for (int d = 0; d < DV / 16; ++d) {
             o[d][0] *= alpha0;
             o[d][1] *= alpha1;
             o[d][2] *= alpha0;
@@ -851,9 +908,9 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
         const uint32_t b0 = movmatrix_trans(pack_bf16(p0, p1));
         const uint32_t b1 = movmatrix_trans(pack_bf16(p2, p3));
 #pragma unroll
-        for (int d = 0; d < DH / 16; ++d) {
+        for (int d = 0; d < DV / 16; ++d) {
           uint32_t a[4];
-          ldmatrix_x4_trans(a, tile_at<USE_TMA>(vt, key0 + ((lane >> 4) & 1) * 8 + (lane & 7), d * 16 + ((lane >> 3) & 1) * 8));
+          ldmatrix_x4_trans(a, tile_at<USE_TMA, VPITCH>(vt, key0 + ((lane >> 4) & 1) * 8 + (lane & 7), d * 16 + ((lane >> 3) & 1) * 8));
           mma16816(o[d], a, b0, b1);
         }
       }
@@ -883,7 +940,7 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
       l1 += __shfl_xor_sync(0xffffffffu, l1, off);
     }
     // Merge the warps through shared memory (the tiles are no longer needed).
-    float* wm = reinterpret_cast<float*>(sk);  // [W][8] max, [W][8] sum, then [W][rows_valid][DH]
+    float* wm = reinterpret_cast<float*>(sk);  // [W][8] max, [W][8] sum, then [W][rows_valid][DV]
     float* wl = wm + D8_WARPS * 8;
     float* wo = wl + D8_WARPS * 8;
     if (g == 0) {
@@ -893,20 +950,20 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
       wl[warp * 8 + 2 * t + 1] = l1;
     }
 #pragma unroll
-    for (int d = 0; d < DH / 16; ++d) {
+    for (int d = 0; d < DV / 16; ++d) {
       if (2 * t < rows_valid) {
-        wo[((size_t)warp * rows_valid + 2 * t) * DH + d * 16 + g] = o[d][0];
-        wo[((size_t)warp * rows_valid + 2 * t) * DH + d * 16 + g + 8] = o[d][2];
+        wo[((size_t)warp * rows_valid + 2 * t) * DV + d * 16 + g] = o[d][0];
+        wo[((size_t)warp * rows_valid + 2 * t) * DV + d * 16 + g + 8] = o[d][2];
       }
       if (2 * t + 1 < rows_valid) {
-        wo[((size_t)warp * rows_valid + 2 * t + 1) * DH + d * 16 + g] = o[d][1];
-        wo[((size_t)warp * rows_valid + 2 * t + 1) * DH + d * 16 + g + 8] = o[d][3];
+        wo[((size_t)warp * rows_valid + 2 * t + 1) * DV + d * 16 + g] = o[d][1];
+        wo[((size_t)warp * rows_valid + 2 * t + 1) * DV + d * 16 + g + 8] = o[d][3];
       }
     }
     __syncthreads();
     const size_t pidx = (size_t)item * p.num_kv_heads + m;
-    for (int i = threadIdx.x; i < rows_valid * DH; i += D8_NT) {
-      const int r = i / DH, d = i - r * DH;
+    for (int i = threadIdx.x; i < rows_valid * DV; i += D8_NT) {
+      const int r = i / DV, d = i - r * DV;
       float mx = -INFINITY;
 #pragma unroll
       for (int w = 0; w < D8_WARPS; ++w) mx = fmaxf(mx, wm[w * 8 + r]);
@@ -915,11 +972,11 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
 #pragma unroll
         for (int w = 0; w < D8_WARPS; ++w) {
           const float scale = fast_exp2(wm[w * 8 + r] - mx);
-          num += scale * wo[((size_t)w * rows_valid + r) * DH + d];
+          num += scale * wo[((size_t)w * rows_valid + r) * DV + d];
           den += scale * wl[w * 8 + r];
         }
       }
-      p.part_o[(pidx * p.rows_max + r) * DH + d] = den > 0.f ? num / den : 0.f;
+      p.part_o[(pidx * p.rows_max + r) * DV + d] = den > 0.f ? num / den : 0.f;
       if (d == 0) {
         p.part_ml[(pidx * p.rows_max + r) * 2] = mx;
         p.part_ml[(pidx * p.rows_max + r) * 2 + 1] = den;
@@ -957,7 +1014,7 @@ __device__ __forceinline__ bool ws_item(const AttnParams& p, int work, WsItem& w
   w.row0 = p.cu_q[w.b];
   w.q_len = p.cu_q[w.b + 1] - w.row0;
   w.qs = p.q_start[w.b];
-  w.kv_lo = p.window > 0 ? max(w.qs - p.window + 1, 0) : 0;
+  w.kv_lo = lowest_key(p, w.qs);
   const int kv_hi = w.qs + w.q_len;
   w.begin = max(chunk_index * p.chunk, (w.kv_lo / 64) * 64);
   w.end = min((chunk_index + 1) * p.chunk, kv_hi);
@@ -972,7 +1029,7 @@ __device__ __forceinline__ void mbar_arrive_one(uint64_t* bar) {
 __global__ void __launch_bounds__(WS_NT)
 attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, const __grid_constant__ CUtensorMap tmap,
                       int box_rows) {
-  constexpr int TILE_ELEMS = D8_BN * DH;
+  constexpr int TILE_ELEMS = D8_BN * DH, VTILE_ELEMS = D8_BN * DV;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   unsigned char* aligned = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
   bf16* sk = reinterpret_cast<bf16*>(aligned);  // [STAGES] key tiles
@@ -1053,7 +1110,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
 #pragma unroll
           for (int sl = 0; sl < SLABS; ++sl) {
             tma_load_box(sk + (size_t)stage * TILE_ELEMS + sl * SLAB_ELEMS + r * 64, &tmap, sl * 64, (int)krow, &full[stage]);
-            tma_load_box(sv + (size_t)stage * TILE_ELEMS + sl * SLAB_ELEMS + r * 64, &tmap, sl * 64, (int)vrow, &full[stage]);
+            tma_load_box(sv + (size_t)stage * VTILE_ELEMS + sl * SLAB_ELEMS + r * 64, &tmap, sl * 64, (int)vrow, &full[stage]);
           }
         }
       }
@@ -1081,7 +1138,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
     if (w.n_tiles == 0) {
       // Nothing of this chunk is visible: an empty partial result.
       if (warp == 0) {
-        for (int i = lane; i < rows_valid * DH; i += 32) p.part_o[pidx * p.rows_max * DH + i] = 0.f;
+        for (int i = lane; i < rows_valid * DV; i += 32) p.part_o[pidx * p.rows_max * DV + i] = 0.f;
         if (lane < rows_valid) {
           p.part_ml[(pidx * p.rows_max + lane) * 2] = -INFINITY;
           p.part_ml[(pidx * p.rows_max + lane) * 2 + 1] = 0.f;
@@ -1103,13 +1160,14 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
     const int pos0 = 2 * t < rows_valid ? w.qs + (2 * t) / group : -1;
     const int pos1 = 2 * t + 1 < rows_valid ? w.qs + (2 * t + 1) / group : -1;
     const float inv_cap = p.cap > 0.f ? 1.0f / p.cap : 0.f;
-    const bool biased = p.distance != nullptr;
-    const RowBias bias0 = row_bias(p.distance, p.num_q_heads, w.m * group + (2 * t) % group);
-    const RowBias bias1 = row_bias(p.distance, p.num_q_heads, w.m * group + (2 * t + 1) % group);
+    const int biased = bias_kind(p);
+    const RowBias bias0 = row_bias(p, w.m * group + (2 * t) % group);
+    const RowBias bias1 = row_bias(p, w.m * group + (2 * t + 1) % group);
+    const int lo0 = lowest_key(p, pos0), lo1 = lowest_key(p, pos1);
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-    float o[DH / 16][4];
+    float o[DV / 16][4];
 #pragma unroll
-    for (int d = 0; d < DH / 16; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
+    for (int d = 0; d < DV / 16; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
 
     int last_stage = 0;
     for (int it = 0; it < w.n_tiles; ++it, ++seq) {
@@ -1120,13 +1178,13 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
         return;
       }
       const bf16* kt = sk + (size_t)stage * TILE_ELEMS;
-      const bf16* vt = sv + (size_t)stage * TILE_ELEMS;
+      const bf16* vt = sv + (size_t)stage * VTILE_ELEMS;
       const int key0 = warp * 16;
       const int j_first = w.begin + it * D8_BN + key0;
       if (j_first < w.kv_lo || j_first + 16 > w.end) {
         // Value rows of keys that are not the request's must read as zeros (only this warp reads them).
-        for (int i = lane; i < 16 * (DH / 8); i += 32) {
-          const int r = i / (DH / 8), c = i - r * (DH / 8);
+        for (int i = lane; i < 16 * (DV / 8); i += 32) {
+          const int r = i / (DV / 8), c = i - r * (DV / 8);
           const int j = j_first + r;
           if (j < w.kv_lo || j >= w.end)
             *reinterpret_cast<uint4*>(const_cast<bf16*>(tile_at<true>(vt, key0 + r, c * 8))) = make_uint4(0, 0, 0, 0);
@@ -1151,8 +1209,8 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
         if (p.cap > 0.f) v = p.cap * fast_tanh(v * inv_cap);
         const int j = j_first + g + (e >> 1) * 8;
         const int pos = (e & 1) ? pos1 : pos0;
-        if (biased) v -= distance_loss((e & 1) ? bias1 : bias0, pos - j);
-        const bool keep = j <= pos && (p.window <= 0 || pos - j < p.window);
+        if (biased) v -= distance_loss((e & 1) ? bias1 : bias0, pos - j, biased);
+        const bool keep = j <= pos && j >= ((e & 1) ? lo1 : lo0);
         sc[e] = keep ? v * LOG2E : -INFINITY;
       }
       float mx0 = fmaxf(sc[0], sc[2]), mx1 = fmaxf(sc[1], sc[3]);
@@ -1172,7 +1230,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
       l1 = l1 * alpha1 + p1 + p3;
       if (__any_sync(0xffffffffu, alpha0 != 1.f || alpha1 != 1.f)) {
 #pragma unroll
-        for (int d = 0; d < DH / 16; ++d) {
+        for (int d = 0; d < DV / 16; ++d) {
           o[d][0] *= alpha0;
           o[d][1] *= alpha1;
           o[d][2] *= alpha0;
@@ -1182,7 +1240,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
       const uint32_t b0 = movmatrix_trans(pack_bf16(p0, p1));
       const uint32_t b1 = movmatrix_trans(pack_bf16(p2, p3));
 #pragma unroll
-      for (int d = 0; d < DH / 16; ++d) {
+      for (int d = 0; d < DV / 16; ++d) {
         uint32_t a[4];
         ldmatrix_x4_trans(a, tile_at<true>(vt, key0 + ((lane >> 4) & 1) * 8 + (lane & 7), d * 16 + ((lane >> 3) & 1) * 8));
         mma16816(o[d], a, b0, b1);
@@ -1201,7 +1259,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
     // Merge the consumer warps in the last tile's stage: all have left it when the first
     // consumer barrier is passed (the producer cannot refill it before `empty` is signalled).
     asm volatile("bar.sync 1, %0;\n" ::"n"(D8_WARPS * 32) : "memory");
-    float* wo = reinterpret_cast<float*>(sk + (size_t)last_stage * TILE_ELEMS);  // [W][rows_valid][DH]
+    float* wo = reinterpret_cast<float*>(sk + (size_t)last_stage * TILE_ELEMS);  // [W][rows_valid][DV]
     if (g == 0) {
       wm[warp * 8 + 2 * t] = m0;
       wm[warp * 8 + 2 * t + 1] = m1;
@@ -1209,19 +1267,19 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
       wl[warp * 8 + 2 * t + 1] = l1;
     }
 #pragma unroll
-    for (int d = 0; d < DH / 16; ++d) {
+    for (int d = 0; d < DV / 16; ++d) {
       if (2 * t < rows_valid) {
-        wo[((size_t)warp * rows_valid + 2 * t) * DH + d * 16 + g] = o[d][0];
-        wo[((size_t)warp * rows_valid + 2 * t) * DH + d * 16 + g + 8] = o[d][2];
+        wo[((size_t)warp * rows_valid + 2 * t) * DV + d * 16 + g] = o[d][0];
+        wo[((size_t)warp * rows_valid + 2 * t) * DV + d * 16 + g + 8] = o[d][2];
       }
       if (2 * t + 1 < rows_valid) {
-        wo[((size_t)warp * rows_valid + 2 * t + 1) * DH + d * 16 + g] = o[d][1];
-        wo[((size_t)warp * rows_valid + 2 * t + 1) * DH + d * 16 + g + 8] = o[d][3];
+        wo[((size_t)warp * rows_valid + 2 * t + 1) * DV + d * 16 + g] = o[d][1];
+        wo[((size_t)warp * rows_valid + 2 * t + 1) * DV + d * 16 + g + 8] = o[d][3];
       }
     }
     asm volatile("bar.sync 1, %0;\n" ::"n"(D8_WARPS * 32) : "memory");
-    for (int i = threadIdx.x; i < rows_valid * DH; i += D8_WARPS * 32) {
-      const int r = i / DH, d = i - r * DH;
+    for (int i = threadIdx.x; i < rows_valid * DV; i += D8_WARPS * 32) {
+      const int r = i / DV, d = i - r * DV;
       float mx = -INFINITY;
 #pragma unroll
       for (int x = 0; x < D8_WARPS; ++x) mx = fmaxf(mx, wm[x * 8 + r]);
@@ -1230,11 +1288,11 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
 #pragma unroll
         for (int x = 0; x < D8_WARPS; ++x) {
           const float scale = fast_exp2(wm[x * 8 + r] - mx);
-          num += scale * wo[((size_t)x * rows_valid + r) * DH + d];
+          num += scale * wo[((size_t)x * rows_valid + r) * DV + d];
           den += scale * wl[x * 8 + r];
         }
       }
-      p.part_o[(pidx * p.rows_max + r) * DH + d] = den > 0.f ? num / den : 0.f;
+      p.part_o[(pidx * p.rows_max + r) * DV + d] = den > 0.f ? num / den : 0.f;
       if (d == 0) {
         p.part_ml[(pidx * p.rows_max + r) * 2] = mx;
         p.part_ml[(pidx * p.rows_max + r) * 2 + 1] = den;
@@ -1250,15 +1308,15 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
 // Merges the chunks of every (token, query head): one block each.  Its warps take the
 // chunks in turn (warp w: chunks w, w + 8, ...), then add up in a fixed order.
 constexpr int COMBINE_WARPS = 8;
-constexpr int DPL = (DH + 31) / 32;  // output elements per lane
+constexpr int DPL = (DV + 31) / 32;  // output elements per lane
 
 __global__ void __launch_bounds__(COMBINE_WARPS * 32)
 attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                     const int* __restrict__ token_seq, const int* __restrict__ cu_q,
                     const int* __restrict__ split_start, const int* __restrict__ split_count,
-                    bf16* __restrict__ out, int num_q_heads, int num_kv_heads, int rows_max,
+                    bf16* __restrict__ out, const float* __restrict__ sink, int num_q_heads, int num_kv_heads, int rows_max,
                     int* __restrict__ work_counter) {
-  __shared__ float s_acc[COMBINE_WARPS][DH];
+  __shared__ float s_acc[COMBINE_WARPS][DV];
   __shared__ float s_den[COMBINE_WARPS];
   __shared__ float s_max[COMBINE_WARPS];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -1289,7 +1347,7 @@ attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ 
 #pragma unroll
     for (int i = 0; i < DPL; ++i) {
       const int d = lane + 32 * i;
-      o[i] = d < DH ? part_o[pidx * DH + d] : 0.f;
+      o[i] = d < DV ? part_o[pidx * DV + d] : 0.f;
     }
     if (ls > 0.f) {  // an empty chunk stored zeros
       const float m_new = fmaxf(m_run, ms);
@@ -1304,7 +1362,7 @@ attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ 
 #pragma unroll
   for (int i = 0; i < DPL; ++i) {
     const int d = lane + 32 * i;
-    if (d < DH) s_acc[warp][d] = acc[i];
+    if (d < DV) s_acc[warp][d] = acc[i];
   }
   if (lane == 0) {
     s_den[warp] = den;
@@ -1321,9 +1379,10 @@ attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ 
     scale[w] = s_max[w] == -INFINITY ? 0.f : fast_exp2(s_max[w] - mx);
     den += s_den[w] * scale[w];
   }
+  if (sink != nullptr) den += fast_exp2(sink[h] * LOG2E - mx);
   const float inv = den > 0.f ? 1.0f / den : 0.f;
-  bf16* op = out + ((size_t)tkn * num_q_heads + h) * DH;
-  for (int d = threadIdx.x; d < DH; d += COMBINE_WARPS * 32) {
+  bf16* op = out + ((size_t)tkn * num_q_heads + h) * DV;
+  for (int d = threadIdx.x; d < DV; d += COMBINE_WARPS * 32) {
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < COMBINE_WARPS; ++w) v = fmaf(s_acc[w][d], scale[w], v);
@@ -1331,14 +1390,15 @@ attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ 
   }
 }
 
-constexpr size_t prefill_smem(int rows) { return (size_t)(rows + 4 * BN) * PITCH * sizeof(bf16); }
-constexpr size_t DECODE_SMEM_KV = (size_t)(16 + 2 * DEC_STAGES * DEC_BN) * PITCH * sizeof(bf16);
+constexpr size_t prefill_smem(int rows) { return ((size_t)(rows + 2 * BN) * PITCH + (size_t)2 * BN * VPITCH) * sizeof(bf16); }
+constexpr size_t DECODE_SMEM_KV =
+    ((size_t)(16 + DEC_STAGES * DEC_BN) * PITCH + (size_t)DEC_STAGES * DEC_BN * VPITCH) * sizeof(bf16);
 constexpr size_t DECODE_SMEM_MERGE =
-    16 * PITCH * sizeof(bf16) + (size_t)(2 * DEC_WARPS * 16 + DEC_WARPS * 16 * DH) * sizeof(float);
+    16 * PITCH * sizeof(bf16) + (size_t)(2 * DEC_WARPS * 16 + DEC_WARPS * 16 * DV) * sizeof(float);
 constexpr size_t DECODE_SMEM = DECODE_SMEM_KV > DECODE_SMEM_MERGE ? DECODE_SMEM_KV : DECODE_SMEM_MERGE;
-constexpr size_t DECODE8_SMEM_KV = (size_t)(2 * D8_STAGES * D8_BN) * PITCH * sizeof(bf16);
-constexpr size_t DECODE8_SMEM_TMA_KV = (size_t)(2 * D8_STAGES * D8_BN) * DH * sizeof(bf16);
-constexpr size_t DECODE8_SMEM_MERGE = (size_t)(2 * D8_WARPS * 8 + D8_WARPS * 8 * DH) * sizeof(float);
+constexpr size_t DECODE8_SMEM_KV = (size_t)D8_STAGES * D8_BN * (PITCH + VPITCH) * sizeof(bf16);
+constexpr size_t DECODE8_SMEM_TMA_KV = (size_t)D8_STAGES * D8_BN * (DH + DV) * sizeof(bf16);
+constexpr size_t DECODE8_SMEM_MERGE = (size_t)(2 * D8_WARPS * 8 + D8_WARPS * 8 * DV) * sizeof(float);
 constexpr size_t DECODE8_SMEM = DECODE8_SMEM_KV > DECODE8_SMEM_MERGE ? DECODE8_SMEM_KV : DECODE8_SMEM_MERGE;
 
 }  // namespace
@@ -1360,7 +1420,11 @@ static int blocks_resident(Kernel kernel, int threads, size_t smem, int* out) {
 
 #define SB_CONCAT2(a, b) a##b
 #define SB_CONCAT(a, b) SB_CONCAT2(a, b)
+#if SB_VALUE_DIM == SB_HEAD_DIM
 #define SB_FN(name) SB_CONCAT(SB_CONCAT(name, _hd), SB_HEAD_DIM)
+#else
+#define SB_FN(name) SB_CONCAT(SB_CONCAT(SB_CONCAT(name, _hd), SB_HEAD_DIM), SB_CONCAT(v, SB_VALUE_DIM))
+#endif
 
 // Ragged prefill attention.  items: [num_items, 2] (sequence, first token of a tile of
 // rows_per_tile / G tokens); rows_per_tile is 64 or 128.  Tiles of 64 rows run with two key
@@ -1369,23 +1433,23 @@ static int blocks_resident(Kernel kernel, int threads, size_t smem, int* out) {
 static int prefill_launch(const void* q, const void* cache, const int* block_table, int max_pages,
                           const int* cu_q, const int* q_start, void* out, int num_q_heads,
                           int num_kv_heads, int page_size, int num_pages, float cap, int window,
-                          const float* distance,
-                          const int* items, int num_items, int rows_per_tile, int single_key_group,
+                          const float* distance, int linear, const float* sink, int key_chunk, const int* items, int num_items, int rows_per_tile, int single_key_group,
                           const void* pool, const int* pool_table, int pool_max_pages, int pool_len,
                           int pool_pages, int* err, cudaStream_t stream) {
   if (num_items == 0) return 0;
   if (num_kv_heads <= 0 || num_q_heads % num_kv_heads || num_q_heads / num_kv_heads > rows_per_tile) return -8;
-  if (pool != nullptr && (pool_len <= 0 || window <= 0)) return -8;
+  if (pool != nullptr && (pool_len <= 0 || window <= 0 || !ONE_SIZE || sink != nullptr)) return -8;
+  if (key_chunk > 0 && window > 0) return -8;
   AttnParams p{};
-  p.distance = distance;
+  p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk;
   p.q = (const bf16*)q; p.cache = (const bf16*)cache; p.block_table = block_table; p.max_pages = max_pages;
   p.cu_q = cu_q; p.q_start = q_start; p.out = (bf16*)out; p.num_q_heads = num_q_heads;
   p.num_kv_heads = num_kv_heads; p.page_size = page_size; p.num_pages = num_pages; p.cap = cap;
   p.window = window; p.items = items; p.err = err;
   p.pool = (const bf16*)pool; p.pool_table = pool_table; p.pool_max_pages = pool_max_pages; p.pool_len = pool_len;
   p.pool_entries = pool_len > 0 ? (page_size + pool_len - 1) / pool_len : 0; p.pool_pages = pool_pages;
-  // The merge of two key groups needs [BM][DH] floats where the tiles were.
-  constexpr bool split_fits = (size_t)(2 * 64 + 64 * DH) * sizeof(float) <= (size_t)4 * BN * PITCH * sizeof(bf16);
+  // The merge of two key groups needs [BM][DV] floats where the tiles were.
+  constexpr bool split_fits = (size_t)(2 * 64 + 64 * DV) * sizeof(float) <= (size_t)2 * BN * (PITCH + VPITCH) * sizeof(bf16);
   if (rows_per_tile == 128) {
     static bool configured = false;
     if (!configured) {
@@ -1426,7 +1490,7 @@ extern "C" int SB_FN(sb_attn_prefill)(const void* q, const void* cache, const in
                                       const int* items, int num_items, int rows_per_tile, int single_key_group,
                                       int* err, cudaStream_t stream) {
   return prefill_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_q_heads, num_kv_heads, page_size,
-                        num_pages, cap, window, nullptr, items, num_items, rows_per_tile, single_key_group, nullptr,
+                        num_pages, cap, window, nullptr, 0, nullptr, 0, items, num_items, rows_per_tile, single_key_group, nullptr,
                         nullptr, 0, 0, 0, err, stream);
 }
 
@@ -1437,24 +1501,25 @@ extern "C" int SB_FN(sb_attn_prefill_pooled)(const void* q, const void* cache, c
                                              const void* pool, const int* pool_table, int pool_max_pages, int pool_len,
                                              int pool_pages, int* err, cudaStream_t stream) {
   return prefill_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_q_heads, num_kv_heads, page_size,
-                        num_pages, cap, window, nullptr, items, num_items, rows_per_tile, single_key_group, pool,
+                        num_pages, cap, window, nullptr, 0, nullptr, 0, items, num_items, rows_per_tile, single_key_group, pool,
                         pool_table, pool_max_pages, pool_len, pool_pages, err, stream);
 }
 
-// The same with a distance bias: `distance` float32 [2, Hq] (see AttnParams).
+// The same with a distance bias, chunks of keys and a sink (each optional, see AttnParams).
 extern "C" int SB_FN(sb_attn_prefill_biased)(const void* q, const void* cache, const int* block_table, int max_pages,
                                              const int* cu_q, const int* q_start, void* out, int num_q_heads,
                                              int num_kv_heads, int page_size, int num_pages, float cap, int window,
                                              const int* items, int num_items, int rows_per_tile, int single_key_group,
-                                             const float* distance, int* err, cudaStream_t stream) {
+                                             const float* distance, int linear, const float* sink, int key_chunk,
+                                             int* err, cudaStream_t stream) {
   return prefill_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_q_heads, num_kv_heads, page_size,
-                        num_pages, cap, window, distance, items, num_items, rows_per_tile, single_key_group, nullptr,
+                        num_pages, cap, window, distance, linear, sink, key_chunk, items, num_items, rows_per_tile, single_key_group, nullptr,
                         nullptr, 0, 0, 0, err, stream);
 }
 
 // Split-key attention for sequences with at most 16 query rows per kv head, and the merge.
 // items: [num_items, 2] (sequence or -1, chunk index); chunk: keys per chunk, a multiple of 64;
-// part_o / part_ml: scratch of num_items * Hkv * rows_max * (DH | 2) floats;
+// part_o / part_ml: scratch of num_items * Hkv * rows_max * (DV | 2) floats;
 // work_counter: one int that is zero before the first launch; the merge kernel zeroes it again;
 // split_start / split_count: per sequence, its range of items (count 0: not handled here).
 // older_keys_settled: the caller vouches that every key and value below q_start was written
@@ -1467,22 +1532,23 @@ extern "C" int SB_FN(sb_attn_decode)(const void* q, const void* cache, const int
                                      int chunk, float* part_o, float* part_ml, int* work_counter,
                                      int rows_max, const int* split_start, const int* split_count, int variant,
                                      const void* tensor_map, int older_keys_settled, const float* distance,
-                                     int* err, cudaStream_t stream) {
+                                     int linear, const float* sink, int key_chunk, int* err, cudaStream_t stream) {
   // variant: 0 picks the kernel by rows_max (<= 8: the turned-round kernel, fed by TMA through a
   // producer warp when a tensor map is given and the shapes allow); 1 forbids TMA; 2 uses TMA
   // without the producer warp; 16 forces the 16-row kernel.
   if (num_items == 0) return 0;
   if (num_kv_heads <= 0 || num_q_heads % num_kv_heads || rows_max > 16 || chunk % 64) return -8;
+  if (key_chunk > 0 && window > 0) return -8;
   AttnParams p{};
   p.q = (const bf16*)q; p.cache = (const bf16*)cache; p.block_table = block_table; p.max_pages = max_pages;
   p.cu_q = cu_q; p.q_start = q_start; p.out = (bf16*)out; p.num_q_heads = num_q_heads;
   p.num_kv_heads = num_kv_heads; p.page_size = page_size; p.num_pages = num_pages; p.cap = cap;
   p.window = window; p.items = items; p.chunk = chunk; p.part_o = part_o; p.part_ml = part_ml;
   p.rows_max = rows_max; p.older_keys_settled = older_keys_settled; p.err = err;
-  p.distance = distance;
+  p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk;
   const int total_work = num_items * num_kv_heads;
   const bool power_of_two_pages = (page_size & (page_size - 1)) == 0;
-  constexpr size_t ws_merge = (size_t)(D8_WARPS * 8 * DH) * sizeof(float);
+  constexpr size_t ws_merge = (size_t)(D8_WARPS * 8 * DV) * sizeof(float);
   constexpr bool ws_fits = ws_merge <= (size_t)D8_BN * DH * sizeof(bf16);  // the merge borrows one key tile
   if (rows_max <= 8 && (variant == 0 || variant == 3) && TMA_OK && ws_fits && tensor_map != nullptr && power_of_two_pages) {
     static int resident_ws = 0;
@@ -1529,7 +1595,7 @@ extern "C" int SB_FN(sb_attn_decode)(const void* q, const void* cache, const int
   }
   SB_LAUNCH_CHECK();
   sb_launch_early(attn_combine_kernel, (unsigned)(num_tokens * num_q_heads), COMBINE_WARPS * 32, 0, stream,
-      part_o, part_ml, token_seq, cu_q, split_start, split_count, (bf16*)out, num_q_heads, num_kv_heads,
+      part_o, part_ml, token_seq, cu_q, split_start, split_count, (bf16*)out, sink, num_q_heads, num_kv_heads,
       rows_max, work_counter);
   SB_LAUNCH_CHECK();
   return 0;
@@ -1540,7 +1606,7 @@ extern "C" int SB_FN(sb_attn_decode)(const void* q, const void* cache, const int
 // this many blocks evenly.  Returns the count, or a negative status.
 extern "C" int SB_FN(sb_attn_decode_resident)(int with_tensor_map) {
   int resident = 0, rc;
-  constexpr size_t ws_merge = (size_t)(D8_WARPS * 8 * DH) * sizeof(float);
+  constexpr size_t ws_merge = (size_t)(D8_WARPS * 8 * DV) * sizeof(float);
   constexpr bool ws_fits = ws_merge <= (size_t)D8_BN * DH * sizeof(bf16);
   if (with_tensor_map && TMA_OK && ws_fits) {
     constexpr size_t smem = (size_t)(2 * WS_STAGES * D8_BN) * DH * sizeof(bf16) + 1024;

@@ -78,8 +78,11 @@ struct TcParams {
   float cap;
   int window;
   // optional, float32 [2, Hq]: r1 and r2 per query head; the score of query i and key j loses
-  // r1 log(1 + r2 (i - j)) (not together with a cap)
+  // r1 log(1 + r2 (i - j)).  With `linear`, float32 [Hq]: it loses r1 (i - j).  (Not together with a cap.)
   const float* distance;
+  int linear;
+  int key_chunk;      // > 0 (without a window): position i sees the keys from (i / C) * C on
+  const float* sink;  // optional, float32 [Hq]: exp(sink) joins the denominator (not together with a cap)
   // 1: the block first writes the term for every (distance, head of its kv head) into shared memory
   // behind the tiles, [window][group] floats, and the softmax threads read it there
   int bias_table;
@@ -101,6 +104,12 @@ __device__ __forceinline__ float fast_tanh(float x) {
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+// The lowest key that the query at `pos` sees.
+__device__ __forceinline__ int lowest_key(const TcParams& p, int pos) {
+  if (p.window > 0) return max(pos - p.window + 1, 0);
+  return p.key_chunk > 0 ? max(pos, 0) / p.key_chunk * p.key_chunk : 0;
 }
 
 __global__ void __launch_bounds__(TC_THREADS)
@@ -127,8 +136,8 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
   const int ntok = min(tokens_per_tile, q_len - i0);
   const int rows_valid = ntok * group;
   const int p0 = qs + i0, p1 = qs + i0 + ntok - 1;
-  const int kv_lo = p.window > 0 ? max(qs - p.window + 1, 0) : 0;  // lowest key the request still holds
-  const int lo = p.window > 0 ? max(p0 - p.window + 1, 0) : 0;     // lowest key this tile can see
+  const int kv_lo = lowest_key(p, qs);  // lowest key the request still holds
+  const int lo = lowest_key(p, p0);     // lowest key this tile can see
   const int kv_hi = p1 + 1;
   const int tile0 = (lo / BN) * BN;
   const int n_tiles = (kv_hi - tile0 + BN - 1) / BN;
@@ -311,6 +320,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
     // Positions of this warp's first and last row, for deciding whether a tile needs masking.
     const bool rows_full = quarter * 32 + 31 < rows_valid;
     const int warp_pos_lo = p0 + (quarter * 32) / group, warp_pos_hi = p0 + (quarter * 32 + 31) / group;
+    const int row_lo = lowest_key(p, pos), warp_lo = lowest_key(p, warp_pos_hi);  // the lowest keys seen
     const float inv_cap = p.cap > 0.f ? 1.0f / p.cap : 0.f;
     const float scale2 = p.cap > 0.f ? p.cap * LOG2E : LOG2E;  // from x (tanh's value, or the score) to log2 units
     // The distance bias of this thread's row: r1 ln 2 and r2 of its head.
@@ -318,8 +328,9 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
     const bool tabled = p.bias_table != 0;
     const int head_in_group = r < rows_valid ? r % group : 0;
     const int head = m * group + head_in_group;
-    const float bias_r1 = biased ? p.distance[head] * 0.6931471805599453f : 0.f;
-    const float bias_r2 = biased ? p.distance[p.num_q_heads + head] : 0.f;
+    const bool linear = biased && p.linear != 0;
+    const float bias_r1 = biased ? p.distance[head] * (linear ? 1.0f : 0.6931471805599453f) : 0.f;
+    const float bias_r2 = biased && !linear ? p.distance[p.num_q_heads + head] : 0.f;
     float m_own = -INFINITY, l = 0.f;  // the maximum this thread's sum is relative to; the sum
     bool ok = true;
     if (QT_DIMS > 0) {
@@ -351,7 +362,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
       uint32_t sr[CW];
       tmem_load_32x32(tmem + lane_base + S_COL0 + sb * BN + part * CW, sr);
       tmem_wait_load();
-      const bool need_mask = !rows_full || j0 + BN - 1 > warp_pos_lo || (p.window > 0 && warp_pos_hi - j0 >= p.window);
+      const bool need_mask = !rows_full || j0 + BN - 1 > warp_pos_lo || j0 < warp_lo;
       float mx = -INFINITY;
       if (need_mask) {
 #pragma unroll
@@ -359,12 +370,14 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
           float v = __uint_as_float(sr[c]);
           if (p.cap > 0.f) v = fast_tanh(v * inv_cap);
           const int key = j0 + part * CW + c;
-          if (biased) {
+          if (linear) {
+            v -= bias_r1 * (float)max(pos - key, 0);
+          } else if (biased) {
             const int d = max(pos - key, 0);
             v -= tabled ? bias_tab[min(d, p.window - 1) * group + head_in_group]
                         : bias_r1 * __log2f(fmaf(bias_r2, (float)d, 1.0f));
           }
-          v = (key <= pos && (p.window <= 0 || pos - key < p.window)) ? v : -INFINITY;
+          v = (key <= pos && key >= row_lo) ? v : -INFINITY;
           sr[c] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -373,7 +386,9 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
         for (int c = 0; c < CW; ++c) {
           float v = __uint_as_float(sr[c]);
           if (p.cap > 0.f) v = fast_tanh(v * inv_cap);
-          if (biased) {
+          if (linear) {
+            v -= bias_r1 * (float)(pos - (j0 + part * CW + c));
+          } else if (biased) {
             const int d = pos - (j0 + part * CW + c);  // every key is visible: 0 <= d < window
             v -= tabled ? bias_tab[d * group + head_in_group] : bias_r1 * __log2f(fmaf(bias_r2, (float)d, 1.0f));
           }
@@ -487,6 +502,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
       l = 0.f;
 #pragma unroll
       for (int q = 0; q < GROUPS * SPLIT; ++q) l += row_sum[q][r];
+      if (p.sink != nullptr && r < rows_valid) l += fast_exp2(p.sink[head] * LOG2E - m_final);  // it has no value
     }
     if (ok && !mbar_wait_bounded(&o_done, 0)) ok = false;
     tc_fence_after_sync();
@@ -564,10 +580,11 @@ static_assert(V_STAGES == 2, "the zeroing of value rows looks two tiles back");
 static int prefill_tc_launch(const void* q, const void* cache, const int* block_table, int max_pages,
                              const int* cu_q, const int* q_start, void* out, int num_tokens,
                              int num_q_heads, int num_kv_heads, int page_size, int num_pages, float cap,
-                             int window, const float* distance, const int* items, int num_items, int* err,
-                             cudaStream_t stream) {
+                             int window, const float* distance, int linear, const float* sink, int key_chunk,
+                             const int* items, int num_items, int* err, cudaStream_t stream) {
   if (num_items == 0) return 0;
-  if (distance != nullptr && cap > 0.f) return -13;
+  if ((distance != nullptr || sink != nullptr) && cap > 0.f) return -13;
+  if (key_chunk > 0 && window > 0) return -13;
   if (num_kv_heads <= 0 || num_q_heads % num_kv_heads) return -8;
   const int group = num_q_heads / num_kv_heads;
   if (group > BM || BM % group || (page_size & (page_size - 1))) return -11;
@@ -591,14 +608,14 @@ static int prefill_tc_launch(const void* q, const void* cache, const int* block_
   p.block_table = block_table; p.max_pages = max_pages; p.cu_q = cu_q; p.q_start = q_start; p.out = (bf16*)out;
   p.num_q_heads = num_q_heads; p.num_kv_heads = num_kv_heads; p.page_size = page_size; p.num_pages = num_pages;
   p.cap = cap; p.window = window; p.items = items; p.box_rows = box_rows; p.err = err;
-  p.distance = distance;
+  p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk;
   size_t table_bytes = 0;
   static int table_allowed = -1;  // SIMPLY_B200_BIAS_TABLE=0: every softmax thread computes its terms (experiments)
   if (table_allowed < 0) {
     const char* e = getenv("SIMPLY_B200_BIAS_TABLE");
     table_allowed = (e && e[0] == '0') ? 0 : 1;
   }
-  if (table_allowed && distance != nullptr && window > 0 && (size_t)window * group * sizeof(float) <= TC_TABLE_MAX)
+  if (table_allowed && distance != nullptr && !linear && window > 0 && (size_t)window * group * sizeof(float) <= TC_TABLE_MAX)
     table_bytes = (size_t)window * group * sizeof(float);
   p.bias_table = table_bytes > 0 ? 1 : 0;
   static bool configured = false;
@@ -618,18 +635,18 @@ extern "C" int SB_FN(sb_attn_prefill_tc)(const void* q, const void* cache, const
                                          int num_q_heads, int num_kv_heads, int page_size, int num_pages, float cap,
                                          int window, const int* items, int num_items, int* err, cudaStream_t stream) {
   return prefill_tc_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_tokens, num_q_heads, num_kv_heads,
-                           page_size, num_pages, cap, window, nullptr, items, num_items, err, stream);
+                           page_size, num_pages, cap, window, nullptr, 0, nullptr, 0, items, num_items, err, stream);
 }
 
-// The same with a distance bias: `distance` float32 [2, Hq] (see TcParams); no cap beside it.
+// The same with a distance bias, chunks of keys and a sink (each optional, see TcParams); no cap beside them.
 extern "C" int SB_FN(sb_attn_prefill_tc_biased)(const void* q, const void* cache, const int* block_table,
                                                 int max_pages, const int* cu_q, const int* q_start, void* out,
                                                 int num_tokens, int num_q_heads, int num_kv_heads, int page_size,
                                                 int num_pages, float cap, int window, const int* items,
-                                                int num_items, const float* distance, int* err,
-                                                cudaStream_t stream) {
+                                                int num_items, const float* distance, int linear, const float* sink,
+                                                int key_chunk, int* err, cudaStream_t stream) {
   return prefill_tc_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_tokens, num_q_heads, num_kv_heads,
-                           page_size, num_pages, cap, window, distance, items, num_items, err, stream);
+                           page_size, num_pages, cap, window, distance, linear, sink, key_chunk, items, num_items, err, stream);
 }
 
 #endif  // head sizes that are no multiple of 64 do not get this kernel

@@ -37,6 +37,8 @@ class KernelBuildError(RuntimeError):
 
 # Sources that are compiled once per head size (-DSB_HEAD_DIM=N) into libraries of their own.
 PER_HEAD_DIM = ("attention_mma.cu", "attention_tc.cu", "attention_tc_pair.cu")
+# ... and those of them that also take value heads of another size (-DSB_VALUE_DIM=M).
+PER_TWO_SIZES = ("attention_mma.cu",)
 
 
 # Compiled once per shape of a cache of latents (-DSB_LATENT_KD=N -DSB_LATENT_VD=M).
@@ -94,16 +96,26 @@ def build(verbose: bool = True, force: bool = False) -> str:
   return _build(sources(), LIB_NAME, [], verbose, force)
 
 
-def attention_lib_name(head_dim: int) -> str:
-  return f"libsimply_b200_attn_hd{head_dim}.so"
+def attention_suffix(head_dim: int, value_dim: int | None = None) -> str:
+  """How a library's entry points and its file name say which sizes it is for."""
+  return f"hd{head_dim}" if value_dim in (None, head_dim) else f"hd{head_dim}v{value_dim}"
 
 
-def build_attention(head_dim: int, verbose: bool = True, force: bool = False) -> str:
-  """Compiles the tensor-core attention kernels for one head size; returns the library's path."""
-  if head_dim % 16 or not 16 <= head_dim <= 256:
-    raise KernelBuildError(f"tensor-core attention takes head sizes 16, 32, ..., 256; got {head_dim}")
-  srcs = [os.path.join(CSRC, f) for f in PER_HEAD_DIM]
-  return _build(srcs, attention_lib_name(head_dim), [f"-DSB_HEAD_DIM={head_dim}"], verbose, force)
+def attention_lib_name(head_dim: int, value_dim: int | None = None) -> str:
+  return f"libsimply_b200_attn_{attention_suffix(head_dim, value_dim)}.so"
+
+
+def build_attention(head_dim: int, verbose: bool = True, force: bool = False, value_dim: int | None = None) -> str:
+  """Compiles the tensor-core attention kernels for one head size (or for key and value heads of two
+  sizes: then the mma.sync kernels alone); returns the library's path."""
+  for size in (head_dim, head_dim if value_dim is None else value_dim):
+    if size % 16 or not 16 <= size <= 256:
+      raise KernelBuildError(f"tensor-core attention takes head sizes 16, 32, ..., 256; got {size}")
+  if value_dim is None or value_dim == head_dim:
+    srcs, defines = PER_HEAD_DIM, [f"-DSB_HEAD_DIM={head_dim}"]
+  else:
+    srcs, defines = PER_TWO_SIZES, [f"-DSB_HEAD_DIM={head_dim}", f"-DSB_VALUE_DIM={value_dim}"]
+  return _build([os.path.join(CSRC, f) for f in srcs], attention_lib_name(head_dim, value_dim), defines, verbose, force)
 
 
 def latent_shape_ok(row_dim: int, value_dim: int) -> bool:
@@ -189,16 +201,16 @@ def load() -> ctypes.CDLL:
     return _lib
 
 
-_attention_libs: dict[int, ctypes.CDLL] = {}
+_attention_libs: dict[str, ctypes.CDLL] = {}
 
 
-def load_attention(head_dim: int) -> ctypes.CDLL:
-  """Builds if needed and loads the attention library of one head size."""
+def load_attention(head_dim: int, value_dim: int | None = None) -> ctypes.CDLL:
+  """Builds if needed and loads the attention library of one head size (or pair of sizes)."""
   with _lock:
-    lib = _attention_libs.get(head_dim)
+    key = attention_suffix(head_dim, value_dim)
+    lib = _attention_libs.get(key)
     if lib is None:
-      lib = ctypes.CDLL(build_attention(head_dim))
-      _attention_libs[head_dim] = lib
+      lib = _attention_libs[key] = ctypes.CDLL(build_attention(head_dim, value_dim=value_dim))
     return lib
 
 

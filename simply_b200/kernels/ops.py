@@ -89,12 +89,14 @@ class AttentionGraphPlan:
   split_count [batch]."""
 
   def __init__(self, ops: "CudaOps", window: int | None, group: int, num_kv_heads: int, head_dim: int,
-               batch: int, bucket: int, max_burst: int, page_size: int):
-    self.key = ops._plan_key(window, group, num_kv_heads, head_dim, page_size)
-    self.window, self.group, self.batch = window, group, batch
+               batch: int, bucket: int, max_burst: int, page_size: int, key_chunk: int | None = None,
+               value_dim: int | None = None):
+    self.key = ops._plan_key(window, group, num_kv_heads, head_dim, page_size, key_chunk, value_dim)
+    self.window, self.key_chunk, self.group, self.batch = window, key_chunk, group, batch
     # Most keys a sequence of this bucket sees in such a layer during a burst.
-    span = min(bucket, window + max_burst + 64) if window else bucket
-    self.chunk = ops.decode_chunk_for([bucket - span] * batch, [bucket] * batch, num_kv_heads, head_dim)
+    reach = window or key_chunk
+    span = min(bucket, reach + max_burst + 64) if reach else bucket
+    self.chunk = ops.decode_chunk_for([bucket - span] * batch, [bucket] * batch, num_kv_heads, head_dim, value_dim)
     self.per_seq = -(-span // self.chunk) + 1
     self.words = batch * self.per_seq * 2 + 2 * batch
 
@@ -105,14 +107,14 @@ class AttentionGraphPlan:
                 split_start=view[n:n + self.batch], split_count=view[n + self.batch:])
 
   def fill(self, host_words: np.ndarray, lengths: np.ndarray, steps: int) -> None:
-    items, start, count = CudaOps.static_decode_plan(lengths, steps, self.window, self.chunk, self.per_seq)
+    items, start, count = CudaOps.static_decode_plan(lengths, steps, self.window, self.chunk, self.per_seq, self.key_chunk)
     n = items.size
     host_words[:n] = items.reshape(-1)
     host_words[n:n + self.batch] = start
     host_words[n + self.batch:] = count
 
   def ranges(self, lengths: np.ndarray, steps: int):
-    return CudaOps.decode_chunk_range(lengths, steps, self.window, self.chunk)
+    return CudaOps.decode_chunk_range(lengths, steps, self.window, self.chunk, self.key_chunk)
 
 
 class PooledAttentionGraphPlan:
@@ -153,7 +155,7 @@ class CudaOps:
       raise KernelError(f"kernels are built for sm_100a; this device is sm_{major}{minor}")
     self._declare()
     self.err = torch.zeros(1, dtype=torch.int32, device=self.device)
-    self._attn_fns: dict[int, tuple] = {}
+    self._attn_fns: dict[tuple[int, int], tuple] = {}
     self._latent_fns: dict[tuple[int, int], Any] = {}
     self._tensor_maps: dict[tuple, tuple] = {}
     # Work counter of the split-key attention kernel: zero between launches (its merge kernel resets it).
@@ -163,7 +165,7 @@ class CudaOps:
     # Split-key attention: the chunk length is chosen so that the work items fill the kernel's
     # persistent grid evenly; decode_chunk > 0 fixes it instead (a multiple of 64).
     self.decode_chunk = 0
-    self._decode_slots: dict[int, int] = {}
+    self._decode_slots: dict[tuple[int, int], int] = {}
     # 0: the kernel is picked by the number of query rows; 1 forbids TMA; 16 forces the 16-row kernel (tests).
     self.decode_variant = 0
     self.direct_library_products = True  # False: through torch.mm
@@ -407,7 +409,9 @@ class CudaOps:
   # ---- checks ---------------------------------------------------------------
   def check_attention(self, head_dim: int, num_heads: int, num_kv_heads: int, value_dim: int | None = None) -> None:
     """Refuses shapes no kernel takes; compiles the tensor-core kernels of this head size."""
-    if value_dim is not None and value_dim != head_dim:
+    if value_dim is not None and value_dim != head_dim:  # (what the tensor-core kernels refuse, the general one takes)
+      if self._uses_tensor_core_attention(head_dim, num_heads // num_kv_heads, value_dim):
+        self._attention_lib(head_dim, value_dim)
       return
     if head_dim <= 0 or head_dim % 2 or head_dim > 512:
       raise KernelError(f"attention kernels take even head sizes up to 512, got {head_dim}")
@@ -416,55 +420,58 @@ class CudaOps:
     if self._uses_tensor_core_attention(head_dim, num_heads // num_kv_heads):
       self._attention_lib(head_dim)
 
-  def _uses_tensor_core_attention(self, head_dim: int, group: int) -> bool:
-    return (self.dtype == torch.bfloat16 and self.tensor_core_attention and head_dim % 16 == 0
-            and head_dim <= 256 and group <= 64)  # a group must fit a 64-row tile
+  def _uses_tensor_core_attention(self, head_dim: int, group: int, value_dim: int | None = None) -> bool:
+    value_dim = head_dim if value_dim is None else value_dim
+    return (self.dtype == torch.bfloat16 and self.tensor_core_attention and head_dim % 16 == 0 and value_dim % 16 == 0
+            and head_dim <= 256 and value_dim <= 256 and group <= 64)  # a group must fit a 64-row tile
 
-  def _attention_lib(self, head_dim: int):
-    fns = self._attn_fns.get(head_dim)
+  def _attention_lib(self, head_dim: int, value_dim: int | None = None):
+    value_dim = head_dim if value_dim is None else value_dim
+    fns = self._attn_fns.get((head_dim, value_dim))
     if fns is None:
-      lib = build.load_attention(head_dim)
+      lib = build.load_attention(head_dim, value_dim)
+      suffix = build.attention_suffix(head_dim, value_dim)
       c_int, c_float, c_void = ctypes.c_int, ctypes.c_float, ctypes.c_void_p
-      prefill = getattr(lib, f"sb_attn_prefill_hd{head_dim}")
+      prefill = getattr(lib, f"sb_attn_prefill_{suffix}")
       prefill.argtypes = [c_void, c_void, c_void, c_int, c_void, c_void, c_void, c_int, c_int, c_int, c_int,
                           c_float, c_int, c_void, c_int, c_int, c_int, c_void, c_void]
       prefill.restype = c_int
-      prefill_pooled = getattr(lib, f"sb_attn_prefill_pooled_hd{head_dim}")
+      prefill_pooled = getattr(lib, f"sb_attn_prefill_pooled_{suffix}")
       prefill_pooled.argtypes = prefill.argtypes[:-2] + [c_void, c_void, c_int, c_int, c_int, c_void, c_void]
       prefill_pooled.restype = c_int
-      decode = getattr(lib, f"sb_attn_decode_hd{head_dim}")
+      decode = getattr(lib, f"sb_attn_decode_{suffix}")
       decode.argtypes = [c_void, c_void, c_void, c_int, c_void, c_void, c_void, c_void, c_int, c_int, c_int,
                          c_int, c_int, c_float, c_int, c_void, c_int, c_int, c_void, c_void, c_void, c_int,
-                         c_void, c_void, c_int, c_void, c_int, c_void, c_void, c_void]
+                         c_void, c_void, c_int, c_void, c_int, c_void, c_int, c_void, c_int, c_void, c_void]
       decode.restype = c_int
-      prefill_biased = getattr(lib, f"sb_attn_prefill_biased_hd{head_dim}")
-      prefill_biased.argtypes = prefill.argtypes[:-2] + [c_void, c_void, c_void]
+      prefill_biased = getattr(lib, f"sb_attn_prefill_biased_{suffix}")
+      prefill_biased.argtypes = prefill.argtypes[:-2] + [c_void, c_int, c_void, c_int, c_void, c_void]
       prefill_biased.restype = c_int
-      make_map = getattr(lib, f"sb_attn_tensor_map_hd{head_dim}")
+      make_map = getattr(lib, f"sb_attn_tensor_map_{suffix}")
       make_map.argtypes = [c_void, c_void, ctypes.c_longlong, c_int]
       make_map.restype = c_int
       prefill_tc = prefill_tc_biased = None
-      if head_dim % 64 == 0:
-        prefill_tc = getattr(lib, f"sb_attn_prefill_tc_hd{head_dim}")
+      if head_dim % 64 == 0 and value_dim == head_dim:
+        prefill_tc = getattr(lib, f"sb_attn_prefill_tc_{suffix}")
         prefill_tc.argtypes = [c_void, c_void, c_void, c_int, c_void, c_void, c_void, c_int, c_int, c_int, c_int,
                                c_int, c_float, c_int, c_void, c_int, c_void, c_void]
         prefill_tc.restype = c_int
-        prefill_tc_biased = getattr(lib, f"sb_attn_prefill_tc_biased_hd{head_dim}")
-        prefill_tc_biased.argtypes = prefill_tc.argtypes[:-2] + [c_void, c_void, c_void]
+        prefill_tc_biased = getattr(lib, f"sb_attn_prefill_tc_biased_{suffix}")
+        prefill_tc_biased.argtypes = prefill_tc.argtypes[:-2] + [c_void, c_int, c_void, c_int, c_void, c_void]
         prefill_tc_biased.restype = c_int
       prefill_pair = None
-      if head_dim in (128, 256):
-        prefill_pair = getattr(lib, f"sb_attn_prefill_pair_hd{head_dim}")
+      if head_dim in (128, 256) and value_dim == head_dim:
+        prefill_pair = getattr(lib, f"sb_attn_prefill_pair_{suffix}")
         prefill_pair.argtypes = [c_void, c_void, c_void, c_int, c_void, c_void, c_void, c_int, c_int, c_int, c_int,
                                  c_int, c_float, c_int, c_void, c_int, c_void, c_void]
         prefill_pair.restype = c_int
-      resident = getattr(lib, f"sb_attn_decode_resident_hd{head_dim}")
+      resident = getattr(lib, f"sb_attn_decode_resident_{suffix}")
       resident.argtypes, resident.restype = [c_int], c_int
       slots = resident(1)
       if slots <= 0:
         raise KernelError(f"sb_attn_decode_resident: {_STATUS.get(slots, slots)}")
-      self._decode_slots[head_dim] = slots
-      fns = self._attn_fns[head_dim] = (prefill, decode, make_map, prefill_tc, prefill_pair, prefill_pooled,
+      self._decode_slots[(head_dim, value_dim)] = slots
+      fns = self._attn_fns[(head_dim, value_dim)] = (prefill, decode, make_map, prefill_tc, prefill_pair, prefill_pooled,
                                         prefill_biased, prefill_tc_biased)
     return fns
 
@@ -480,7 +487,8 @@ class CudaOps:
       self._latent_fns[(row_dim, value_dim)] = fn
     return fn
 
-  def decode_chunk_for(self, kv_lo: Sequence[int], kv_hi: Sequence[int], num_kv_heads: int, head_dim: int) -> int:
+  def decode_chunk_for(self, kv_lo: Sequence[int], kv_hi: Sequence[int], num_kv_heads: int, head_dim: int,
+                       value_dim: int | None = None) -> int:
     """Chunk length of split-key attention for sequences that see the keys [kv_lo, kv_hi).
 
     A work item is one chunk of one (sequence, kv head); the kernel's persistent grid draws items
@@ -491,8 +499,9 @@ class CudaOps:
     """
     if self.decode_chunk:
       return self.decode_chunk
-    self._attention_lib(head_dim)
-    slots = self._decode_slots[head_dim]
+    value_dim = head_dim if value_dim is None else value_dim
+    self._attention_lib(head_dim, value_dim)
+    slots = self._decode_slots[(head_dim, value_dim)]
     lo, hi = np.asarray(kv_lo, dtype=np.int64), np.asarray(kv_hi, dtype=np.int64)
     # (From 128 keys: with 64 a lone sequence's window layers were 13 % slower than with 128,
     # although their items fit the grid either way: twice the items and twice the chunks to merge.)
@@ -509,16 +518,24 @@ class CudaOps:
   DECODE_ITEM_COST = 48
 
   @staticmethod
-  def decode_chunk_range(q_start: np.ndarray, steps: int, window: int | None, chunk: int) -> tuple[np.ndarray, np.ndarray]:
+  def lowest_keys(positions: np.ndarray, window: int | None, key_chunk: int | None) -> np.ndarray:
+    """The lowest key each of these positions sees (a window, chunks of keys, or all)."""
+    if window:
+      return np.maximum(positions - window + 1, 0)
+    return positions // key_chunk * key_chunk if key_chunk else np.zeros_like(positions)
+
+  @staticmethod
+  def decode_chunk_range(q_start: np.ndarray, steps: int, window: int | None, chunk: int,
+                         key_chunk: int | None = None) -> tuple[np.ndarray, np.ndarray]:
     """First and last chunk index per sequence that a decode burst of `steps` steps touches: from
     the lowest key visible at the first step to the highest at the last."""
     qs = np.asarray(q_start, dtype=np.int64)
-    lo = np.maximum(qs - window + 1, 0) // 64 * 64 if window else np.zeros_like(qs)
+    lo = CudaOps.lowest_keys(qs, window, key_chunk) // 64 * 64
     return lo // chunk, (qs + steps - 1) // chunk
 
   @staticmethod
   def static_decode_plan(q_start: np.ndarray, steps: int, window: int | None, chunk: int,
-                         items_per_seq: int) -> tuple[np.ndarray, np.ndarray, np.ndarray]:
+                         items_per_seq: int, key_chunk: int | None = None) -> tuple[np.ndarray, np.ndarray, np.ndarray]:
     """Work list of the split-key kernel for a decode burst replayed from a CUDA graph.
 
     Every sequence gets exactly `items_per_seq` items, so the launch has a fixed size:
@@ -530,7 +547,7 @@ class CudaOps:
     b = len(q_start)
     items = np.full((b, items_per_seq, 2), -1, dtype=np.int32)
     count = np.zeros(b, dtype=np.int32)
-    firsts, lasts = CudaOps.decode_chunk_range(q_start, steps, window, chunk)
+    firsts, lasts = CudaOps.decode_chunk_range(q_start, steps, window, chunk, key_chunk)
     for i, (first, last) in enumerate(zip(firsts.tolist(), lasts.tolist())):
       n = last - first + 1
       if n > items_per_seq:
@@ -576,11 +593,14 @@ class CudaOps:
       return 128
     return self.prefill_rows or 64
 
-  def _plan_key(self, window: int | None, group: int, num_kv_heads: int, head_dim: int, page_size: int) -> tuple:
+  def _plan_key(self, window: int | None, group: int, num_kv_heads: int, head_dim: int, page_size: int,
+                key_chunk: int | None = None, value_dim: int | None = None) -> tuple:
     """Where a step keeps the work lists of one kind of attention layer in `ctx.memo`.  Layers
     share lists only if everything the lists are cut for agrees: the window, the group, the
     number of kv heads and the head size (they set the chunk length) and the rows of a prefill tile."""
-    return ("attention_plan", window, group, num_kv_heads, head_dim, self._prefill_rows(head_dim, group, page_size))
+    key = ("attention_plan", window, group, num_kv_heads, head_dim, self._prefill_rows(head_dim, group, page_size))
+    other_values = value_dim if value_dim != head_dim else None
+    return key if key_chunk is None and other_values is None else key + (key_chunk, other_values)
 
   def attention_graph_plan(self, *, window: int | None, num_heads: int, num_kv_heads: int, head_dim: int,
                            batch: int, bucket: int, max_burst: int, page_size: int, key_chunk: int | None = None,
@@ -588,9 +608,10 @@ class CudaOps:
     """The static work list a decode graph needs for one kind of attention layer, or None when
     the kernel that serves it reads no list (the general kernel)."""
     group = num_heads // num_kv_heads
-    if not self._uses_tensor_core_attention(head_dim, group) or value_dim is not None or key_chunk is not None:
+    if not self._uses_tensor_core_attention(head_dim, group, value_dim):
       return None
-    return AttentionGraphPlan(self, window, group, num_kv_heads, head_dim, batch, bucket, max_burst, page_size)
+    return AttentionGraphPlan(self, window, group, num_kv_heads, head_dim, batch, bucket, max_burst, page_size,
+                              key_chunk, value_dim)
 
   def pooled_attention_graph_plan(self, *, window: int | None, num_heads: int, num_kv_heads: int, head_dim: int,
                                   value_dim: int, pool: int, batch: int, page_size: int):
@@ -602,7 +623,8 @@ class CudaOps:
     return PooledAttentionGraphPlan(self._plan_key(window, group, num_kv_heads, head_dim, page_size) + ("pooled", pool), batch)
 
   def _attention_plan(self, ctx: Any, window: int | None, group: int, force_rows: int = 0,
-                      num_kv_heads: int = 1, head_dim: int = 0, tag: tuple = (), all_tiles: bool = False) -> dict:
+                      num_kv_heads: int = 1, head_dim: int = 0, tag: tuple = (), all_tiles: bool = False,
+                      key_chunk: int | None = None, value_dim: int | None = None) -> dict:
     """Work lists of the two tensor-core kernels for this step, per kind of layer (`_plan_key`).
 
     Sequences with at most 16 query rows per kv head (one or a few new tokens) go to the
@@ -610,7 +632,7 @@ class CudaOps:
     absolute position, one work item per chunk.  The others are cut into tiles of
     64 // group or 128 // group tokens for the prefill kernel, heaviest tile first.
     """
-    key = self._plan_key(window, group, num_kv_heads, head_dim, ctx.page_size) + tag
+    key = self._plan_key(window, group, num_kv_heads, head_dim, ctx.page_size, key_chunk, value_dim) + tag
     plan = ctx.memo.get(key)
     if plan is not None:
       return plan
@@ -625,7 +647,7 @@ class CudaOps:
     for b in np.nonzero(~small)[0]:
       for i0 in range(0, int(q_len[b]), tokens_per_tile):
         last = int(q_start[b]) + min(i0 + tokens_per_tile, int(q_len[b]))
-        first = max(int(q_start[b]) + i0 - window + 1, 0) if window else 0
+        first = int(self.lowest_keys(q_start[b] + i0, window, key_chunk))
         pre.append((last - first, int(b), i0))
     pre.sort(key=lambda x: -x[0])
     if force_rows in (128, 256):
@@ -638,12 +660,11 @@ class CudaOps:
     else:
       prefill_items = np.array([(b, i0) for _, b, i0 in pre], dtype=np.int32).reshape(-1, 2)
     kv_hi = q_start + q_len
-    kv_lo = np.maximum(q_start - window + 1, 0) if window else np.zeros_like(q_start)
-    kv_lo = kv_lo // 64 * 64
+    kv_lo = self.lowest_keys(q_start, window, key_chunk) // 64 * 64
     dec = np.nonzero(small)[0]
     chunk = 64
     if len(dec):
-      chunk = self.decode_chunk_for(kv_lo[dec], kv_hi[dec], num_kv_heads, head_dim)
+      chunk = self.decode_chunk_for(kv_lo[dec], kv_hi[dec], num_kv_heads, head_dim, value_dim)
     split_start = np.zeros(num_seqs, dtype=np.int32)
     split_count = np.zeros(num_seqs, dtype=np.int32)
     dec_items = []
@@ -1025,18 +1046,19 @@ class CudaOps:
     value_dim = head_dim if value_dim is None else value_dim
     out = self._new(t, num_heads * value_dim, dtype=q.dtype)
     group = num_heads // num_kv_heads
-    if (values_in_keys or sink is not None) and (logit_softcap or pooled is not None):
+    if (values_in_keys or sink is not None or key_chunk is not None) and (logit_softcap or pooled is not None):
       raise KernelError("latent rows and sinks go with neither a score cap nor pooled blocks")
     if distance_bias is not None and (pooled is not None or values_in_keys):
       raise KernelError("a distance bias goes with neither pooled blocks nor latent rows")
     if key_chunk is not None and (window or pooled is not None or values_in_keys):
       raise KernelError("chunks of keys go with neither a window, pooled blocks nor latent rows")
     linear_bias = int(distance_bias is not None and distance_bias.shape[0] == 1)
-    # (a distance bias with key size = value size in bfloat16: the mma.sync tile kernels below)
-    biased_on_tensor_cores = (distance_bias is not None and value_dim == head_dim and q.dtype == torch.bfloat16
-                              and self._uses_tensor_core_attention(head_dim, group))
-    if (pooled is not None or value_dim != head_dim or values_in_keys or sink is not None or key_chunk is not None or linear_bias
-        or (distance_bias is not None and not biased_on_tensor_cores)):
+    # What the tensor-core kernels below take beside a window: value heads of another size (the mma.sync
+    # kernels), and the options that their general entry points have.
+    special = distance_bias is not None or sink is not None or key_chunk is not None
+    on_tensor_cores = (q.dtype == torch.bfloat16 and self._uses_tensor_core_attention(head_dim, group, value_dim)
+                       and pooled is None and not values_in_keys)
+    if pooled is not None or values_in_keys or ((special or value_dim != head_dim) and not on_tensor_cores):
       pool, pool_table, pool_len = pooled if pooled is not None else (None, None, 0)
       if pool is not None and pool.dtype != storage.dtype:
         raise KernelError("block entries and the cache must share one dtype")
@@ -1093,15 +1115,18 @@ class CudaOps:
         if rc:
           raise KernelError(f"sb_attn_prefill_pooled: {_STATUS.get(rc, rc)}")
       return out
-    if q.dtype == torch.bfloat16 and self._uses_tensor_core_attention(head_dim, group):
-      prefill, decode, _, prefill_tc, prefill_pair = self._attention_lib(head_dim)[:5]
-      # A distance bias: the tcgen05 kernel by single blocks where it takes the shape (no cap beside
-      # it), else the mma.sync tile kernel; not the kernel by pairs.
+    if on_tensor_cores:
+      fns = self._attention_lib(head_dim, value_dim)
+      prefill, decode, _, prefill_tc, prefill_pair = fns[:5]
+      # A distance bias, a sink or chunks of keys: the tcgen05 kernel by single blocks where it takes the
+      # shape (no cap beside them), else the mma.sync tile kernel; not the kernel by pairs.
+      options = (_ptr(distance_bias), linear_bias, _ptr(sink), int(key_chunk or 0))
+      kind = dict(key_chunk=key_chunk, value_dim=value_dim)
       use_tc = (prefill_tc is not None and self._prefill_uses_tcgen05(head_dim, group, ctx.page_size)
-                and (distance_bias is None or not logit_softcap))
+                and (not special or not logit_softcap))
       use_pair = (prefill_pair is not None and self._prefill_uses_pairs(head_dim, group, ctx.page_size)
-                  and distance_bias is None)
-      plan = self._attention_plan(ctx, window, group, 256 if use_pair else (128 if use_tc else 0), num_kv_heads, head_dim)
+                  and not special)
+      plan = self._attention_plan(ctx, window, group, 256 if use_pair else (128 if use_tc else 0), num_kv_heads, head_dim, **kind)
       common = (_ptr(q), _ptr(storage), _ptr(block_table), block_table.shape[1], _ptr(ctx.cu_q),
                 _ptr(ctx.q_start))
       sizes = (num_heads, num_kv_heads, ctx.page_size, storage.shape[0], float(logit_softcap), int(window or 0))
@@ -1111,12 +1136,12 @@ class CudaOps:
         self.launches += 1
         if rc:
           raise KernelError(f"sb_attn_prefill_pair: {_STATUS.get(rc, rc)}")
-      elif plan["num_prefill"] and use_tc and distance_bias is not None:
+      elif plan["num_prefill"] and use_tc and special:
         tiles = plan
         if plan["rows_per_tile"] != 128 or plan.get("item_width") != 3:  # (a list cut for another kernel)
-          tiles = self._attention_plan(ctx, window, group, 128, num_kv_heads, head_dim, tag=("rows", 128))
-        rc = self._attention_lib(head_dim)[7](*common, _ptr(out), t, *sizes, _ptr(tiles["prefill_items"]),
-                                              tiles["num_prefill"], _ptr(distance_bias), _ptr(self.err), self._stream())
+          tiles = self._attention_plan(ctx, window, group, 128, num_kv_heads, head_dim, tag=("rows", 128), **kind)
+        rc = fns[7](*common, _ptr(out), t, *sizes, _ptr(tiles["prefill_items"]),
+                                              tiles["num_prefill"], *options, _ptr(self.err), self._stream())
         self.launches += 1
         if rc:
           raise KernelError(f"sb_attn_prefill_tc_biased: {_STATUS.get(rc, rc)}")
@@ -1126,13 +1151,13 @@ class CudaOps:
         self.launches += 1
         if rc:
           raise KernelError(f"sb_attn_prefill_tc: {_STATUS.get(rc, rc)}")
-      elif plan["num_prefill"] and distance_bias is not None:
+      elif plan["num_prefill"] and special:
         tiles = plan
         if plan.get("item_width", 2) != 2:  # (a list cut for the tcgen05 kernels, made by a layer without a bias)
-          tiles = self._attention_plan(ctx, window, group, 64, num_kv_heads, head_dim, tag=("rows", 64))
-        rc = self._attention_lib(head_dim)[6](
+          tiles = self._attention_plan(ctx, window, group, 64, num_kv_heads, head_dim, tag=("rows", 64), **kind)
+        rc = fns[6](
             *common, _ptr(out), *sizes, _ptr(tiles["prefill_items"]), tiles["num_prefill"], tiles["rows_per_tile"],
-            int(self.prefill_single_key_group), _ptr(distance_bias), _ptr(self.err), self._stream())
+            int(self.prefill_single_key_group), *options, _ptr(self.err), self._stream())
         self.launches += 1
         if rc:
           raise KernelError(f"sb_attn_prefill_biased: {_STATUS.get(rc, rc)}")
@@ -1144,14 +1169,14 @@ class CudaOps:
           raise KernelError(f"sb_attn_prefill: {_STATUS.get(rc, rc)}")
       if plan["num_decode"]:
         n = plan["num_decode"] * num_kv_heads * plan["rows_max"]
-        part_o = self._new(n * head_dim, dtype=torch.float32)
+        part_o = self._new(n * value_dim, dtype=torch.float32)
         part_ml = self._new(n * 2, dtype=torch.float32)
         rc = decode(*common, _ptr(ctx.token_seq), _ptr(out), t, *sizes, _ptr(plan["decode_items"]),
                     plan["num_decode"], plan["chunk"], _ptr(part_o), _ptr(part_ml), _ptr(self._attn_counter),
                     plan["rows_max"],
                     _ptr(plan["split_start"]), _ptr(plan["split_count"]), self.decode_variant,
-                    self._tensor_map(storage, head_dim, ctx.page_size),
-                    int(getattr(ctx, "older_keys_settled", False)), _ptr(distance_bias), _ptr(self.err), self._stream())
+                    self._tensor_map(storage, head_dim, ctx.page_size) if value_dim == head_dim else None,
+                    int(getattr(ctx, "older_keys_settled", False)), *options, _ptr(self.err), self._stream())
         self.launches += 2
         if rc:
           raise KernelError(f"sb_attn_decode: {_STATUS.get(rc, rc)}")

@@ -104,11 +104,10 @@ class QKNormAttention(Mixer):
           window=self.window, num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, head_dim=self.head_dim,
           value_dim=self.value_dim, pool=self.pool, batch=batch, page_size=page_size)
       return [plan] if plan is not None else []
-    if self.value_dim != self.head_dim:
-      return []
+    other = {"value_dim": self.value_dim} if self.value_dim != self.head_dim else {}
     plan = ops.attention_graph_plan(
         window=self.window, num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, head_dim=self.head_dim,
-        batch=batch, bucket=bucket, max_burst=max_burst, page_size=page_size)
+        batch=batch, bucket=bucket, max_burst=max_burst, page_size=page_size, **other)
     return [plan] if plan is not None else []
 
   # ---- weights ----------------------------------------------------------------
@@ -123,7 +122,8 @@ class QKNormAttention(Mixer):
 
   def bind(self, tensors, ops) -> None:
     if self.head_dim % 2 == 0:  # (odd head sizes run on the general kernel, which takes any)
-      ops.check_attention(self.head_dim, self.num_heads, self.num_kv_heads)
+      other = (self.value_dim,) if self.value_dim != self.head_dim and self.pool is None else ()
+      ops.check_attention(self.head_dim, self.num_heads, self.num_kv_heads, *other)
     names = [self.q_proj.name] + ([self.k_proj.name, self.v_proj.name] if self.project_kv else [])
     qkv = fuse_rows([tensors[n] for n in names])
     extra = -qkv.shape[0] % 8  # whole 16-byte groups of output features for the products' stores
