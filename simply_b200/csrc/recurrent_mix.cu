@@ -637,12 +637,203 @@ forget_scan_kernel(const float* __restrict__ qf, const float* __restrict__ v, fl
   }
 }
 
+// ---------------------------------------------------------------------------
+// The same walk for long portions, with a patch of the state per lane: 4 neighbouring rows x 4 neighbouring
+// columns, so that a fetched element of q, f, k or v serves four multiply-adds (above, one; there the
+// fetches from shared memory, not the arithmetic, set the pace).  RG lanes (a power of two, 4 to 32) stand over
+// the rows, 32 / RG groups of four columns per warp.  Four tokens go together: the updates of an element are a
+// chain of one multiply-add per token, and the sixteen sums (token, column) of a lane meet over the RG
+// lanes in a butterfly that halves what is passed on at every step.  Heads of 16 to 128 channels in
+// whole groups of four; rows and columns beyond the state's stay zero.
+// ---------------------------------------------------------------------------
+#define PATCH_CHUNK 16
+#define PATCH_BUFFERS 4
+#define PATCH_TOGETHER 8  // tokens (divides the chunk)
+
+// Sums of NV values over RG neighbouring lanes: lane rg (below NV) ends with the value number returned by
+// the steps below, in v[0 .. left); `left` values per lane where there are more values than lanes.
+template <int RG, int NV>
+__device__ __forceinline__ void meet(float (&v)[NV], int rg, int& index) {
+  index = 0;
+  int n = NV;
+#pragma unroll
+  for (int o = 1; o < RG; o <<= 1) {
+    if (n > 1) {
+      n >>= 1;
+      const bool upper = (rg & o) != 0;
+      if (upper) index += n;
+#pragma unroll
+      for (int j = 0; j < NV / 2; ++j)
+        if (j < n) {
+          const float send = upper ? v[j] : v[j + n];
+          const float keep = upper ? v[j + n] : v[j];
+          v[j] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], o);
+    }
+  }
+}
+
+template <int RG, int KINDS, int TOKENS>
+__device__ __forceinline__ void patch_tokens(float (&s)[4][4], const float* tok, int per_token, int row_first,
+                                             int col_local, int rg, float* out_first, size_t out_stride, int cols_left) {
+  constexpr int NP = RG * 4, NV = TOKENS * 4;
+  float y[NV];
+#pragma unroll
+  for (int t = 0; t < TOKENS; ++t) {
+    const float* p = tok + t * per_token;
+    const float4 q4 = *reinterpret_cast<const float4*>(p + row_first);
+    const float4 f4 = *reinterpret_cast<const float4*>(p + NP + row_first);
+    const float4 k4 = KINDS == 3 ? *reinterpret_cast<const float4*>(p + 2 * NP + row_first)
+                                 : make_float4(1.0f - f4.x, 1.0f - f4.y, 1.0f - f4.z, 1.0f - f4.w);
+    const float4 v4 = *reinterpret_cast<const float4*>(p + KINDS * NP + col_local);
+    const float q[4] = {q4.x, q4.y, q4.z, q4.w}, f[4] = {f4.x, f4.y, f4.z, f4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w};
+    const float v[4] = {v4.x, v4.y, v4.z, v4.w};
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      float sum = 0.f;
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        s[r][c] = fmaf(f[r], s[r][c], k[r] * v[c]);
+        sum = fmaf(s[r][c], q[r], sum);
+      }
+      y[t * 4 + c] = sum;
+    }
+  }
+  int index;
+  meet<RG, NV>(y, rg, index);
+  constexpr int LEFT = NV > RG ? NV / RG : 1;
+  if (rg < NV) {
+#pragma unroll
+    for (int j = 0; j < LEFT; ++j) {
+      const int at = index + j, t = at >> 2, c = at & 3;
+      if (c < cols_left) out_first[t * out_stride + c] = y[j];
+    }
+  }
+}
+
+template <int RG, int KINDS>
+__global__ void __launch_bounds__(128)
+linear_patch_kernel(const float* __restrict__ qf, const float* __restrict__ v, float* __restrict__ state,
+                    const int* __restrict__ cu_q, const int* __restrict__ slots, int num_slots, int H, int d, int dv,
+                    float* __restrict__ out, int* err) {
+  pdl_wait_block();
+  pdl_launch_dependents();
+  constexpr int CG = 32 / RG, NP = RG * 4, COLS = 4 * CG * 4;  // column groups per warp; rows of a warp; a block's columns
+  constexpr int PER_TOKEN = KINDS * NP + COLS;
+  extern __shared__ __align__(16) float stage[];  // a ring of PATCH_BUFFERS x PATCH_CHUNK x (q | f | (k) | v)
+  const int h = blockIdx.x, b = blockIdx.y, col0 = blockIdx.z * COLS;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int rg = lane % RG, row_first = rg * 4, col_local = (warp * CG + lane / RG) * 4, col_first = col0 + col_local;
+  const int first = cu_q[b], n = cu_q[b + 1] - first;
+  const int slot = slots[b];
+  if (slot < 0 || slot >= num_slots) {
+    if (threadIdx.x == 0) atomicOr(err, SB_ERR_BAD_SLOT);
+    return;
+  }
+  const int copies = rows_sharing_slot(slots, b, gridDim.y);
+  if (copies == 0) return;  // an earlier row of the slot does this row's work
+  // what no copy ever writes stays zero: rows from d on, columns from the head's last on
+  for (int i = threadIdx.x; i < PATCH_BUFFERS * PATCH_CHUNK * PER_TOKEN; i += blockDim.x) stage[i] = 0.f;
+  __syncthreads();
+  const int n_qf = H * d, d4 = d >> 2, cols_here = min(COLS, dv - col0);
+  const bool wide_v = (dv & 3) == 0;
+  const int v_pieces = wide_v ? cols_here >> 2 : 0;
+  // One 16-byte piece per thread and token (KINDS d / 4 pieces of the vectors, the rest of v).
+  const int piece = threadIdx.x;
+  const float* src = nullptr;
+  size_t src_stride = 0;
+  int dst_at = 0;
+  if (piece < KINDS * d4) {
+    const int kind = piece / d4, c = (piece - kind * d4) * 4;
+    src = qf + ((size_t)first * KINDS + kind) * n_qf + (size_t)h * d + c;
+    src_stride = (size_t)KINDS * n_qf;
+    dst_at = kind * NP + c;
+  } else if (piece < KINDS * d4 + v_pieces) {
+    const int c = (piece - KINDS * d4) * 4;
+    src = v + ((size_t)first * H + h) * dv + col0 + c;
+    src_stride = (size_t)H * dv;
+    dst_at = KINDS * NP + c;
+  }
+  auto issue = [&](int which, int base) {
+    float* buf = stage + which * PATCH_CHUNK * PER_TOKEN;
+    const int count = min(PATCH_CHUNK, n - base);
+    if (src != nullptr) {
+      const float* from = src + (size_t)base * src_stride;
+      for (int i = 0; i < count; ++i) scan_copy16(buf + i * PER_TOKEN + dst_at, from + i * src_stride);
+    }
+    if (!wide_v) {
+      for (int idx = threadIdx.x; idx < count * cols_here; idx += blockDim.x) {
+        const int i = idx / cols_here, c = idx - i * cols_here;
+        scan_copy4(buf + i * PER_TOKEN + KINDS * NP + c, v + ((size_t)(first + base + i) * H + h) * dv + col0 + c);
+      }
+    }
+  };
+  for (int p = 0; p < PATCH_BUFFERS - 1; ++p) {
+    if (p * PATCH_CHUNK < n) issue(p, p * PATCH_CHUNK);
+    asm volatile("cp.async.commit_group;\n" ::);
+  }
+  float* S = state + ((size_t)slot * H + h) * d * dv;
+  float s[4][4];
+#pragma unroll
+  for (int r = 0; r < 4; ++r)
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+      s[r][c] = (row_first + r < d && col_first + c < dv) ? S[(size_t)(row_first + r) * dv + col_first + c] : 0.f;
+  const size_t out_stride = (size_t)H * dv;
+  const int cols_left = dv - col_first;  // of this lane's four (may be none)
+  int which = 0;
+  for (int base = 0; base < n; base += PATCH_CHUNK, which = which + 1 == PATCH_BUFFERS ? 0 : which + 1) {
+    const int count = min(PATCH_CHUNK, n - base);
+    const int ahead = base + (PATCH_BUFFERS - 1) * PATCH_CHUNK;  // goes where the chunk before this one was
+    if (ahead < n) issue(which == 0 ? PATCH_BUFFERS - 1 : which - 1, ahead);
+    asm volatile("cp.async.commit_group;\n" ::);
+    asm volatile("cp.async.wait_group %0;\n" ::"n"(PATCH_BUFFERS - 1));
+    __syncthreads();
+    const float* buf = stage + which * PATCH_CHUNK * PER_TOKEN;
+    float* dst = out + ((size_t)(first + base) * H + h) * dv + col_first;
+    int i = 0;
+    for (; i + PATCH_TOGETHER <= count; i += PATCH_TOGETHER)
+      patch_tokens<RG, KINDS, PATCH_TOGETHER>(s, buf + i * PER_TOKEN, PER_TOKEN, row_first, col_local, rg, dst + i * out_stride, out_stride, cols_left);
+    for (; i < count; ++i)
+      patch_tokens<RG, KINDS, 1>(s, buf + i * PER_TOKEN, PER_TOKEN, row_first, col_local, rg, dst + i * out_stride, out_stride, cols_left);
+    __syncthreads();  // the buffer is filled again in the next round
+  }
+  asm volatile("cp.async.wait_group 0;\n" ::);
+#pragma unroll
+  for (int r = 0; r < 4; ++r)
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+      if (row_first + r < d && col_first + c < dv) S[(size_t)(row_first + r) * dv + col_first + c] = s[r][c];
+}
+
+template <int RG, int KINDS>
+static int launch_linear_patch(const float* qf, const float* v, float* state, const int* cu_q, const int* slots,
+                               int num_seqs, int num_slots, int H, int d, int dv, float* out, int* err,
+                               cudaStream_t stream) {
+  constexpr int COLS = 4 * (32 / RG) * 4;
+  constexpr size_t smem = (size_t)PATCH_BUFFERS * PATCH_CHUNK * (KINDS * RG * 4 + COLS) * sizeof(float);
+  if (smem > 48 * 1024)
+    cudaFuncSetAttribute(linear_patch_kernel<RG, KINDS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  sb_launch_plain(linear_patch_kernel<RG, KINDS>, dim3(H, num_seqs, (dv + COLS - 1) / COLS), 128, smem, stream, qf, v,
+                  state, cu_q, slots, num_slots, H, d, dv, out, err);
+  SB_LAUNCH_CHECK();
+  return 0;
+}
+
 // The walk over float32 inputs qf [T, KINDS, H d] and v [T, H dv].
 template <int KINDS>
 static int launch_forget_scan(const float* qf, const float* v, float* state, const int* cu_q, const int* slots,
                               int num_seqs, int num_slots, int H, int d, int dv, int max_q_len, float* out, int* err,
                               cudaStream_t stream) {
   const bool vec = d % 4 == 0;
+  if (vec && max_q_len >= 64 && d >= 16 && d <= 128) {
+    if (d <= 16) return launch_linear_patch<4, KINDS>(qf, v, state, cu_q, slots, num_seqs, num_slots, H, d, dv, out, err, stream);
+    if (d <= 32) return launch_linear_patch<8, KINDS>(qf, v, state, cu_q, slots, num_seqs, num_slots, H, d, dv, out, err, stream);
+    if (d <= 64) return launch_linear_patch<16, KINDS>(qf, v, state, cu_q, slots, num_seqs, num_slots, H, d, dv, out, err, stream);
+    return launch_linear_patch<32, KINDS>(qf, v, state, cu_q, slots, num_seqs, num_slots, H, d, dv, out, err, stream);
+  }
   const int rows = (vec && d <= 8 * 32) ? 8 : 32;
   int rs = 1;
   while (rs * rows < d) rs <<= 1;
@@ -739,6 +930,7 @@ gated_linear_inputs_kernel(const T* __restrict__ pre, int row_width, int low_off
     float z[TOKENS];
 #pragma unroll
     for (int i = 0; i < TOKENS; ++i) z[i] = bias[c];
+#pragma unroll 8
     for (int r = 0; r < rank; ++r) {
       const float wr = w[(size_t)r * n_qf + c];
 #pragma unroll

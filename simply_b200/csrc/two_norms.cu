@@ -53,26 +53,32 @@ __device__ __forceinline__ void block_sums(float (&v)[M], float* scratch) {
   }
 }
 
-// Rows of one 16-byte vector per thread: everything a block needs is loaded before its first sum.
+// Rows of one 16-byte vector per thread: everything a block needs is loaded before its first sum.  ROWS 1 is
+// the kernel of short steps: there the weights, the request's place and its old row are fetched ahead as
+// well.  Larger ROWS keep the registers low, so that one block's sums and stores overlap another's loads.
 template <typename T, int ROWS, int MAX_THREADS>
-__global__ void __launch_bounds__(MAX_THREADS) two_norms_kernel(const TwoNorms p) {
+__global__ void __launch_bounds__(MAX_THREADS, ROWS == 1 ? 1 : 2) two_norms_kernel(const TwoNorms p) {
   constexpr int N = Vec<T>::N;
+  constexpr bool AHEAD = ROWS == 1;
   __shared__ float scratch[(ROWS + 1) * 32];
   const int i = threadIdx.x * N;
   const bool on = i < p.width;
   float w1[N], w2[N], sh[N];
+  auto load_weights = [&]() {
 #pragma unroll
-  for (int k = 0; k < N; ++k) w1[k] = w2[k] = sh[k] = 0.f;
-  if (on) {  // weights: before the wait
-    load_scalars<N>(p.w1, p.w1_f32, i, w1);
-    if (p.w2 != nullptr) load_scalars<N>(p.w2, p.w2_f32, i, w2);
-    if (p.shift != nullptr) load_scalars<N>(p.shift, 1, i, sh);
-  }
+    for (int k = 0; k < N; ++k) w1[k] = w2[k] = sh[k] = 0.f;
+    if (on) {
+      load_scalars<N>(p.w1, p.w1_f32, i, w1);
+      if (p.w2 != nullptr) load_scalars<N>(p.w2, p.w2_f32, i, w2);
+      if (p.shift != nullptr) load_scalars<N>(p.shift, 1, i, sh);
+    }
 #pragma unroll
-  for (int k = 0; k < N; ++k) {
-    w1[k] += p.one1;
-    w2[k] += p.one2;
-  }
+    for (int k = 0; k < N; ++k) {
+      w1[k] += p.one1;
+      w2[k] += p.one2;
+    }
+  };
+  if constexpr (AHEAD) load_weights();  // (no kernel writes them: before the wait)
   pdl_wait_block();
   pdl_launch_dependents();
   const float inv_width = 1.0f / (float)p.width;
@@ -81,18 +87,18 @@ __global__ void __launch_bounds__(MAX_THREADS) two_norms_kernel(const TwoNorms p
     for (int k = 0; k < N; ++k) v[k] = 0.f;
     if (!on || t < 0 || t >= p.num_tokens) return;
     const size_t at = (size_t)t * p.width + i;
-    float b[N], b2[N];
 #pragma unroll
     for (int k = 0; k < N; k += 4) Vec<float>::load(p.h + at + k, v + k);
-    if (p.branch != nullptr) Vec<T>::load(reinterpret_cast<const T*>(p.branch) + at, b);
-    if (p.branch2 != nullptr) Vec<T>::load(reinterpret_cast<const T*>(p.branch2) + at, b2);
+    float b[N];
     if (p.branch != nullptr) {
+      Vec<T>::load(reinterpret_cast<const T*>(p.branch) + at, b);
 #pragma unroll
       for (int k = 0; k < N; ++k) v[k] += b[k];
     }
     if (p.branch2 != nullptr) {
+      Vec<T>::load(reinterpret_cast<const T*>(p.branch2) + at, b);
 #pragma unroll
-      for (int k = 0; k < N; ++k) v[k] += b2[k];
+      for (int k = 0; k < N; ++k) v[k] += b[k];
     }
   };
   const int t0 = blockIdx.x * ROWS;
@@ -100,6 +106,39 @@ __global__ void __launch_bounds__(MAX_THREADS) two_norms_kernel(const TwoNorms p
   float x[ROWS + 1][N], sums[ROWS + 1];
 #pragma unroll
   for (int m = 0; m <= ROWS; ++m) load_row(p.shift != nullptr || m > 0 ? t0 - 1 + m : -1, x[m]);
+  // The request of every row, and for a request's first token the row's part of the state.
+  int first[ROWS], last[ROWS], slot[ROWS], copies[ROWS];
+  float old[AHEAD ? N : 1];
+#pragma unroll
+  for (int m = 0; m < ROWS; ++m) {
+    const int t = t0 + m;
+    first[m] = -1;
+    last[m] = t;
+    slot[m] = 0;
+    copies[m] = 1;
+    if (p.shift != nullptr && t < p.num_tokens) {
+      const int b = p.token_seq[t];
+      first[m] = p.cu_q[b];
+      if (first[m] == t) {
+        last[m] = p.cu_q[b + 1] - 1;
+        slot[m] = p.slots[b];
+        if (slot[m] < 0 || slot[m] >= p.num_slots) {
+          if (threadIdx.x == 0) atomicOr(p.err, SB_ERR_BAD_SLOT);
+          copies[m] = 0;
+        } else {
+          copies[m] = rows_sharing_slot(p.slots, b, p.num_seqs);  // 0: an earlier row of the slot writes this one's results
+        }
+        if constexpr (AHEAD) {
+#pragma unroll
+          for (int k = 0; k < N; ++k) old[k] = 0.f;
+          if (on && copies[m] > 0) {
+#pragma unroll
+            for (int k = 0; k < N; k += 4) Vec<float>::load(p.state + (size_t)slot[m] * p.width + i + k, old + k);
+          }
+        }
+      }
+    }
+  }
 #pragma unroll
   for (int m = 0; m <= ROWS; ++m) {
     sums[m] = 0.f;
@@ -107,73 +146,69 @@ __global__ void __launch_bounds__(MAX_THREADS) two_norms_kernel(const TwoNorms p
     for (int k = 0; k < N; ++k) sums[m] = fmaf(x[m][k], x[m][k], sums[m]);
   }
   block_sums<ROWS + 1>(sums, scratch);
+  if constexpr (!AHEAD) load_weights();
 #pragma unroll
   for (int m = 1; m <= ROWS; ++m) {
     const int t = t0 - 1 + m;
     if (t >= p.num_tokens) break;
+    if (copies[m - 1] == 0) continue;
     const float mean = sums[m] * inv_width;
     const float r1 = 1.0f / sqrtf(mean + p.eps1);
-    float y[N], out[N], y2[N];
+    const bool starts = first[m - 1] == t;  // (the same for the whole block)
+    float out[N];
+    if (starts) {
+      float* st = p.state + (size_t)slot[m - 1] * p.width + i;
 #pragma unroll
-    for (int k = 0; k < N; ++k) out[k] = y[k] = x[m][k] * r1 * w1[k];
-    int copies = 1;
-    if (p.shift != nullptr) {
-      const int b = p.token_seq[t], first = p.cu_q[b], n = p.cu_q[b + 1] - first;
-      float before[N];
-      if (t > first) {
-        const float rp = 1.0f / sqrtf(sums[m - 1] * inv_width + p.eps1);
+      for (int k = 0; k < N; ++k) out[k] = 0.f;
+      if constexpr (AHEAD) {
 #pragma unroll
-        for (int k = 0; k < N; ++k) before[k] = x[m - 1][k] * rp * w1[k];
-      } else {
-        const int slot = p.slots[b];
-        if (slot < 0 || slot >= p.num_slots) {
-          if (threadIdx.x == 0) atomicOr(p.err, SB_ERR_BAD_SLOT);
-          continue;
-        }
-        copies = rows_sharing_slot(p.slots, b, p.num_seqs);
-        if (copies == 0) continue;  // an earlier row of the slot writes this one's results
-        float* st = p.state + (size_t)slot * p.width + i;
+        for (int k = 0; k < N; ++k) out[k] = old[k];
+      } else if (on) {
 #pragma unroll
-        for (int k = 0; k < N; ++k) before[k] = 0.f;
-        if (on) {
+        for (int k = 0; k < N; k += 4) Vec<float>::load(st + k, out + k);
+      }
+      float z[N], rl = r1;
 #pragma unroll
-          for (int k = 0; k < N; k += 4) Vec<float>::load(st + k, before + k);
-        }
-        if (n == 1) {
-          if (on) {
+      for (int k = 0; k < N; ++k) z[k] = x[m][k];
+      if (last[m - 1] != t) {
+        float s[1] = {0.f};
+        load_row(last[m - 1], z);
 #pragma unroll
-            for (int k = 0; k < N; k += 4) Vec<float>::store(st + k, y + k);
-          }
-        } else {
-          float z[N], s[1] = {0.f};
-          load_row(first + n - 1, z);
-#pragma unroll
-          for (int k = 0; k < N; ++k) s[0] = fmaf(z[k], z[k], s[0]);
-          block_sums<1>(s, scratch);
-          const float rl = 1.0f / sqrtf(s[0] * inv_width + p.eps1);
-#pragma unroll
-          for (int k = 0; k < N; ++k) z[k] *= rl * w1[k];
-          if (on) {
-#pragma unroll
-            for (int k = 0; k < N; k += 4) Vec<float>::store(st + k, z + k);
-          }
-        }
+        for (int k = 0; k < N; ++k) s[0] = fmaf(z[k], z[k], s[0]);
+        block_sums<1>(s, scratch);
+        rl = 1.0f / sqrtf(s[0] * inv_width + p.eps1);
       }
 #pragma unroll
-      for (int k = 0; k < N; ++k) out[k] = fmaf(before[k] - y[k], sh[k], y[k]);
+      for (int k = 0; k < N; ++k) z[k] *= rl * w1[k];
+      if (on) {
+#pragma unroll
+        for (int k = 0; k < N; k += 4) Vec<float>::store(st + k, z + k);
+      }
+    } else {
+      const float rp = 1.0f / sqrtf(sums[m - 1] * inv_width + p.eps1);
+#pragma unroll
+      for (int k = 0; k < N; ++k) out[k] = x[m - 1][k] * rp * w1[k];
     }
     if (!on) continue;
-    const float r2 = p.eps2 == p.eps1 ? r1 : 1.0f / sqrtf(mean + p.eps2);
 #pragma unroll
-    for (int k = 0; k < N; ++k) y2[k] = x[m][k] * r2 * w2[k];
-    for (int c = 0; c < copies; ++c) {  // (rows that repeat a request follow it)
+    for (int k = 0; k < N; ++k) {
+      const float y = x[m][k] * r1 * w1[k];
+      out[k] = fmaf(out[k] - y, sh[k], y);  // (without a shift its factors are zero)
+    }
+    const float r2 = p.eps2 == p.eps1 ? r1 : 1.0f / sqrtf(mean + p.eps2);
+    for (int c = 0; c < copies[m - 1]; ++c) {  // (rows that repeat a request follow it)
       const size_t at = (size_t)(t + c) * p.width + i;
       if (p.h_out != nullptr) {
 #pragma unroll
         for (int k = 0; k < N; k += 4) Vec<float>::store(p.h_out + at + k, x[m] + k);
       }
       Vec<T>::store(reinterpret_cast<T*>(p.y) + at, out);
-      if (p.w2 != nullptr) Vec<T>::store(reinterpret_cast<T*>(p.y2) + at, y2);
+      if (p.w2 != nullptr) {
+        float y2[N];
+#pragma unroll
+        for (int k = 0; k < N; ++k) y2[k] = x[m][k] * r2 * w2[k];
+        Vec<T>::store(reinterpret_cast<T*>(p.y2) + at, y2);
+      }
     }
   }
 }
@@ -264,7 +299,7 @@ extern "C" int sb_residual_two_norms(const float* h, float* h_out, const void* b
     const int threads = ((width / vec + 31) / 32) * 32;
     // Many tokens: several per block, so that fewer rows are read once more for the token after them.
     // (Blocks of more than 512 threads keep to one row: their registers would not hold more.)
-    int rows = rows_per_block > 0 ? rows_per_block : (num_tokens >= 512 && shift != nullptr ? 3 : 1);
+    int rows = rows_per_block > 0 ? rows_per_block : (num_tokens >= 512 && shift != nullptr ? 2 : 1);
     if (threads > 512) rows = 1;
 #define SB_TWO_NORMS_OF(T_, R_, M_) \
   sb_launch(two_norms_kernel<T_, R_, M_>, (unsigned)((num_tokens + R_ - 1) / R_), threads, 0, stream, p)

@@ -1,8 +1,8 @@
 """Prefill and decode throughput of a design beside the engine's closest other model at equal size
-(Generax beside Gemma 2, Sapivik beside Generax, Zesapel beside Sapivik, Nulezen beside Sapivik), and the time of every kernel
-call of one step of each with its share of the measured peaks.
+(Generax beside Gemma 2, Sapivik beside Generax, Zesapel beside Sapivik, Nulezen beside Sapivik, Mononex beside
+Sapivik and Zesapel), and the time of every kernel call of one step of each with its share of the measured peaks.
 
-Used by `bench.py --design generax|sapivik|zesapel|nulezen` (the default benchmark does not import this file).  Layer
+Used by `bench.py --design generax|sapivik|zesapel|nulezen|mononex` (the default benchmark does not import this file).  Layer
 shapes resemble a real model's; weights are random.  Per size and design:
 
 * prefill: one 2,048-token prompt in one step, median of 5 after 3 warm-up steps, CUDA events;
@@ -120,6 +120,28 @@ def nulezen_dict(s: dict) -> dict:
   return d
 
 
+def mononex_dict(s: dict) -> dict:
+  """Attention by chunks, attention over latents and gated linear attention in turn (one layer in three is
+  plain attention and one in three recurrent, as in the neighbours' arms), each beside a dense feed-forward
+  without a gate; the second attention layer reads the first one's keys.  The latent's sizes are the
+  Zesapel arm's, the recurrence's heads the Sapivik arm's."""
+  att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+         "mask": {"size": WINDOW}}
+  latent = {"heads": s["heads"], "dim": s["dim"], "rot_dim": s["dim"] // 2, "vdim": s["dim"], "q_rank": s["width"] // 2,
+            "kv_rank": 4 * s["dim"], "scale": (s["dim"] + s["dim"] // 2) ** -0.5,
+            "rot": {"dims": s["dim"] // 2, "base": 10000.0,
+                    "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+  rec = {"heads": s["heads"], "dim": s["dim"], "vdim": s["dim"], "tau": 16.0}
+  kinds = (("attention", att), ("latent_attention", latent), ("gla", rec))
+  layers = []
+  for i in range(s["layers"]):
+    kind, m = kinds[i % 3]
+    m = dict(m, kv_from=0) if kind == "attention" and i > 0 else dict(m)
+    layers.append({"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": s["ff"]}})
+  return {"architecture": "Mononex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "layers": layers,
+          "decay_rank": RANK, "max_context": 8192}
+
+
 def gemma2_dict(s: dict) -> dict:
   return {"architectures": ["Gemma2ForCausalLM"], "hidden_size": s["width"], "num_hidden_layers": s["layers"],
           "num_attention_heads": s["heads"], "num_key_value_heads": s["kv_heads"], "head_dim": s["dim"],
@@ -166,7 +188,7 @@ class TimedOps:
       moved = sum(_nbytes(t) for t in tensors) + _nbytes(out)
       flops = 0.0
       ctx = next((a for a in list(args) + list(kw.values()) if hasattr(a, "num_tokens") and hasattr(a, "cu_q")), None)
-      if name in ("linear", "gated_linear", "lm_head", "linear_xielu", "linear_wide"):
+      if name in ("linear", "gated_linear", "lm_head", "linear_xielu", "linear_wide", "linear_relu_squared"):
         x, w = args[0], args[1]
         flops = 2.0 * x.shape[0] * w.shape[0] * w.shape[1]
       if name == "mix_experts":
@@ -185,10 +207,14 @@ class TimedOps:
         pairs = seen = 0
         for s0, n in zip(starts, lens):
           pos = np.arange(s0, s0 + n)
-          keys = np.minimum(pos + 1, window)
+          chunk = kw.get("key_chunk")
+          keys = pos % chunk + 1 if chunk else np.minimum(pos + 1, window)
           if kw.get("pooled") is not None:
             keys = keys + np.maximum(pos - window + 1, 0) // kw["pooled"][2]
           pairs += int(keys.sum())
+          if chunk:
+            seen += int(s0 + n - s0 // chunk * chunk)
+            continue
           seen += int(min(s0 + n, window + n)) + (int((s0 + n) // kw["pooled"][2]) if kw.get("pooled") is not None else 0)
         flops = 2.0 * pairs * heads * (dim + vdim)
         moved += seen * kv_heads * (dim + (0 if kw.get("values_in_keys") else vdim)) * args[1].element_size()
@@ -199,6 +225,10 @@ class TimedOps:
         flops = 6.0 * args[0].shape[0] * kw["num_heads"] * kw["head_dim"] * kw["value_dim"]
       if name == "forget_gate_scan" and ctx is not None:
         moved += 2 * args[3][0].numel() * 4 * ctx.num_seqs
+        flops = 5.0 * args[0].shape[0] * kw["num_heads"] * kw["head_dim"] * kw["value_dim"]
+      if name == "gated_linear_scan" and ctx is not None:
+        state = args[5]
+        moved += 2 * state[0].numel() * 4 * ctx.num_seqs - _nbytes(state)
         flops = 5.0 * args[0].shape[0] * kw["num_heads"] * kw["head_dim"] * kw["value_dim"]
       if name in ("general_delta_scan", "state_space_scan") and ctx is not None:
         state = args[4] if name == "general_delta_scan" else args[6]
@@ -261,13 +291,13 @@ def _prefill_ms(engine, tokens: int, vocab: int) -> float:
 
 
 PAIRS = {"generax": ("generax", "gemma2"), "sapivik": ("sapivik", "generax"), "zesapel": ("zesapel", "sapivik"),
-         "nulezen": ("nulezen", "sapivik")}
+         "nulezen": ("nulezen", "sapivik"), "mononex": ("mononex", "sapivik", "zesapel")}
 DICTS = {"generax": generax_dict, "gemma2": gemma2_dict, "sapivik": sapivik_dict, "zesapel": zesapel_dict,
-         "nulezen": nulezen_dict}
+         "nulezen": nulezen_dict, "mononex": mononex_dict}
 
 
 def run(args, peaks: dict, time_decode, design: str = "generax") -> dict:
-  """The design and its neighbour at every size; `time_decode` is bench.py's burst timer."""
+  """The design and its neighbours at every size; `time_decode` is bench.py's burst timer."""
   from simply_b200 import Engine, EngineConfig, StepEntry
   from simply_b200.config import config_from_dict
 
