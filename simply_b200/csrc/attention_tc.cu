@@ -1,5 +1,7 @@
 // Ragged paged prefill attention on the fifth-generation tensor cores (tcgen05), compiled once
-// per head size (-DSB_HEAD_DIM=N, N a multiple of 64 up to 256).
+// per head size (-DSB_HEAD_DIM=N, N a multiple of 16 up to 256) and, where value heads have another size,
+// per pair of sizes (-DSB_VALUE_DIM=M, likewise).  A size that is no multiple of 64 takes whole slabs of 64
+// dims in shared memory, whose rest the copies fill with zeros.
 //
 //   s = q . k                 (q is already rotated and scaled)
 //   s = cap * tanh(s / cap)   if cap > 0          simply/model_lib.py:621-626
@@ -14,7 +16,7 @@
 //                              product runs two key tiles ahead of the one below)
 //   P            = softmax numerators of S as bfloat16, written over S in tensor memory: the
 //                  next product's 128-row operand comes from there
-//   O[128 x DH] += P . V       tcgen05.mma, accumulator in tensor memory for the whole walk
+//   O[128 x DV] += P . V       tcgen05.mma, accumulator in tensor memory for the whole walk
 // Roles: warp 0 TMA producer of Q (once) and of the key tiles, warp 2 of the value tiles (both
 // from the paged cache through the block table), warps 1 and 3 MMA issue (one thread each: Q.K^T
 // and P.V), warps 4..19
@@ -35,15 +37,17 @@
 #ifndef SB_HEAD_DIM
 #define SB_HEAD_DIM 256
 #endif
-
-#if SB_HEAD_DIM % 64 == 0
+#ifndef SB_VALUE_DIM
+#define SB_VALUE_DIM SB_HEAD_DIM
+#endif
 
 namespace {
 
 using namespace sbx;
 
-constexpr int DH = SB_HEAD_DIM;
-constexpr int BM = 128, BN = 64, SLABS = DH / 64;
+constexpr int DH = SB_HEAD_DIM, DV = SB_VALUE_DIM;
+constexpr int BM = 128, BN = 64, SLABS = (DH + 63) / 64, VSLABS = (DV + 63) / 64;
+static_assert(DH % 16 == 0 && DV % 16 == 0 && DH <= 256 && DV <= 256, "sizes are multiples of 16 up to 256");
 // With a head size of 256 the first 128 dims of Q live in tensor memory (as the 128-row operand of
 // the first eight products of a tile, which then read only K from shared memory: with Q from
 // shared memory a 128 x 64 x 16 product waits about 75 cycles for its operands, twice what it
@@ -51,17 +55,16 @@ constexpr int BM = 128, BN = 64, SLABS = DH / 64;
 constexpr int QT_DIMS = DH == 256 ? 128 : 0;          // dims of Q in tensor memory
 constexpr int QT_COLS = QT_DIMS / 2;                  // two bfloat16 per column
 constexpr int QS_SLABS = SLABS - QT_DIMS / 64;        // slabs of 64 dims of Q in shared memory
-constexpr int Q_BYTES = BM * QS_SLABS * 128, KV_TILE_BYTES = BN * DH * 2;
+constexpr int Q_BYTES = BM * QS_SLABS * 128, K_TILE_BYTES = BN * SLABS * 128, V_TILE_BYTES = BN * VSLABS * 128;
 constexpr int K_STAGES = 3, V_STAGES = 2;
 constexpr int GROUPS = 2;          // softmax groups: group g takes the key tiles j with j % 2 == g
 constexpr int SPLIT = 2;           // softmax threads per query row within a group
 constexpr int CW = BN / SPLIT;     // columns of a key tile per softmax thread
-constexpr int OW = DH / (GROUPS * SPLIT);  // columns of O per softmax thread in the epilogue
-static_assert(CW == 32 && OW % 16 == 0, "tensor-memory loads of 32 and 16 columns");
+static_assert(CW == 32, "tensor-memory loads of 32 columns");
 constexpr int TC_THREADS = 128 + 128 * GROUPS * SPLIT;  // warps: key producer, MMA, value producer, spare, softmax
 constexpr int S_BUFS = 3;                               // S buffers: Q.K^T runs two key tiles ahead of P.V
 constexpr int S_COL0 = 0, O_COL0 = S_BUFS * BN;         // S buffers from column 0, O behind them
-constexpr int QT_COL0 = O_COL0 + DH;                    // Q's first dims behind O
+constexpr int QT_COL0 = O_COL0 + DV;                    // Q's first dims behind O
 constexpr int TMEM_COLS = QT_COL0 + QT_COLS <= 256 ? 256 : 512;  // a power of two that holds the S buffers, O and Q's part
 static_assert(QT_COL0 + QT_COLS <= 512, "tensor memory has 512 columns");
 constexpr float LOG2E = 1.4426950408889634f;
@@ -114,14 +117,15 @@ __device__ __forceinline__ int lowest_key(const TcParams& p, int pos) {
 
 __global__ void __launch_bounds__(TC_THREADS)
 attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map_q,
-                       const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_out) {
+                       const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
+                       const __grid_constant__ CUtensorMap map_out) {
   pdl_wait();
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char smem_raw[];
   unsigned char* base = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
   unsigned char* sq = base;                               // [QS_SLABS][128 rows][128 B]
   unsigned char* sk = sq + Q_BYTES;                       // [K_STAGES][SLABS][64 keys][128 B]
-  unsigned char* sv = sk + K_STAGES * KV_TILE_BYTES;      // [V_STAGES][SLABS][64 keys][128 B]
+  unsigned char* sv = sk + K_STAGES * K_TILE_BYTES;       // [V_STAGES][VSLABS][64 keys][128 B]
   __shared__ __align__(8) uint64_t q_full, qt_ready, k_full[K_STAGES], v_full[V_STAGES], s_full[2 * S_BUFS], p_ready[4], pv_done[S_BUFS], o_done, x_bar[GROUPS][4], m_bar[2][4], l_bar[4];
   __shared__ float row_max[GROUPS][SPLIT][BM];  // the parts' row maxima of a group's tile
   __shared__ float row_m[2][BM];                // the running maximum after a tile, by tile parity
@@ -162,7 +166,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
   }
   // The distance term depends on (head, distance) alone: with a window that fits, a table of it
   // spares the softmax threads a logarithm per score (the special-function pipe is their busiest).
-  float* bias_tab = reinterpret_cast<float*>(sv + V_STAGES * KV_TILE_BYTES);
+  float* bias_tab = reinterpret_cast<float*>(sv + V_STAGES * V_TILE_BYTES);
   if (p.bias_table) {
     for (int i = threadIdx.x; i < p.window * group; i += TC_THREADS) {
       const int d = i / group, h = m * group + (i - d * group);
@@ -185,7 +189,9 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
       const bool values = warp == 2;
       uint64_t* full = values ? v_full : k_full;
       unsigned char* ring = values ? sv : sk;
-      const int stages = values ? V_STAGES : K_STAGES;
+      const int stages = values ? V_STAGES : K_STAGES, slabs = values ? VSLABS : SLABS;
+      const int tile_bytes = values ? V_TILE_BYTES : K_TILE_BYTES;
+      const CUtensorMap* map = values ? &map_v : &map_k;
       if (!values && QS_SLABS > 0) {
         mbar_arrive_expect_tx(&q_full, Q_BYTES);
         for (int sl = 0; sl < QS_SLABS; ++sl)  // box: 64 dims x G heads x 128 / G tokens, rows in (token, head) order
@@ -210,7 +216,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
           const long long page = p.block_table[(size_t)b * p.max_pages + key / p.page_size];
           if (page >= 0 && page < p.num_pages) ++boxes;
         }
-        mbar_arrive_expect_tx(&full[s], boxes * SLABS * p.box_rows * 128);
+        mbar_arrive_expect_tx(&full[s], boxes * slabs * p.box_rows * 128);
         for (int r = 0; r < BN; r += p.box_rows) {
           const int key = j0 + r;
           if (key >= kv_hi || key + p.box_rows <= kv_lo) continue;
@@ -219,9 +225,9 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
             atomicOr(p.err, SB_ERR_BAD_PAGE);
             continue;
           }
-          const long long row = ((page * 2 + (values ? 1 : 0)) * p.num_kv_heads + m) * p.page_size + (key & (p.page_size - 1));
-          for (int sl = 0; sl < SLABS; ++sl)
-            tma_load_2d(ring + s * KV_TILE_BYTES + sl * (BN * 128) + r * 128, &map_kv, sl * 64, (int)row, &full[s]);
+          const int row = m * p.page_size + (key & (p.page_size - 1));  // of the page's key rows, or of its value rows
+          for (int sl = 0; sl < slabs; ++sl)
+            tma_load_3d(ring + s * tile_bytes + sl * (BN * 128) + r * 128, map, sl * 64, row, (int)page, &full[s]);
         }
       }
     }
@@ -253,7 +259,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
           break;
         }
         tc_fence_after_sync();
-        const uint64_t k_desc = k_desc0 + (uint64_t)((s * KV_TILE_BYTES) >> 4);
+        const uint64_t k_desc = k_desc0 + (uint64_t)((s * K_TILE_BYTES) >> 4);
         const uint32_t s_tmem = tmem + S_COL0 + (j % S_BUFS) * BN;
 #pragma unroll
         for (int ks = 0; ks < DH / 16; ++ks) {
@@ -273,7 +279,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
   } else if (warp == 3) {
     // ---- MMA issue of O += P.V (one thread) ---------------------------------------------------------
     if (lane == 0) {
-      const uint32_t idesc_pv = idesc_bf16_f32(BM, DH, false, true);  // V: the N index (dims) is contiguous
+      const uint32_t idesc_pv = idesc_bf16_f32(BM, DV, false, true);  // V: the N index (dims) is contiguous
       const uint64_t v_desc0 = smem_desc_sw128(sv, BN * 128, 1024);
       bool ok = true;
       for (int j = 0; ok && j < n_tiles; ++j) {
@@ -290,7 +296,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
           // P comes from tensor memory, where it overwrote the tile's S: 16 keys are 8 columns of
           // two bfloat16 each.  16 keys further in V = 16 rows of 128 bytes; the next 64 dims are
           // one slab (BN * 128 bytes) further.
-          const uint64_t bdesc = v_desc0 + (uint64_t)((s * KV_TILE_BYTES + kk * 16 * 128) >> 4);
+          const uint64_t bdesc = v_desc0 + (uint64_t)((s * V_TILE_BYTES + kk * 16 * 128) >> 4);
           tc_mma_f16_ts(tmem + O_COL0, tmem + S_COL0 + (j % S_BUFS) * BN + kk * 8, bdesc, idesc_pv, j > 0 || kk > 0);
         }
         tc_commit(&pv_done[j % S_BUFS]);  // also frees the value tile's stage
@@ -449,7 +455,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
         }
         tc_fence_after_sync();
 #pragma unroll 1
-        for (int c = part * (DH / SPLIT); c < (part + 1) * (DH / SPLIT); c += 16) {
+        for (int c = part * 16; c < DV; c += 16 * SPLIT) {
           uint32_t o[16];
           tmem_load_32x16(tmem + lane_base + O_COL0 + c, o);
           tmem_wait_load();
@@ -479,11 +485,11 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
           ok = false;
           break;
         }
-        for (int i = (quarter + 4 * part) * 32 + lane; i < BN * SLABS * 8; i += 128 * SPLIT) {
+        for (int i = (quarter + 4 * part) * 32 + lane; i < BN * VSLABS * 8; i += 128 * SPLIT) {
           const int key_row = (i / 8) % BN, sl = i / (8 * BN), c = i % 8;
           const int key = j0 + key_row;
           if (key < kv_lo || key >= kv_hi)
-            *reinterpret_cast<uint4*>(sv + s * KV_TILE_BYTES + sl * (BN * 128) + key_row * 128 + c * 16) = make_uint4(0, 0, 0, 0);
+            *reinterpret_cast<uint4*>(sv + s * V_TILE_BYTES + sl * (BN * 128) + key_row * 128 + c * 16) = make_uint4(0, 0, 0, 0);
         }
         fence_proxy_async();  // the zeroed value rows are visible to the tensor core's reads
       }
@@ -506,7 +512,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
     }
     if (ok && !mbar_wait_bounded(&o_done, 0)) ok = false;
     tc_fence_after_sync();
-    // A full tile leaves through shared memory (the key stages, free by now) in the layout Q came
+    // A full tile leaves through shared memory (the key and value stages, free by now) in the layout Q came
     // in, as TMA stores of whole lines: stored straight from registers, 16 bytes per lane at a
     // row's stride, the 64 KB of a tile took 3.7 us of a block's time.  A tile that ends with its
     // sequence is stored row by row: a box would reach into the next sequence's rows.
@@ -515,9 +521,9 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
       // Every lane takes part in the warp-wide tensor-memory loads; only rows of the sequence store.
       const float inv = l > 0.f ? 1.0f / l : 0.f;
       const bool valid = r < rows_valid;
-      bf16* op = p.out + ((size_t)(row0 + i0 + (valid ? r / group : 0)) * p.num_q_heads + m * group + (valid ? r % group : 0)) * DH;
+      bf16* op = p.out + ((size_t)(row0 + i0 + (valid ? r / group : 0)) * p.num_q_heads + m * group + (valid ? r % group : 0)) * DV;
 #pragma unroll 1
-      for (int c = sw * OW; c < (sw + 1) * OW; c += 16) {
+      for (int c = sw * 16; c < DV; c += 16 * GROUPS * SPLIT) {
         uint32_t o[16];
         tmem_load_32x16(tmem + lane_base + O_COL0 + c, o);
         tmem_wait_load();
@@ -545,7 +551,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
       fence_proxy_async();
       asm volatile("bar.sync 1, %0;\n" ::"n"(128 * GROUPS * SPLIT) : "memory");  // the softmax warps
       if (warp == 4 && lane == 0 && !s_failed) {
-        for (int sl = 0; sl < SLABS; ++sl) tma_store_3d(&map_out, sk + sl * (BM * 128), sl * 64, m * group, row0 + i0);
+        for (int sl = 0; sl < VSLABS; ++sl) tma_store_3d(&map_out, sk + sl * (BM * 128), sl * 64, m * group, row0 + i0);
         tma_store_commit();
         tma_store_wait_read();  // shared memory has been read; the grid's end covers the writes
       }
@@ -558,21 +564,27 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
   if (warp == 1) tmem_dealloc(tmem, TMEM_COLS);
 }
 
-constexpr size_t TC_SMEM = (size_t)Q_BYTES + (K_STAGES + V_STAGES) * KV_TILE_BYTES + 1024;
+constexpr size_t TC_SMEM = (size_t)Q_BYTES + K_STAGES * K_TILE_BYTES + V_STAGES * V_TILE_BYTES + 1024;
 // Room for the table of distance terms behind the tiles: what a block may have (227 KB) less its
 // static shared memory, 48 KB at most.
 constexpr size_t TC_SMEM_LIMIT = 232448 - 6144;
 constexpr size_t TC_TABLE_MAX = TC_SMEM_LIMIT <= TC_SMEM ? 0 : (TC_SMEM_LIMIT - TC_SMEM < 48 * 1024 ? TC_SMEM_LIMIT - TC_SMEM : 48 * 1024);
 static_assert(QT_DIMS == 0 || QT_DIMS / (GROUPS * SPLIT) == 32, "each softmax thread stores 32 dims of Q");
+static_assert(BM * VSLABS * 128 <= K_STAGES * K_TILE_BYTES + V_STAGES * V_TILE_BYTES, "the result leaves through the stages");
 static_assert(V_STAGES == 2, "the zeroing of value rows looks two tiles back");
 
 }  // namespace
 
 #define SB_CONCAT2(a, b) a##b
 #define SB_CONCAT(a, b) SB_CONCAT2(a, b)
+#if SB_VALUE_DIM == SB_HEAD_DIM
 #define SB_FN(name) SB_CONCAT(SB_CONCAT(name, _hd), SB_HEAD_DIM)
+#else
+#define SB_FN(name) SB_CONCAT(SB_CONCAT(SB_CONCAT(name, _hd), SB_HEAD_DIM), SB_CONCAT(v, SB_VALUE_DIM))
+#endif
 
-// Ragged prefill attention on tcgen05.  q: [T, Hq, DH]; cache: [pages, 2, Hkv, page_size, DH];
+// Ragged prefill attention on tcgen05.  q: [T, Hq, DH]; out: [T, Hq * DV]; cache: per page [Hkv, page_size, DH]
+// keys, then [Hkv, page_size, DV] values;
 // items: [num_items, 3] (sequence, first token of a tile of 128 / G tokens, kv head), in the order in
 // which the blocks are to start (longest walk first over all heads, so that the SMs that are free
 // first take the longest walks left).  Returns -11 when
@@ -590,19 +602,25 @@ static int prefill_tc_launch(const void* q, const void* cache, const int* block_
   if (group > BM || BM % group || (page_size & (page_size - 1))) return -11;
   SbEncodeTiled encode = sb_encode_tiled();
   if (!encode) return -12;
-  CUtensorMap map_q, map_kv, map_out;
-  for (int which = 0; which < 2; ++which) {  // q and out have the same shape
-    const cuuint64_t dims[3] = {(cuuint64_t)DH, (cuuint64_t)num_q_heads, (cuuint64_t)num_tokens};
-    const cuuint64_t strides[2] = {(cuuint64_t)DH * 2, (cuuint64_t)num_q_heads * DH * 2};
-    const cuuint32_t box[3] = {64u, (cuuint32_t)group, (cuuint32_t)(BM / group)};
+  CUtensorMap map_q, map_k, map_v, map_out;
+  // Every map has rows of one size: (dims, rows, outer), fetched or stored in boxes of 64 dims.
+  auto make = [&](CUtensorMap* map, const void* base, int dim, long long rows, long long outer, long long outer_bytes, int box_rows,
+                  int box_outer) {
+    const cuuint64_t dims[3] = {(cuuint64_t)dim, (cuuint64_t)rows, (cuuint64_t)outer};
+    const cuuint64_t strides[2] = {(cuuint64_t)dim * 2, (cuuint64_t)outer_bytes};
+    const cuuint32_t box[3] = {64u, (cuuint32_t)box_rows, (cuuint32_t)box_outer};
     const cuuint32_t elem[3] = {1u, 1u, 1u};
-    if (encode(which == 0 ? &map_q : &map_out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, which == 0 ? const_cast<void*>(q) : out, dims, strides, box, elem,
-               CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
-      return -12;
-  }
+    return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, elem,
+                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                  CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+  };
   const int box_rows = page_size < BN ? page_size : BN;
-  if (sb_make_map_2d(&map_kv, cache, (long long)num_pages * 2 * num_kv_heads * page_size, DH, box_rows) != 0) return -12;
+  const long long page_rows = (long long)num_kv_heads * page_size, page_bytes = page_rows * (DH + DV) * 2;
+  if (!make(&map_q, q, DH, num_q_heads, num_tokens, (long long)num_q_heads * DH * 2, group, BM / group) ||
+      !make(&map_out, out, DV, num_q_heads, num_tokens, (long long)num_q_heads * DV * 2, group, BM / group) ||
+      !make(&map_k, cache, DH, page_rows, num_pages, page_bytes, box_rows, 1) ||
+      !make(&map_v, (const bf16*)cache + page_rows * DH, DV, page_rows, num_pages, page_bytes, box_rows, 1))
+    return -12;
   TcParams p{};
   p.q = (const bf16*)q;
   p.block_table = block_table; p.max_pages = max_pages; p.cu_q = cu_q; p.q_start = q_start; p.out = (bf16*)out;
@@ -625,7 +643,7 @@ static int prefill_tc_launch(const void* q, const void* cache, const int* block_
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  sb_launch(attn_prefill_tc_kernel, dim3(num_items), TC_THREADS, TC_SMEM + table_bytes, stream, p, map_q, map_kv, map_out);
+  sb_launch(attn_prefill_tc_kernel, dim3(num_items), TC_THREADS, TC_SMEM + table_bytes, stream, p, map_q, map_k, map_v, map_out);
   SB_LAUNCH_CHECK();
   return 0;
 }
@@ -648,5 +666,3 @@ extern "C" int SB_FN(sb_attn_prefill_tc_biased)(const void* q, const void* cache
   return prefill_tc_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_tokens, num_q_heads, num_kv_heads,
                            page_size, num_pages, cap, window, distance, linear, sink, key_chunk, items, num_items, err, stream);
 }
-
-#endif  // head sizes that are no multiple of 64 do not get this kernel

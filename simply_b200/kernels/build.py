@@ -38,7 +38,7 @@ class KernelBuildError(RuntimeError):
 # Sources that are compiled once per head size (-DSB_HEAD_DIM=N) into libraries of their own.
 PER_HEAD_DIM = ("attention_mma.cu", "attention_tc.cu", "attention_tc_pair.cu")
 # ... and those of them that also take value heads of another size (-DSB_VALUE_DIM=M).
-PER_TWO_SIZES = ("attention_mma.cu",)
+PER_TWO_SIZES = ("attention_mma.cu", "attention_tc.cu")
 
 
 # Compiled once per shape of a cache of latents (-DSB_LATENT_KD=N -DSB_LATENT_VD=M).
@@ -107,7 +107,7 @@ def attention_lib_name(head_dim: int, value_dim: int | None = None) -> str:
 
 def build_attention(head_dim: int, verbose: bool = True, force: bool = False, value_dim: int | None = None) -> str:
   """Compiles the tensor-core attention kernels for one head size (or for key and value heads of two
-  sizes: then the mma.sync kernels alone); returns the library's path."""
+  sizes: then without the kernel by pairs of blocks); returns the library's path."""
   for size in (head_dim, head_dim if value_dim is None else value_dim):
     if size % 16 or not 16 <= size <= 256:
       raise KernelBuildError(f"tensor-core attention takes head sizes 16, 32, ..., 256; got {size}")

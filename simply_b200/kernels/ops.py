@@ -174,7 +174,8 @@ class CudaOps:
     # 0: prefill tiles of 64 query rows; 64 or 128 forces a size.
     self.prefill_rows = 0
     # Prefill attention on the tcgen05 tensor cores where the shapes allow (head size a multiple of
-    # 64, group dividing 128, page size a power of two); False keeps the mma.sync kernel.
+    # 64, or of 16 where value heads have another size or an option beside the window is in use; group
+    # dividing 128, page size a power of two); False keeps the mma.sync kernel.
     self.prefill_tcgen05 = True
     # ... and there by pairs of blocks (cta_group::2) where the shapes allow (head size 128 or 256,
     # pages of at least 64 tokens); False keeps single blocks (tests).
@@ -450,15 +451,13 @@ class CudaOps:
       make_map = getattr(lib, f"sb_attn_tensor_map_{suffix}")
       make_map.argtypes = [c_void, c_void, ctypes.c_longlong, c_int]
       make_map.restype = c_int
-      prefill_tc = prefill_tc_biased = None
-      if head_dim % 64 == 0 and value_dim == head_dim:
-        prefill_tc = getattr(lib, f"sb_attn_prefill_tc_{suffix}")
-        prefill_tc.argtypes = [c_void, c_void, c_void, c_int, c_void, c_void, c_void, c_int, c_int, c_int, c_int,
-                               c_int, c_float, c_int, c_void, c_int, c_void, c_void]
-        prefill_tc.restype = c_int
-        prefill_tc_biased = getattr(lib, f"sb_attn_prefill_tc_biased_{suffix}")
-        prefill_tc_biased.argtypes = prefill_tc.argtypes[:-2] + [c_void, c_int, c_void, c_int, c_void, c_void]
-        prefill_tc_biased.restype = c_int
+      prefill_tc = getattr(lib, f"sb_attn_prefill_tc_{suffix}")
+      prefill_tc.argtypes = [c_void, c_void, c_void, c_int, c_void, c_void, c_void, c_int, c_int, c_int, c_int,
+                             c_int, c_float, c_int, c_void, c_int, c_void, c_void]
+      prefill_tc.restype = c_int
+      prefill_tc_biased = getattr(lib, f"sb_attn_prefill_tc_biased_{suffix}")
+      prefill_tc_biased.argtypes = prefill_tc.argtypes[:-2] + [c_void, c_int, c_void, c_int, c_void, c_void]
+      prefill_tc_biased.restype = c_int
       prefill_pair = None
       if head_dim in (128, 256) and value_dim == head_dim:
         prefill_pair = getattr(lib, f"sb_attn_prefill_pair_{suffix}")
@@ -472,7 +471,7 @@ class CudaOps:
         raise KernelError(f"sb_attn_decode_resident: {_STATUS.get(slots, slots)}")
       self._decode_slots[(head_dim, value_dim)] = slots
       fns = self._attn_fns[(head_dim, value_dim)] = (prefill, decode, make_map, prefill_tc, prefill_pair, prefill_pooled,
-                                        prefill_biased, prefill_tc_biased)
+                                                              prefill_biased, prefill_tc_biased)
     return fns
 
   def _latent_fn(self, row_dim: int, value_dim: int):
@@ -576,8 +575,9 @@ class CudaOps:
       self._tensor_maps[key] = buf
     return ctypes.c_void_p(buf[1]) if buf[1] is not None else None
 
-  def _prefill_uses_tcgen05(self, head_dim: int, group: int, page_size: int) -> bool:
-    return (self.prefill_tcgen05 and head_dim % 64 == 0 and 128 % group == 0
+  def _prefill_uses_tcgen05(self, head_dim: int, group: int, page_size: int, any_size: bool = False) -> bool:
+    """`any_size`: also head sizes that are no multiple of 64."""
+    return (self.prefill_tcgen05 and (any_size or head_dim % 64 == 0) and 128 % group == 0
             and page_size & (page_size - 1) == 0)
 
   def _prefill_uses_pairs(self, head_dim: int, group: int, page_size: int) -> bool:
@@ -1122,7 +1122,7 @@ class CudaOps:
       # shape (no cap beside them), else the mma.sync tile kernel; not the kernel by pairs.
       options = (_ptr(distance_bias), linear_bias, _ptr(sink), int(key_chunk or 0))
       kind = dict(key_chunk=key_chunk, value_dim=value_dim)
-      use_tc = (prefill_tc is not None and self._prefill_uses_tcgen05(head_dim, group, ctx.page_size)
+      use_tc = (self._prefill_uses_tcgen05(head_dim, group, ctx.page_size, special or value_dim != head_dim)
                 and (not special or not logit_softcap))
       use_pair = (prefill_pair is not None and self._prefill_uses_pairs(head_dim, group, ctx.page_size)
                   and not special)
