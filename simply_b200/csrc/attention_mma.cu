@@ -85,10 +85,12 @@ struct AttnParams {
   int pool_max_pages, pool_len, pool_entries, pool_pages;
 };
 
-// The lowest key that the query at `pos` sees.
+// The lowest key that the query at `pos` sees.  (OPT: the kernel may be given the options beside a window;
+// the split-key kernels for few rows exist without them too, which keeps the usual ones as short as they were.)
+template <bool OPT = true>
 __device__ __forceinline__ int lowest_key(const AttnParams& p, int pos) {
   if (p.window > 0) return max(pos - p.window + 1, 0);
-  return p.key_chunk > 0 ? max(pos, 0) / p.key_chunk * p.key_chunk : 0;
+  return OPT && p.key_chunk > 0 ? max(pos, 0) / p.key_chunk * p.key_chunk : 0;
 }
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
@@ -249,12 +251,14 @@ struct RowBias {
   float r1, r2;
 };
 enum { NO_BIAS = 0, LOG_BIAS = 1, LINEAR_BIAS = 2 };
+template <bool OPT = true>
 __device__ __forceinline__ int bias_kind(const AttnParams& p) {
-  return p.distance == nullptr ? NO_BIAS : (p.linear ? LINEAR_BIAS : LOG_BIAS);
+  return !OPT || p.distance == nullptr ? NO_BIAS : (p.linear ? LINEAR_BIAS : LOG_BIAS);
 }
+template <bool OPT = true>
 __device__ __forceinline__ RowBias row_bias(const AttnParams& p, int head) {
   RowBias b{0.f, 0.f};
-  if (p.distance != nullptr) {
+  if (OPT && p.distance != nullptr) {
     b.r1 = p.distance[head];
     if (!p.linear) {
       b.r1 *= 0.6931471805599453f;
@@ -710,7 +714,7 @@ __device__ __forceinline__ const bf16* tile_at(const bf16* tile, int row, int di
   return tile + row * ROW_PITCH + dim;
 }
 
-template <bool USE_TMA>
+template <bool USE_TMA, bool OPT>
 __global__ void __launch_bounds__(D8_NT)
 attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const __grid_constant__ CUtensorMap tmap,
                     int box_rows) {
@@ -749,7 +753,7 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
     if (b < 0) continue;  // filler item of a fixed-size work list
     const int row0 = p.cu_q[b], q_len = p.cu_q[b + 1] - row0, qs = p.q_start[b];
     const int rows_valid = q_len * group;  // <= 8 by the host's routing
-    const int kv_lo = lowest_key(p, qs);
+    const int kv_lo = lowest_key<OPT>(p, qs);
     const int kv_hi = qs + q_len;
     const int begin = max(chunk_index * p.chunk, (kv_lo / 64) * 64);
     const int end = min((chunk_index + 1) * p.chunk, kv_hi);
@@ -814,10 +818,10 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
     const int pos0 = 2 * t < rows_valid ? qs + (2 * t) / group : -1;
     const int pos1 = 2 * t + 1 < rows_valid ? qs + (2 * t + 1) / group : -1;
     const float inv_cap = p.cap > 0.f ? 1.0f / p.cap : 0.f;
-    const int biased = bias_kind(p);
-    const RowBias bias0 = row_bias(p, m * group + (2 * t) % group);
-    const RowBias bias1 = row_bias(p, m * group + (2 * t + 1) % group);
-    const int lo0 = lowest_key(p, pos0), lo1 = lowest_key(p, pos1);
+    const int biased = bias_kind<OPT>(p);
+    const RowBias bias0 = row_bias<OPT>(p, m * group + (2 * t) % group);
+    const RowBias bias1 = row_bias<OPT>(p, m * group + (2 * t + 1) % group);
+    const int lo0 = lowest_key<OPT>(p, pos0), lo1 = lowest_key<OPT>(p, pos1);
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     float o[DV / 16][4];  // out^T: [dims 16 blk + g | g + 8][rows 2t | 2t + 1]
 #pragma unroll
@@ -1005,6 +1009,7 @@ struct WsItem {
   int b, m, begin, end, kv_lo, n_tiles, qs, q_len, row0;
 };
 
+template <bool OPT>
 __device__ __forceinline__ bool ws_item(const AttnParams& p, int work, WsItem& w) {
   const int item = work / p.num_kv_heads;
   w.m = work - item * p.num_kv_heads;
@@ -1014,7 +1019,7 @@ __device__ __forceinline__ bool ws_item(const AttnParams& p, int work, WsItem& w
   w.row0 = p.cu_q[w.b];
   w.q_len = p.cu_q[w.b + 1] - w.row0;
   w.qs = p.q_start[w.b];
-  w.kv_lo = lowest_key(p, w.qs);
+  w.kv_lo = lowest_key<OPT>(p, w.qs);
   const int kv_hi = w.qs + w.q_len;
   w.begin = max(chunk_index * p.chunk, (w.kv_lo / 64) * 64);
   w.end = min((chunk_index + 1) * p.chunk, kv_hi);
@@ -1026,6 +1031,7 @@ __device__ __forceinline__ void mbar_arrive_one(uint64_t* bar) {
   asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(bar)) : "memory");
 }
 
+template <bool OPT>
 __global__ void __launch_bounds__(WS_NT)
 attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, const __grid_constant__ CUtensorMap tmap,
                       int box_rows) {
@@ -1077,7 +1083,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
       mbar_arrive_one(&work_full[slot]);  // release: the consumers see the slot's content
       if (work >= total_work) return;
       WsItem w;
-      if (!ws_item(p, work, w)) continue;
+      if (!ws_item<OPT>(p, work, w)) continue;
       for (int ti = 0; ti < w.n_tiles; ++ti, ++seq) {
         const int stage = seq % WS_STAGES;
         if (seq >= WS_STAGES && !mbar_wait_bounded(&empty[stage], (seq / WS_STAGES - 1) & 1)) {
@@ -1130,7 +1136,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
     if (lane == 0) mbar_arrive_one(&work_empty[slot]);
     if (work >= total_work) return;
     WsItem w;
-    if (!ws_item(p, work, w)) continue;
+    if (!ws_item<OPT>(p, work, w)) continue;
     const int rows_valid = w.q_len * group;  // <= 8 by the host's routing
     const size_t pidx = (size_t)(work / p.num_kv_heads) * p.num_kv_heads + w.m;
     pdl_wait();  // before the first read of a query and the first write of a result
@@ -1160,10 +1166,10 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
     const int pos0 = 2 * t < rows_valid ? w.qs + (2 * t) / group : -1;
     const int pos1 = 2 * t + 1 < rows_valid ? w.qs + (2 * t + 1) / group : -1;
     const float inv_cap = p.cap > 0.f ? 1.0f / p.cap : 0.f;
-    const int biased = bias_kind(p);
-    const RowBias bias0 = row_bias(p, w.m * group + (2 * t) % group);
-    const RowBias bias1 = row_bias(p, w.m * group + (2 * t + 1) % group);
-    const int lo0 = lowest_key(p, pos0), lo1 = lowest_key(p, pos1);
+    const int biased = bias_kind<OPT>(p);
+    const RowBias bias0 = row_bias<OPT>(p, w.m * group + (2 * t) % group);
+    const RowBias bias1 = row_bias<OPT>(p, w.m * group + (2 * t + 1) % group);
+    const int lo0 = lowest_key<OPT>(p, pos0), lo1 = lowest_key<OPT>(p, pos1);
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     float o[DV / 16][4];
 #pragma unroll
@@ -1310,6 +1316,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
 constexpr int COMBINE_WARPS = 8;
 constexpr int DPL = (DV + 31) / 32;  // output elements per lane
 
+template <bool SINK>
 __global__ void __launch_bounds__(COMBINE_WARPS * 32)
 attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                     const int* __restrict__ token_seq, const int* __restrict__ cu_q,
@@ -1379,7 +1386,7 @@ attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ 
     scale[w] = s_max[w] == -INFINITY ? 0.f : fast_exp2(s_max[w] - mx);
     den += s_den[w] * scale[w];
   }
-  if (sink != nullptr) den += fast_exp2(sink[h] * LOG2E - mx);
+  if constexpr (SINK) den += fast_exp2(sink[h] * LOG2E - mx);
   const float inv = den > 0.f ? 1.0f / den : 0.f;
   bf16* op = out + ((size_t)tkn * num_q_heads + h) * DV;
   for (int d = threadIdx.x; d < DV; d += COMBINE_WARPS * 32) {
@@ -1517,6 +1524,46 @@ extern "C" int SB_FN(sb_attn_prefill_biased)(const void* q, const void* cache, c
                         nullptr, 0, 0, 0, err, stream);
 }
 
+// The split-key kernels for at most 8 query rows per kv head (variant: see the entry point below).
+template <bool OPT>
+static int launch_few_rows(const AttnParams& p, int* work_counter, int total_work, int variant, const void* tensor_map,
+                           cudaStream_t stream) {
+  constexpr size_t ws_merge = (size_t)(D8_WARPS * 8 * DV) * sizeof(float);
+  constexpr bool ws_fits = ws_merge <= (size_t)D8_BN * DH * sizeof(bf16);  // the merge borrows one key tile
+  CUtensorMap map;
+  memset(&map, 0, sizeof(map));
+  if (tensor_map != nullptr) memcpy(&map, tensor_map, sizeof(map));
+  const int box_rows = p.page_size < D8_BN ? p.page_size : D8_BN;
+  if ((variant == 0 || variant == 3) && ws_fits && tensor_map != nullptr) {
+    static int resident_ws = 0;
+    constexpr size_t smem = (size_t)(2 * WS_STAGES * D8_BN) * DH * sizeof(bf16) + 1024;
+    if (resident_ws == 0) {
+      int rc = blocks_resident(attn_decode8ws_kernel<OPT>, WS_NT, smem, &resident_ws);
+      if (rc) return rc;
+    }
+    sb_launch_early(attn_decode8ws_kernel<OPT>, total_work < resident_ws ? total_work : resident_ws, WS_NT, smem, stream,
+        p, work_counter, total_work, map, box_rows);
+  } else if (tensor_map != nullptr && variant != 1) {
+    static int resident_tma = 0;
+    constexpr size_t smem = (DECODE8_SMEM_TMA_KV > DECODE8_SMEM_MERGE ? DECODE8_SMEM_TMA_KV : DECODE8_SMEM_MERGE) + 1024;
+    if (resident_tma == 0) {
+      int rc = blocks_resident(attn_decode8_kernel<true, OPT>, D8_NT, smem, &resident_tma);
+      if (rc) return rc;
+    }
+    sb_launch(attn_decode8_kernel<true, OPT>, total_work < resident_tma ? total_work : resident_tma, D8_NT, smem, stream,
+        p, work_counter, total_work, map, box_rows);
+  } else {
+    static int resident8 = 0;
+    if (resident8 == 0) {
+      int rc = blocks_resident(attn_decode8_kernel<false, OPT>, D8_NT, DECODE8_SMEM, &resident8);
+      if (rc) return rc;
+    }
+    sb_launch(attn_decode8_kernel<false, OPT>, total_work < resident8 ? total_work : resident8, D8_NT, DECODE8_SMEM, stream,
+        p, work_counter, total_work, map, 0);
+  }
+  return 0;
+}
+
 // Split-key attention for sequences with at most 16 query rows per kv head, and the merge.
 // items: [num_items, 2] (sequence or -1, chunk index); chunk: keys per chunk, a multiple of 64;
 // part_o / part_ml: scratch of num_items * Hkv * rows_max * (DV | 2) floats;
@@ -1548,42 +1595,12 @@ extern "C" int SB_FN(sb_attn_decode)(const void* q, const void* cache, const int
   p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk;
   const int total_work = num_items * num_kv_heads;
   const bool power_of_two_pages = (page_size & (page_size - 1)) == 0;
-  constexpr size_t ws_merge = (size_t)(D8_WARPS * 8 * DV) * sizeof(float);
-  constexpr bool ws_fits = ws_merge <= (size_t)D8_BN * DH * sizeof(bf16);  // the merge borrows one key tile
-  if (rows_max <= 8 && (variant == 0 || variant == 3) && TMA_OK && ws_fits && tensor_map != nullptr && power_of_two_pages) {
-    static int resident_ws = 0;
-    constexpr size_t smem = (size_t)(2 * WS_STAGES * D8_BN) * DH * sizeof(bf16) + 1024;
-    if (resident_ws == 0) {
-      int rc = blocks_resident(attn_decode8ws_kernel, WS_NT, smem, &resident_ws);
-      if (rc) return rc;
-    }
-    CUtensorMap map;
-    memcpy(&map, tensor_map, sizeof(map));
-    const int box_rows = page_size < D8_BN ? page_size : D8_BN;
-    sb_launch_early(attn_decode8ws_kernel, total_work < resident_ws ? total_work : resident_ws, WS_NT, smem, stream,
-        p, work_counter, total_work, map, box_rows);
-  } else if (rows_max <= 8 && variant != 16 && TMA_OK && tensor_map != nullptr && power_of_two_pages && variant != 1) {
-    static int resident_tma = 0;
-    constexpr size_t smem = (DECODE8_SMEM_TMA_KV > DECODE8_SMEM_MERGE ? DECODE8_SMEM_TMA_KV : DECODE8_SMEM_MERGE) + 1024;
-    if (resident_tma == 0) {
-      int rc = blocks_resident(attn_decode8_kernel<true>, D8_NT, smem, &resident_tma);
-      if (rc) return rc;
-    }
-    CUtensorMap map;
-    memcpy(&map, tensor_map, sizeof(map));
-    const int box_rows = page_size < D8_BN ? page_size : D8_BN;
-    sb_launch(attn_decode8_kernel<true>, total_work < resident_tma ? total_work : resident_tma, D8_NT, smem, stream,
-        p, work_counter, total_work, map, box_rows);
-  } else if (rows_max <= 8 && variant != 16) {
-    static int resident8 = 0;
-    if (resident8 == 0) {
-      int rc = blocks_resident(attn_decode8_kernel<false>, D8_NT, DECODE8_SMEM, &resident8);
-      if (rc) return rc;
-    }
-    CUtensorMap map;
-    memset(&map, 0, sizeof(map));
-    sb_launch(attn_decode8_kernel<false>, total_work < resident8 ? total_work : resident8, D8_NT, DECODE8_SMEM, stream,
-        p, work_counter, total_work, map, 0);
+  const bool opt = distance != nullptr || key_chunk > 0;
+  const bool with_map = TMA_OK && tensor_map != nullptr && power_of_two_pages;
+  if (rows_max <= 8 && variant != 16) {
+    const int rc = opt ? launch_few_rows<true>(p, work_counter, total_work, variant, with_map ? tensor_map : nullptr, stream)
+                       : launch_few_rows<false>(p, work_counter, total_work, variant, with_map ? tensor_map : nullptr, stream);
+    if (rc) return rc;
   } else {
     static int resident = 0;  // blocks of this kernel the device holds at once
     if (resident == 0) {
@@ -1594,9 +1611,13 @@ extern "C" int SB_FN(sb_attn_decode)(const void* q, const void* cache, const int
         p, work_counter, total_work);
   }
   SB_LAUNCH_CHECK();
-  sb_launch_early(attn_combine_kernel, (unsigned)(num_tokens * num_q_heads), COMBINE_WARPS * 32, 0, stream,
-      part_o, part_ml, token_seq, cu_q, split_start, split_count, (bf16*)out, sink, num_q_heads, num_kv_heads,
-      rows_max, work_counter);
+  const unsigned rows = (unsigned)(num_tokens * num_q_heads);
+  if (sink != nullptr)
+    sb_launch_early(attn_combine_kernel<true>, rows, COMBINE_WARPS * 32, 0, stream, part_o, part_ml, token_seq, cu_q, split_start,
+        split_count, (bf16*)out, sink, num_q_heads, num_kv_heads, rows_max, work_counter);
+  else
+    sb_launch_early(attn_combine_kernel<false>, rows, COMBINE_WARPS * 32, 0, stream, part_o, part_ml, token_seq, cu_q, split_start,
+        split_count, (bf16*)out, sink, num_q_heads, num_kv_heads, rows_max, work_counter);
   SB_LAUNCH_CHECK();
   return 0;
 }
@@ -1610,9 +1631,9 @@ extern "C" int SB_FN(sb_attn_decode_resident)(int with_tensor_map) {
   constexpr bool ws_fits = ws_merge <= (size_t)D8_BN * DH * sizeof(bf16);
   if (with_tensor_map && TMA_OK && ws_fits) {
     constexpr size_t smem = (size_t)(2 * WS_STAGES * D8_BN) * DH * sizeof(bf16) + 1024;
-    rc = blocks_resident(attn_decode8ws_kernel, WS_NT, smem, &resident);
+    rc = blocks_resident(attn_decode8ws_kernel<false>, WS_NT, smem, &resident);
   } else {
-    rc = blocks_resident(attn_decode8_kernel<false>, D8_NT, DECODE8_SMEM, &resident);
+    rc = blocks_resident(attn_decode8_kernel<false, true>, D8_NT, DECODE8_SMEM, &resident);
   }
   return rc ? (rc > 0 ? -rc : rc) : resident;
 }

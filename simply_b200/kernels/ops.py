@@ -647,7 +647,8 @@ class CudaOps:
     for b in np.nonzero(~small)[0]:
       for i0 in range(0, int(q_len[b]), tokens_per_tile):
         last = int(q_start[b]) + min(i0 + tokens_per_tile, int(q_len[b]))
-        first = int(self.lowest_keys(q_start[b] + i0, window, key_chunk))
+        at = int(q_start[b]) + i0
+        first = max(at - window + 1, 0) if window else at // key_chunk * key_chunk if key_chunk else 0
         pre.append((last - first, int(b), i0))
     pre.sort(key=lambda x: -x[0])
     if force_rows in (128, 256):
@@ -1120,7 +1121,7 @@ class CudaOps:
       prefill, decode, _, prefill_tc, prefill_pair = fns[:5]
       # A distance bias, a sink or chunks of keys: the tcgen05 kernel by single blocks where it takes the
       # shape (no cap beside them), else the mma.sync tile kernel; not the kernel by pairs.
-      options = (_ptr(distance_bias), linear_bias, _ptr(sink), int(key_chunk or 0))
+      options = (_ptr(distance_bias), linear_bias, _ptr(sink), int(key_chunk or 0)) if special else (None, 0, None, 0)
       kind = dict(key_chunk=key_chunk, value_dim=value_dim)
       use_tc = (self._prefill_uses_tcgen05(head_dim, group, ctx.page_size, special or value_dim != head_dim)
                 and (not special or not logit_softcap))
