@@ -58,8 +58,10 @@ class PageGroup:
     self.pool = PagePool(num_pages)
     self.max_pages_per_seq = _cdiv(max_seq_len, page_size)
     self.tables = np.full((max_slots, self.max_pages_per_seq), -1, dtype=np.int32)
-    # Pages [first_page, end_page) of a slot are held.
-    self.first_page = np.zeros(max_slots, dtype=np.int64)
+    # Pages [first_page, end_page) of a slot are held, and beside them its first `kept` pages, which
+    # the window's rule does not touch (first_page starts behind them).
+    self.kept = need.kept_pages(page_size)
+    self.first_page = np.full(max_slots, self.kept, dtype=np.int64)
     self.end_page = np.zeros(max_slots, dtype=np.int64)
     self.cache_names: list[str] = []
     self.version = 0  # counts changes of `tables`: who holds a copy can tell whether it is current
@@ -67,8 +69,8 @@ class PageGroup:
   def plan(self, slot: int, cur_len: int, n_new: int) -> tuple[int, int]:
     """(pages to give back, pages to take) for `n_new` tokens after `cur_len` cached ones."""
     first, end = int(self.first_page[slot]), int(self.end_page[slot])
-    new_first = max(first, self.need.first_needed_page_of(cur_len, self.page_size))
-    new_first = min(new_first, end)
+    # (never below `first`, which lies beyond `end` while a request is shorter than what it always keeps)
+    new_first = max(first, min(self.need.first_needed_page_of(cur_len, self.page_size), end))
     new_end = max(end, _cdiv(cur_len + n_new, self.page_size))
     return new_first - first, new_end - end
 
@@ -90,17 +92,17 @@ class PageGroup:
     return back, taken
 
   def release_slot(self, slot: int) -> list[int]:
-    first, end = int(self.first_page[slot]), int(self.end_page[slot])
-    back = [int(p) for p in self.tables[slot, first:end]]
+    back = self.held_pages(slot)
     self.pool.give_back(back)
     self.version += 1
     self.tables[slot, :] = -1
-    self.first_page[slot] = 0
+    self.first_page[slot] = self.kept
     self.end_page[slot] = 0
     return back
 
   def held_pages(self, slot: int) -> list[int]:
-    return [int(p) for p in self.tables[slot, int(self.first_page[slot]):int(self.end_page[slot])]]
+    first, end = int(self.first_page[slot]), int(self.end_page[slot])
+    return [int(p) for p in self.tables[slot, :min(self.kept, end)]] + [int(p) for p in self.tables[slot, first:end]]
 
 
 @dataclasses.dataclass
@@ -339,7 +341,7 @@ class CacheManager:
     for g in self.groups:
       # `PageGroup.plan` for all of them at once.
       first, end = g.first_page[slots], g.end_page[slots]
-      new_first = np.minimum(np.maximum(first, g.need.first_needed_page(cur, self.page_size)), end)
+      new_first = np.maximum(first, np.minimum(g.need.first_needed_page(cur, self.page_size), end))
       new_end = np.maximum(end, -(-(cur + new) // self.page_size))
       back = int((new_first - first).sum()) + sum(n for _, n in self._idle_releasable(g, busy))
       take = int((new_end - end).sum())
@@ -430,7 +432,8 @@ class CacheManager:
         if any(p < 0 for p in pages):
           raise AssertionError(f"slot {slot} holds an invalid page id in {pages}")
         row = g.tables[slot]
-        outside = np.concatenate([row[:int(g.first_page[slot])], row[int(g.end_page[slot]):]])
+        outside = np.concatenate([row[min(g.kept, int(g.end_page[slot])):int(g.first_page[slot])],
+                                  row[int(g.end_page[slot]):]])
         if (outside != -1).any():
           raise AssertionError(f"slot {slot} has page ids outside its held range")
         if self.owner[slot] is not None:
@@ -441,7 +444,7 @@ class CacheManager:
           if length > 0:
             # Everything the request's next query can see must still be held.
             needed = int(g.need.first_needed_page(np.array([length]), self.page_size)[0])
-            if int(g.first_page[slot]) > needed:
+            if int(g.first_page[slot]) > max(needed, g.kept):
               raise AssertionError(f"slot {slot}: pages that are still visible were given back")
         held.extend(pages)
       free = g.pool.free_pages()

@@ -10,7 +10,8 @@ counterpart of the second (its per-request rows hold tokens and positions only,
 
 Caches whose needs have the same `group_key()` share one pool of page ids and one block table
 per request; the need itself says which of a request's pages may be given back
-(`first_needed_page`) and how large its group's pool has to be (`pool_pages`).  A mixer with
+(`first_needed_page`) and how large its group's pool has to be (`pool_pages`), and which of its first pages stay whatever
+the window (`kept_pages`).  A mixer with
 another rule (a dilated window, a pool of its own) subclasses `PagedKVNeed` and overrides these;
 the cache manager calls them and knows no rule of its own.
 """
@@ -44,6 +45,9 @@ class PagedKVNeed:
   # True: an entry has one row of head_dim numbers, whose first value_dim are its value as well
   # (a cache of latents that are key and value at once); a page then holds key rows only.
   values_in_keys: bool = False
+  # With a window: the request's first `keep_first` tokens stay visible to every query, so their
+  # pages are never given back while the request lives.
+  keep_first: int = 0
 
   @property
   def v_dim(self) -> int:
@@ -64,7 +68,13 @@ class PagedKVNeed:
 
   def group_key(self) -> tuple:
     """Needs with equal keys share page ids: the same pages are held, and given back together."""
+    if self.window is not None and self.keep_first > 0:
+      return ("window", self.window, "first", self.keep_first)
     return ("window", self.window)
+
+  def kept_pages(self, page_size: int) -> int:
+    """A request's first pages that are never given back although the window has left them."""
+    return 0 if self.window is None else -(-self.keep_first // page_size)
 
   def first_needed_page(self, lengths: np.ndarray, page_size: int) -> np.ndarray:
     """Per request, the first page that the query after `lengths` cached tokens can still see;
@@ -97,7 +107,8 @@ class PagedKVNeed:
     """True if a cache with this need still holds, at every length, all that `reader` can see."""
     if self.window is None:
       return True
-    return type(reader) is PagedKVNeed and reader.window is not None and reader.window <= self.window
+    return (type(reader) is PagedKVNeed and reader.window is not None and reader.window <= self.window
+            and reader.keep_first <= self.keep_first)
 
   def pool_pages(self, *, page_size: int, max_slots: int, max_seq_len: int, all_pages: int,
                  step_tokens: int, burst_tokens: int) -> int:
@@ -109,7 +120,7 @@ class PagedKVNeed:
     (simply/serving/page_server.py:175-196, simply/utils/ragged_paged_attention.py:95-110, :418-434)."""
     if self.window is None:
       return all_pages
-    per_slot = -(-(self.window - 1 + max(burst_tokens, 1)) // page_size) + 2
+    per_slot = -(-(self.window - 1 + max(burst_tokens, 1)) // page_size) + 2 + self.kept_pages(page_size)
     per_slot = min(per_slot, -(-max_seq_len // page_size))
     return min(all_pages, max_slots * per_slot + -(-step_tokens // page_size))
 

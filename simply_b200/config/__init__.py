@@ -11,6 +11,7 @@ from simply_b200.config.gemma2 import ConfigError, Gemma2Config
 from simply_b200.config.generax import GeneraxConfig
 from simply_b200.config.mononex import MononexConfig
 from simply_b200.config.nulezen import NulezenConfig
+from simply_b200.config.pibulix import PibulixConfig
 from simply_b200.config.sapivik import SapivikConfig
 from simply_b200.config.zesapel import ZesapelConfig
 from simply_b200.config.model_spec import LayerCall, LayerSpec, ModelSpec, PartSpec
@@ -64,6 +65,6 @@ def preset(name: str):
 
 __all__ = [
     "ConfigError", "EngineConfig", "Gemma2Config", "GeneraxConfig", "LayerCall", "LayerSpec", "ModelSpec", "MononexConfig",
-    "NulezenConfig", "PartSpec", "SapivikConfig", "ZesapelConfig", "config_from_dict", "load_config", "preset", "preset_dict", "preset_names",
-    "read_config_json",
+    "NulezenConfig", "PartSpec", "PibulixConfig", "SapivikConfig", "ZesapelConfig", "config_from_dict", "load_config", "preset",
+    "preset_dict", "preset_names", "read_config_json",
 ]

@@ -22,7 +22,8 @@
 // denominator; it has no key and no value.  `distance`: two learned numbers r1, r2 per query head
 // ([2, heads]); the score of query i and key j loses r1 * log(1 + r2 * (i - j)) (float32, log1pf);
 // with `linear` one number r1 per head ([heads]), and the score loses r1 * (i - j).  `chunk` C (without
-// a window): a query sees the keys from (i / C) * C on, its own chunk's.
+// a window): a query sees the keys from (i / C) * C on, its own chunk's.  `keep` n (with a window): the sequence's
+// first n keys stay visible too.
 //
 // This is the true 32-bit path's attention and the fallback of the bfloat16
 // path for shapes its tensor-core kernels refuse.
@@ -124,7 +125,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ ca
                                const T* __restrict__ pool, const int* __restrict__ pool_table,
                                int pool_max_pages, int pool_len, int pool_pages, int tied,
                                const float* __restrict__ sink, const float* __restrict__ distance, int linear,
-                               int chunk, int* err) {
+                               int chunk, int keep, int* err) {
   const float r1 = distance != nullptr ? distance[blockIdx.x % num_q_heads] : 0.f;  // (weights: before the wait)
   const float r2 = distance != nullptr && !linear ? distance[num_q_heads + blockIdx.x % num_q_heads] : 0.f;
   pdl_wait_block();
@@ -174,12 +175,15 @@ paged_attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ ca
 
   const size_t page_stride = (size_t)num_kv_heads * page_size * (tied ? head_dim : head_dim + v_dim);
   const size_t value_base = (size_t)num_kv_heads * page_size * head_dim;
-  for (int tile = (lo / 32) * 32; tile <= pos; tile += 32) {
+  // Tiles of kept first keys, then the tiles from the one that holds the lowest other key on.
+  const int tile_lo = (lo / 32) * 32;
+  for (int tile = keep > 0 ? 0 : tile_lo; tile <= pos; tile += 32) {
+    if (tile < tile_lo && tile >= keep) tile = tile_lo;
     if (((tile >> 5) & (GEN_WARPS - 1)) != warp) continue;  // by the tile's absolute number
     const int j = tile + lane;
     const T* kr = nullptr;
     const T* vr = nullptr;
-    if (j >= lo && j <= pos) {
+    if ((j >= lo || j < keep) && j <= pos) {
       const long long page = block_table[(size_t)b * max_pages + j / page_size];
       if (page < 0 || page >= num_pages) {
         atomicOr(err, SB_ERR_BAD_PAGE);
@@ -234,10 +238,11 @@ extern "C" int sb_paged_attention_general(const void* q, int dtype, const void* 
                                           int window, const void* pool, const int* pool_table,
                                           int pool_max_pages, int pool_len, int pool_pages, int tied,
                                           const float* sink, const float* distance, int linear, int chunk,
-                                          int* err, cudaStream_t stream) {
+                                          int keep, int* err, cudaStream_t stream) {
   if (num_tokens == 0) return 0;
   if (distance != nullptr && pool != nullptr) return -13;
   if (chunk > 0 && (pool != nullptr || window > 0)) return -13;
+  if (keep < 0 || (keep > 0 && (window <= 0 || pool != nullptr || tied))) return -13;
   if (tied && (pool != nullptr || v_dim > head_dim)) return -13;
   // (the values' sums live in registers, GEN_MAX_DPL per lane; a key row only passes through)
   if (head_dim <= 0 || head_dim > 4096 || v_dim <= 0 || v_dim > 32 * GEN_MAX_DPL) return -7;
@@ -250,12 +255,12 @@ extern "C" int sb_paged_attention_general(const void* q, int dtype, const void* 
     sb_launch(paged_attention_generic_kernel<float>, blocks, GEN_WARPS * 32, smem, stream, (const float*)q,
         (const float*)cache, block_table, max_pages, token_seq, positions, (float*)out, num_tokens,
         num_q_heads, num_kv_heads, head_dim, v_dim, page_size, num_pages, cap, window, (const float*)pool, pool_table,
-        pool_max_pages, pool_len, pool_pages, tied, sink, distance, linear, chunk, err);
+        pool_max_pages, pool_len, pool_pages, tied, sink, distance, linear, chunk, keep, err);
   else
     sb_launch(paged_attention_generic_kernel<bf16>, blocks, GEN_WARPS * 32, smem, stream, (const bf16*)q,
         (const bf16*)cache, block_table, max_pages, token_seq, positions, (bf16*)out, num_tokens,
         num_q_heads, num_kv_heads, head_dim, v_dim, page_size, num_pages, cap, window, (const bf16*)pool, pool_table,
-        pool_max_pages, pool_len, pool_pages, tied, sink, distance, linear, chunk, err);
+        pool_max_pages, pool_len, pool_pages, tied, sink, distance, linear, chunk, keep, err);
   SB_LAUNCH_CHECK();
   return 0;
 }
@@ -267,5 +272,5 @@ extern "C" int sb_paged_attention_generic(const void* q, int dtype, const void* 
                                           int* err, cudaStream_t stream) {
   return sb_paged_attention_general(q, dtype, cache, block_table, max_pages, token_seq, positions, out, num_tokens,
                                     num_q_heads, num_kv_heads, head_dim, head_dim, page_size, num_pages, cap,
-                                    window, nullptr, nullptr, 0, 0, 0, 0, nullptr, nullptr, 0, 0, err, stream);
+                                    window, nullptr, nullptr, 0, 0, 0, 0, nullptr, nullptr, 0, 0, 0, err, stream);
 }

@@ -11,7 +11,8 @@
 //
 // Options: a distance term is taken off the scores (r1 log(1 + r2 d), or r1 d); in place of a window,
 // chunks of C keys counted from position 0, of which a query sees its own; a number per head (a sink)
-// whose exponential joins the softmax's denominator.
+// whose exponential joins the softmax's denominator; with a window, a sequence's first keys that stay visible
+// when the window has left them (their tiles come ahead of the window's, what lies between is skipped).
 //
 // Two kernels share the tile code.
 //  * prefill: a block owns 64 query rows of one (sequence, kv head): the G query heads
@@ -71,6 +72,8 @@ struct AttnParams {
   int linear;
   int key_chunk;      // > 0 (without a window): position i sees the keys from (i / C) * C on
   const float* sink;  // optional, float32 [Hq]: exp(sink) joins the denominator
+  int keep_first;     // with a window: keys 0 .. keep_first - 1 stay visible
+  int exact_cap;      // the cap's tanh to float32 accuracy (tanh.approx has 11 bits)
   const int* items;  // prefill: (sequence, first token of the tile); decode: (sequence, chunk)
   int chunk;         // decode: keys per chunk (a multiple of BN)
   float* part_o;     // decode: [items, Hkv, rows_max, DV]
@@ -132,13 +135,17 @@ __device__ __forceinline__ float fast_tanh(float x) {
   asm("tanh.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
+// tanh z = 1 - 2 / (e^(2 z) + 1): its absolute error stays at a few 2^-24
+__device__ __forceinline__ float tanh_by_exp(float x) {
+  return 1.0f - __fdividef(2.0f, fast_exp2(x * (2.0f * LOG2E)) + 1.0f);
+}
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<const uint32_t*>(&v);
 }
 
 // Brings keys [tile, tile + TILE) of (sequence b, kv head m) to shared memory; positions
-// outside [kv_lo, kv_hi) and pages the request does not hold are zero-filled.  The block
+// outside [kv_lo, kv_hi) (kept first keys apart) and pages the request does not hold are zero-filled.  The block
 // first works out where each of the TILE rows lives (one block-table lookup per row, into
 // `row_src`, TILE entries of shared memory), then copies 16 bytes per thread and turn.
 // Ends with the copies issued, not committed.  Contains one __syncthreads.
@@ -149,7 +156,7 @@ __device__ __forceinline__ void load_kv_tile(const AttnParams& p, bf16* sk, bf16
   for (int row = threadIdx.x; row < TILE; row += THREADS) {
     const int j = tile + row;
     long long src = -1, vsrc = -1;
-    if (j >= kv_lo && j < kv_hi) {
+    if ((j >= kv_lo || j < p.keep_first) && j < kv_hi) {
       const int page_index = j / p.page_size;
       const long long page = p.block_table[(size_t)b * p.max_pages + page_index];
       if (page < 0 || page >= p.num_pages) {
@@ -273,13 +280,23 @@ __device__ __forceinline__ float distance_loss(const RowBias& b, int d, int kind
   return b.r1 * (kind == LINEAR_BIAS ? x : __log2f(fmaf(b.r2, x, 1.0f)));
 }
 
+// The cap on a warp's scores to float32 accuracy, ahead of `softmax_pv` (which then gets no cap).
+template <int NKT>
+__device__ __forceinline__ void exact_caps(float (&s)[NKT][4], float cap) {
+  const float inv_cap = 1.0f / cap;
+#pragma unroll
+  for (int i = 0; i < NKT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[i][e] = cap * tanh_by_exp(s[i][e] * inv_cap);
+}
+
 template <int NKT>
 __device__ __forceinline__ void softmax_pv(float (&s)[NKT][4], float (&o)[DV / 8][4], float& m_a, float& m_b,
                                            float& l_a, float& l_b, int pos_a, int pos_b, int lo_a, int lo_b, int j0,
                                            float cap, int window, const bf16* sv, int key0, bool need_mask = true,
                                            int pool_len = 0, int biased = NO_BIAS, RowBias bias_a = RowBias{0.f, 0.f},
-                                           RowBias bias_b = RowBias{0.f, 0.f}) {
-  // lo_a, lo_b: the lowest keys the two rows see.  pool_len > 0: the keys are block entries j0, j0 + 1, ...; a row at `pos` sees the blocks that
+                                           RowBias bias_b = RowBias{0.f, 0.f}, int keep_first = 0) {
+  // lo_a, lo_b: the lowest keys the two rows see (beside the first `keep_first`).  pool_len > 0: the keys are block entries j0, j0 + 1, ...; a row at `pos` sees the blocks that
   // lie wholly before its window, j < (pos - window + 1) / pool_len.
   const int lane = threadIdx.x & 31, t = lane & 3;
   const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f;
@@ -295,7 +312,7 @@ __device__ __forceinline__ void softmax_pv(float (&s)[NKT][4], float (&o)[DV / 8
       if (biased) v -= distance_loss(e < 2 ? bias_a : bias_b, pos - j, biased);
       // need_mask is false (for the whole warp) when every key of the tile is visible to every row.
       const bool keep = pool_len > 0 ? (pos - window + 1 > 0 && j < (pos - window + 1) / pool_len)
-                                     : (!need_mask || (j <= pos && j >= (e < 2 ? lo_a : lo_b)));
+                                     : (!need_mask || (j <= pos && (j >= (e < 2 ? lo_a : lo_b) || j < keep_first)));
       v = keep ? v * LOG2E : -INFINITY;
       s[i][e] = v;
       if (e < 2) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
@@ -383,7 +400,9 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
   const int lo = lowest_key(p, p0);     // lowest key this tile can see
   const int kv_hi = p1 + 1;
   const int tile0 = (lo / BN) * BN;
-  const int n_tiles = (kv_hi - tile0 + BN - 1) / BN;
+  const int n_kept = (min(p.keep_first, tile0) + BN - 1) / BN;  // tiles of kept first keys ahead of the window's
+  const int n_tiles = n_kept + (kv_hi - tile0 + BN - 1) / BN;
+  auto tile_start = [&](int it) { return it < n_kept ? it * BN : tile0 + (it - n_kept) * BN; };
   // Block entries that the tile's last row sees come first, in tiles of their own.
   const int n_blocks = (p.pool != nullptr && p.window > 0 && p1 - p.window + 1 > 0) ? (p1 - p.window + 1) / p.pool_len : 0;
   const int n_pool_tiles = (n_blocks + BN - 1) / BN;
@@ -392,7 +411,7 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
       load_pool_tile<BN, THREADS>(p, sk + stage * BN * PITCH, sv + stage * BN * VPITCH, row_src[stage], it * BN, n_blocks, b, m);
     else
       load_kv_tile<BN, THREADS>(p, sk + stage * BN * PITCH, sv + stage * BN * VPITCH, row_src[stage],
-                                tile0 + (it - n_pool_tiles) * BN, kv_lo, kv_hi, b, m);
+                                tile_start(it - n_pool_tiles), kv_lo, kv_hi, b, m);
   };
   load_tile(0, 0);
   cp_async_commit();
@@ -425,14 +444,16 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
     __syncthreads();
     const bool pooled = it < n_pool_tiles;
     // this warp's first key of the tile (its first block entry, in a tile of those)
-    const int j0 = (pooled ? it * BN : tile0 + (it - n_pool_tiles) * BN) + wn * KEYS;
+    const int j0 = (pooled ? it * BN : tile_start(it - n_pool_tiles)) + wn * KEYS;
     // Every key visible to every row of the warp: below the lowest row's position, inside the
     // highest row's window or chunk.
     const bool need_mask = !rows_full || j0 + KEYS - 1 > warp_pos_lo || j0 < warp_lo;
     float s[KEYS / 8][4];
     scores<KEYS / 8>(s, sq + wm * 16 * PITCH, sk + stage * BN * PITCH, wn * KEYS);
-    softmax_pv<KEYS / 8>(s, o, m_a, m_b, l_a, l_b, pos_a, pos_b, lo_a, lo_b, j0, p.cap, p.window, sv + stage * BN * VPITCH,
-                         wn * KEYS, need_mask, pooled ? p.pool_len : 0, pooled ? NO_BIAS : biased, bias_a, bias_b);
+    if (p.exact_cap) exact_caps<KEYS / 8>(s, p.cap);
+    softmax_pv<KEYS / 8>(s, o, m_a, m_b, l_a, l_b, pos_a, pos_b, lo_a, lo_b, j0, p.exact_cap ? 0.f : p.cap, p.window,
+                         sv + stage * BN * VPITCH, wn * KEYS, need_mask, pooled ? p.pool_len : 0, pooled ? NO_BIAS : biased,
+                         bias_a, bias_b, p.keep_first);
     __syncthreads();
   }
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 1);
@@ -495,6 +516,28 @@ __global__ void __launch_bounds__(WM * WN * 32) attn_prefill_kernel(const AttnPa
   }
 }
 
+// The keys of one work item of the split-key kernels: a chunk's share of the window, and ahead of it (where
+// the chunk holds any below that) the kept first keys.  Tile t of width `BNT` starts at key `tile(t)`.
+template <int BNT, bool OPT>
+struct ItemKeys {
+  int begin, end, start, n_kept, n_tiles;
+  __device__ __forceinline__ ItemKeys(const AttnParams& p, int chunk_index, int kv_lo, int kv_hi) {
+    start = chunk_index * p.chunk;
+    begin = max(start, (kv_lo / 64) * 64);
+    end = min(start + p.chunk, kv_hi);
+    n_kept = 0;
+    if constexpr (OPT) {
+      const int kept_end = min(min(p.keep_first, begin), start + p.chunk);
+      if (kept_end > start) n_kept = (kept_end - start + BNT - 1) / BNT;
+    }
+    n_tiles = n_kept + (end > begin ? (end - begin + BNT - 1) / BNT : 0);
+  }
+  __device__ __forceinline__ int tile(int t) const {
+    if constexpr (OPT) return t < n_kept ? start + t * BNT : begin + (t - n_kept) * BNT;
+    return begin + t * BNT;
+  }
+};
+
 // ---------------------------------------------------------------------------------------
 // Decode: a persistent grid; blocks draw (item, kv head) pairs from a counter until none is
 // left, so short and long chunks balance out.  A block has DEC_BN / 16 warps; warp w owns
@@ -531,9 +574,8 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
     const int rows_valid = q_len * group;  // <= 16 by the host's routing
     const int kv_lo = lowest_key(p, qs);
     const int kv_hi = qs + q_len;
-    const int begin = max(chunk_index * p.chunk, (kv_lo / 64) * 64);
-    const int end = min((chunk_index + 1) * p.chunk, kv_hi);
-    const int n_tiles = end > begin ? (end - begin + DEC_BN - 1) / DEC_BN : 0;
+    const ItemKeys<DEC_BN, true> keys(p, chunk_index, kv_lo, kv_hi);
+    const int end = keys.end, n_tiles = keys.n_tiles;
 
     for (int i = threadIdx.x; i < 16 * CPR; i += DEC_NT) {
       const int row = i / CPR, c = i - row * CPR;
@@ -545,7 +587,7 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
     for (int st = 0; st < DEC_STAGES - 1; ++st) {
       if (st < n_tiles)  // uniform over the block
         load_kv_tile<DEC_BN, DEC_NT>(p, sk + st * DEC_BN * PITCH, sv + st * DEC_BN * VPITCH, row_src[st],
-                                     begin + st * DEC_BN, kv_lo, end, b, m);
+                                     keys.tile(st), kv_lo, end, b, m);
       cp_async_commit();
     }
     const int pos_a = g < rows_valid ? qs + g / group : -1;
@@ -565,13 +607,14 @@ __global__ void __launch_bounds__(DEC_NT) attn_decode_kernel(const AttnParams p,
       if (it + DEC_STAGES - 1 < n_tiles) {
         const int st = (it + DEC_STAGES - 1) % DEC_STAGES;
         load_kv_tile<DEC_BN, DEC_NT>(p, sk + st * DEC_BN * PITCH, sv + st * DEC_BN * VPITCH, row_src[st],
-                                     begin + (it + DEC_STAGES - 1) * DEC_BN, kv_lo, end, b, m);
+                                     keys.tile(it + DEC_STAGES - 1), kv_lo, end, b, m);
       }
       cp_async_commit();
       float s[2][4];
       scores<2>(s, sq, sk + stage * DEC_BN * PITCH, warp * 16);
-      softmax_pv<2>(s, o, m_a, m_b, l_a, l_b, pos_a, pos_b, lo_a, lo_b, begin + it * DEC_BN + warp * 16, p.cap, p.window,
-                    sv + stage * DEC_BN * VPITCH, warp * 16, true, 0, bias_kind(p), bias_a, bias_b);
+      if (p.exact_cap) exact_caps<2>(s, p.cap);
+      softmax_pv<2>(s, o, m_a, m_b, l_a, l_b, pos_a, pos_b, lo_a, lo_b, keys.tile(it) + warp * 16, p.exact_cap ? 0.f : p.cap,
+                    p.window, sv + stage * DEC_BN * VPITCH, warp * 16, true, 0, bias_kind(p), bias_a, bias_b, p.keep_first);
     }
     cp_async_wait<0>();
     __syncthreads();
@@ -755,13 +798,12 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
     const int rows_valid = q_len * group;  // <= 8 by the host's routing
     const int kv_lo = lowest_key<OPT>(p, qs);
     const int kv_hi = qs + q_len;
-    const int begin = max(chunk_index * p.chunk, (kv_lo / 64) * 64);
-    const int end = min((chunk_index + 1) * p.chunk, kv_hi);
-    const int n_tiles = end > begin ? (end - begin + D8_BN - 1) / D8_BN : 0;
+    const ItemKeys<D8_BN, OPT> keys(p, chunk_index, kv_lo, kv_hi);
+    const int end = keys.end, n_tiles = keys.n_tiles;
 
     auto issue_tile = [&](int tile_index, unsigned seq) {
       const int stage = seq % D8_STAGES;
-      const int j0 = begin + tile_index * D8_BN;
+      const int j0 = keys.tile(tile_index);
       if (USE_TMA) {
         // One thread: a box per page piece and 64-column slab, for keys and for values.  Boxes of
         // pages the request does not hold, or wholly outside [kv_lo, end), are not fetched; the
@@ -770,14 +812,14 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
         int boxes = 0;
         for (int r = 0; r < D8_BN; r += box_rows) {
           const int j = j0 + r;
-          if (j >= end || j + box_rows <= kv_lo) continue;
+          if (j >= end || (j + box_rows <= kv_lo && !(OPT && j < p.keep_first))) continue;
           const long long page = p.block_table[(size_t)b * p.max_pages + j / p.page_size];
           if (page >= 0 && page < p.num_pages) ++boxes;
         }
         mbar_arrive_expect_tx(&full[stage], boxes * 2 * SLABS * box_rows * 128);
         for (int r = 0; r < D8_BN; r += box_rows) {
           const int j = j0 + r;
-          if (j >= end || j + box_rows <= kv_lo) continue;
+          if (j >= end || (j + box_rows <= kv_lo && !(OPT && j < p.keep_first))) continue;
           const long long page = p.block_table[(size_t)b * p.max_pages + j / p.page_size];
           if (page < 0 || page >= p.num_pages) {
             atomicOr(p.err, SB_ERR_BAD_PAGE);
@@ -847,14 +889,14 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
         const bf16* kt = sk + (size_t)stage * TILE_ELEMS;
         const bf16* vt = sv + (size_t)stage * VTILE_ELEMS;
         const int key0 = warp * 16;  // this warp's keys of the tile
-        const int j_first = begin + it * D8_BN + key0;
+        const int j_first = keys.tile(it) + key0;
         if (USE_TMA && (j_first < kv_lo || j_first + 16 > end)) {
           // Some of this warp's 16 keys are not the request's: their value rows must read as zeros
           // (0 * garbage could be NaN).  Only this warp reads these rows.
           for (int i = lane; i < 16 * (DV / 8); i += 32) {
             const int r = i / (DV / 8), c = i - r * (DV / 8);
             const int j = j_first + r;
-            if (j < kv_lo || j >= end)
+            if ((j < kv_lo && !(OPT && j < p.keep_first)) || j >= end)
               *reinterpret_cast<uint4*>(const_cast<bf16*>(tile_at<true>(vt, key0 + r, c * 8))) = make_uint4(0, 0, 0, 0);
           }
           asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
@@ -877,11 +919,11 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           float v = s0[e] + s1[e];
-          if (p.cap > 0.f) v = p.cap * fast_tanh(v * inv_cap);
+          if (p.cap > 0.f) v = p.cap * (OPT && p.exact_cap ? tanh_by_exp(v * inv_cap) : fast_tanh(v * inv_cap));
           const int j = j_first + g + (e >> 1) * 8;
           const int pos = (e & 1) ? pos1 : pos0;
           if (biased) v -= distance_loss((e & 1) ? bias1 : bias0, pos - j, biased);
-          const bool keep = j <= pos && j >= ((e & 1) ? lo1 : lo0);
+          const bool keep = j <= pos && (j >= ((e & 1) ? lo1 : lo0) || (OPT && j < p.keep_first));
           sc[e] = keep ? v * LOG2E : -INFINITY;
         }
         float mx0 = fmaxf(sc[0], sc[2]), mx1 = fmaxf(sc[1], sc[3]);
@@ -1006,7 +1048,12 @@ constexpr int WS_RING = 2;
 constexpr int WS_NT = (D8_WARPS + 1) * 32;
 
 struct WsItem {
-  int b, m, begin, end, kv_lo, n_tiles, qs, q_len, row0;
+  int b, m, begin, end, kv_lo, n_tiles, qs, q_len, row0, start, n_kept;
+  template <bool OPT>
+  __device__ __forceinline__ int tile(int t) const {
+    if constexpr (OPT) return t < n_kept ? start + t * D8_BN : begin + (t - n_kept) * D8_BN;
+    return begin + t * D8_BN;
+  }
 };
 
 template <bool OPT>
@@ -1021,9 +1068,12 @@ __device__ __forceinline__ bool ws_item(const AttnParams& p, int work, WsItem& w
   w.qs = p.q_start[w.b];
   w.kv_lo = lowest_key<OPT>(p, w.qs);
   const int kv_hi = w.qs + w.q_len;
-  w.begin = max(chunk_index * p.chunk, (w.kv_lo / 64) * 64);
-  w.end = min((chunk_index + 1) * p.chunk, kv_hi);
-  w.n_tiles = w.end > w.begin ? (w.end - w.begin + D8_BN - 1) / D8_BN : 0;
+  const ItemKeys<D8_BN, OPT> keys(p, chunk_index, w.kv_lo, kv_hi);
+  w.begin = keys.begin;
+  w.end = keys.end;
+  w.start = keys.start;
+  w.n_kept = keys.n_kept;
+  w.n_tiles = keys.n_tiles;
   return true;
 }
 
@@ -1090,7 +1140,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
           atomicOr(p.err, SB_ERR_TIMEOUT);
           return;
         }
-        const int j0 = w.begin + ti * D8_BN;
+        const int j0 = w.tile<OPT>(ti);
         if (!waited && j0 + D8_BN > w.qs) {  // keys from position qs on are written by the step itself
           pdl_wait();
           waited = true;
@@ -1098,14 +1148,14 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
         int boxes = 0;
         for (int r = 0; r < D8_BN; r += box_rows) {
           const int j = j0 + r;
-          if (j >= w.end || j + box_rows <= w.kv_lo) continue;
+          if (j >= w.end || (j + box_rows <= w.kv_lo && !(OPT && j < p.keep_first))) continue;
           const long long page = p.block_table[(size_t)w.b * p.max_pages + j / p.page_size];
           if (page >= 0 && page < p.num_pages) ++boxes;
         }
         mbar_arrive_expect_tx(&full[stage], boxes * 2 * SLABS * box_rows * 128);
         for (int r = 0; r < D8_BN; r += box_rows) {
           const int j = j0 + r;
-          if (j >= w.end || j + box_rows <= w.kv_lo) continue;
+          if (j >= w.end || (j + box_rows <= w.kv_lo && !(OPT && j < p.keep_first))) continue;
           const long long page = p.block_table[(size_t)w.b * p.max_pages + j / p.page_size];
           if (page < 0 || page >= p.num_pages) {
             atomicOr(p.err, SB_ERR_BAD_PAGE);
@@ -1186,13 +1236,13 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
       const bf16* kt = sk + (size_t)stage * TILE_ELEMS;
       const bf16* vt = sv + (size_t)stage * VTILE_ELEMS;
       const int key0 = warp * 16;
-      const int j_first = w.begin + it * D8_BN + key0;
+      const int j_first = w.tile<OPT>(it) + key0;
       if (j_first < w.kv_lo || j_first + 16 > w.end) {
         // Value rows of keys that are not the request's must read as zeros (only this warp reads them).
         for (int i = lane; i < 16 * (DV / 8); i += 32) {
           const int r = i / (DV / 8), c = i - r * (DV / 8);
           const int j = j_first + r;
-          if (j < w.kv_lo || j >= w.end)
+          if ((j < w.kv_lo && !(OPT && j < p.keep_first)) || j >= w.end)
             *reinterpret_cast<uint4*>(const_cast<bf16*>(tile_at<true>(vt, key0 + r, c * 8))) = make_uint4(0, 0, 0, 0);
         }
         __syncwarp();
@@ -1212,11 +1262,11 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         float v = s0[e] + s1[e];
-        if (p.cap > 0.f) v = p.cap * fast_tanh(v * inv_cap);
+        if (p.cap > 0.f) v = p.cap * (OPT && p.exact_cap ? tanh_by_exp(v * inv_cap) : fast_tanh(v * inv_cap));
         const int j = j_first + g + (e >> 1) * 8;
         const int pos = (e & 1) ? pos1 : pos0;
         if (biased) v -= distance_loss((e & 1) ? bias1 : bias0, pos - j, biased);
-        const bool keep = j <= pos && j >= ((e & 1) ? lo1 : lo0);
+        const bool keep = j <= pos && (j >= ((e & 1) ? lo1 : lo0) || (OPT && j < p.keep_first));
         sc[e] = keep ? v * LOG2E : -INFINITY;
       }
       float mx0 = fmaxf(sc[0], sc[2]), mx1 = fmaxf(sc[1], sc[3]);
@@ -1440,7 +1490,7 @@ static int blocks_resident(Kernel kernel, int threads, size_t smem, int* out) {
 static int prefill_launch(const void* q, const void* cache, const int* block_table, int max_pages,
                           const int* cu_q, const int* q_start, void* out, int num_q_heads,
                           int num_kv_heads, int page_size, int num_pages, float cap, int window,
-                          const float* distance, int linear, const float* sink, int key_chunk, const int* items, int num_items, int rows_per_tile, int single_key_group,
+                          const float* distance, int linear, const float* sink, int key_chunk, int keep_first, const int* items, int num_items, int rows_per_tile, int single_key_group,
                           const void* pool, const int* pool_table, int pool_max_pages, int pool_len,
                           int pool_pages, int* err, cudaStream_t stream) {
   if (num_items == 0) return 0;
@@ -1448,7 +1498,9 @@ static int prefill_launch(const void* q, const void* cache, const int* block_tab
   if (pool != nullptr && (pool_len <= 0 || window <= 0 || !ONE_SIZE || sink != nullptr)) return -8;
   if (key_chunk > 0 && window > 0) return -8;
   AttnParams p{};
-  p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk;
+  if (keep_first < 0 || (keep_first > 0 && (window <= 0 || pool != nullptr))) return -8;
+  p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk; p.keep_first = keep_first;
+  p.exact_cap = cap > 0.f && (sink != nullptr || keep_first > 0);
   p.q = (const bf16*)q; p.cache = (const bf16*)cache; p.block_table = block_table; p.max_pages = max_pages;
   p.cu_q = cu_q; p.q_start = q_start; p.out = (bf16*)out; p.num_q_heads = num_q_heads;
   p.num_kv_heads = num_kv_heads; p.page_size = page_size; p.num_pages = num_pages; p.cap = cap;
@@ -1497,7 +1549,7 @@ extern "C" int SB_FN(sb_attn_prefill)(const void* q, const void* cache, const in
                                       const int* items, int num_items, int rows_per_tile, int single_key_group,
                                       int* err, cudaStream_t stream) {
   return prefill_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_q_heads, num_kv_heads, page_size,
-                        num_pages, cap, window, nullptr, 0, nullptr, 0, items, num_items, rows_per_tile, single_key_group, nullptr,
+                        num_pages, cap, window, nullptr, 0, nullptr, 0, 0, items, num_items, rows_per_tile, single_key_group, nullptr,
                         nullptr, 0, 0, 0, err, stream);
 }
 
@@ -1508,19 +1560,19 @@ extern "C" int SB_FN(sb_attn_prefill_pooled)(const void* q, const void* cache, c
                                              const void* pool, const int* pool_table, int pool_max_pages, int pool_len,
                                              int pool_pages, int* err, cudaStream_t stream) {
   return prefill_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_q_heads, num_kv_heads, page_size,
-                        num_pages, cap, window, nullptr, 0, nullptr, 0, items, num_items, rows_per_tile, single_key_group, pool,
+                        num_pages, cap, window, nullptr, 0, nullptr, 0, 0, items, num_items, rows_per_tile, single_key_group, pool,
                         pool_table, pool_max_pages, pool_len, pool_pages, err, stream);
 }
 
-// The same with a distance bias, chunks of keys and a sink (each optional, see AttnParams).
+// The same with a distance bias, chunks of keys, a sink and kept first keys (each optional, see AttnParams).
 extern "C" int SB_FN(sb_attn_prefill_biased)(const void* q, const void* cache, const int* block_table, int max_pages,
                                              const int* cu_q, const int* q_start, void* out, int num_q_heads,
                                              int num_kv_heads, int page_size, int num_pages, float cap, int window,
                                              const int* items, int num_items, int rows_per_tile, int single_key_group,
                                              const float* distance, int linear, const float* sink, int key_chunk,
-                                             int* err, cudaStream_t stream) {
+                                             int keep_first, int* err, cudaStream_t stream) {
   return prefill_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_q_heads, num_kv_heads, page_size,
-                        num_pages, cap, window, distance, linear, sink, key_chunk, items, num_items, rows_per_tile, single_key_group, nullptr,
+                        num_pages, cap, window, distance, linear, sink, key_chunk, keep_first, items, num_items, rows_per_tile, single_key_group, nullptr,
                         nullptr, 0, 0, 0, err, stream);
 }
 
@@ -1579,7 +1631,8 @@ extern "C" int SB_FN(sb_attn_decode)(const void* q, const void* cache, const int
                                      int chunk, float* part_o, float* part_ml, int* work_counter,
                                      int rows_max, const int* split_start, const int* split_count, int variant,
                                      const void* tensor_map, int older_keys_settled, const float* distance,
-                                     int linear, const float* sink, int key_chunk, int* err, cudaStream_t stream) {
+                                     int linear, const float* sink, int key_chunk, int keep_first, int* err,
+                                     cudaStream_t stream) {
   // variant: 0 picks the kernel by rows_max (<= 8: the turned-round kernel, fed by TMA through a
   // producer warp when a tensor map is given and the shapes allow); 1 forbids TMA; 2 uses TMA
   // without the producer warp; 16 forces the 16-row kernel.
@@ -1592,10 +1645,12 @@ extern "C" int SB_FN(sb_attn_decode)(const void* q, const void* cache, const int
   p.num_kv_heads = num_kv_heads; p.page_size = page_size; p.num_pages = num_pages; p.cap = cap;
   p.window = window; p.items = items; p.chunk = chunk; p.part_o = part_o; p.part_ml = part_ml;
   p.rows_max = rows_max; p.older_keys_settled = older_keys_settled; p.err = err;
-  p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk;
+  if (keep_first < 0 || (keep_first > 0 && window <= 0)) return -8;
+  p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk; p.keep_first = keep_first;
+  p.exact_cap = cap > 0.f && (sink != nullptr || keep_first > 0);
   const int total_work = num_items * num_kv_heads;
   const bool power_of_two_pages = (page_size & (page_size - 1)) == 0;
-  const bool opt = distance != nullptr || key_chunk > 0;
+  const bool opt = distance != nullptr || key_chunk > 0 || keep_first > 0 || p.exact_cap;
   const bool with_map = TMA_OK && tensor_map != nullptr && power_of_two_pages;
   if (rows_max <= 8 && variant != 16) {
     const int rc = opt ? launch_few_rows<true>(p, work_counter, total_work, variant, with_map ? tensor_map : nullptr, stream)

@@ -462,6 +462,184 @@ extern "C" int sb_rotate_headnorm_store(const void* proj, int row_width, int dty
 }
 
 // ---------------------------------------------------------------------------
+// Attention whose q, k and v pass a short causal convolution, then (q and k) a norm per head with a
+// scale per channel, then the rotation.  Row of `proj`: q (H d) | k (G d) | v (G dv) | whatever follows.
+//   u_t  = sum_j w[j, c] p_(t - taps + 1 + j, c)    p: the sequence's projected rows; before the step's
+//                                                  first token the state's, zeros before the sequence
+//   x    = u / sqrt(mean_head u^2 + eps) * scale   q and k heads
+//   pair (i, i + rot/2), or neighbours, turned by position * rot_freq[i]; q times q_scale
+// A warp takes one head of a few tokens in a row: what the taps read again is in L1.
+// With `alone` every sequence brings one token, and the warp that has read a channel's state moves it
+// on (of rows that share a slot the first serves all); else a kernel of its own does, after this one.
+// ---------------------------------------------------------------------------
+#define SB_ERR_BAD_SLOT 16
+constexpr int PREP_WARPS = 8;
+
+template <typename T, int TAPS>  // TAPS: 0 none, 2 .. 4, -1 any number
+__global__ void __launch_bounds__(PREP_WARPS * 32)
+conv_headnorm_store_kernel(const T* __restrict__ proj, int row_width, const float* __restrict__ conv_w, int taps_rt,
+                           float* __restrict__ state, const int* __restrict__ slots, int num_slots, int num_seqs, int alone,
+                           const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, float q_scale,
+                           const float* __restrict__ rot_freq, int rot_dims, int interleaved, T* __restrict__ q_out,
+                           T* __restrict__ cache, const int* __restrict__ block_table, int max_pages,
+                           const int* __restrict__ token_seq, const int* __restrict__ cu_q,
+                           const int* __restrict__ positions, int num_tokens, int rows_per_block, int H, int G, int d, int dv,
+                           int page_size, int num_pages, int write_cache, int* err) {
+  pdl_wait_block();
+  pdl_launch_dependents();
+  extern __shared__ float prep_smem[];  // cos and sin of the block's tokens, then a head's row per warp
+  const int half = rot_dims / 2, hd = max(d, dv);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t0 = blockIdx.x * rows_per_block, rows = min(rows_per_block, num_tokens - t0);
+  for (int i = threadIdx.x; i < rows * half; i += blockDim.x) {
+    const int r = i / half, a = i - r * half;
+    sincosf((float)positions[t0 + r] * rot_freq[a], prep_smem + (2 * r + 1) * half + a, prep_smem + 2 * r * half + a);
+  }
+  __syncthreads();
+  const int head = blockIdx.y * PREP_WARPS + warp;
+  if (head >= H + 2 * G) return;
+  float* buf = prep_smem + 2 * rows_per_block * half + (size_t)warp * hd;
+  const int taps = TAPS >= 0 ? TAPS : taps_rt;
+  const bool is_q = head < H, is_v = head >= H + G;
+  const int n = is_v ? dv : d;                                            // channels of this head
+  const int c0 = is_v ? (H + G) * d + (head - H - G) * dv : head * d;     // its first channel
+  const int channels = (H + G) * d + G * dv;
+  const float* scale_w = is_q ? q_norm : k_norm;
+  const size_t page_stride = (size_t)G * page_size * (d + dv);
+
+  for (int r = 0; r < rows; ++r) {
+    const int t = t0 + r, b = token_seq[t];
+    const int i = t - cu_q[b];  // the token's place among the step's tokens of its sequence
+    int copies = 1;
+    float* st = nullptr;
+    if (taps > 1) {
+      const int slot = slots[b];
+      if (slot < 0 || slot >= num_slots) {
+        if (lane == 0) atomicOr(err, SB_ERR_BAD_SLOT);
+        continue;
+      }
+      st = state + (size_t)slot * (taps - 1) * channels + c0;
+      if (alone) {
+        copies = rows_sharing_slot(slots, b, num_seqs);
+        if (copies == 0) continue;  // an earlier row's warp serves this one
+      }
+    }
+    const T* x = proj + (size_t)t * row_width + c0;
+    float ss = 0.f;
+    for (int c = lane; c < n; c += 32) {
+      const float own = to_f32<T>(x[c]);
+      float u = own;
+      if (taps > 0) {
+        const float* w = conv_w + c0 + c;  // [taps][channels]
+        if (alone) {
+          u = 0.f;
+#pragma unroll
+          for (int j = 0; j + 1 < taps; ++j) {
+            const float s = st[(size_t)j * channels + c];
+            u = fmaf(w[(size_t)j * channels], s, u);
+            if (j > 0) st[(size_t)(j - 1) * channels + c] = s;
+          }
+          u = fmaf(w[(size_t)(taps - 1) * channels], own, u);
+          if (taps > 1) st[(size_t)(taps - 2) * channels + c] = own;
+        } else {
+          u = 0.f;
+#pragma unroll
+          for (int j = 0; j < taps; ++j) {
+            const int at = i - (taps - 1) + j;
+            const float p = j == taps - 1 ? own
+                            : at >= 0     ? to_f32<T>(x[c - (long long)(taps - 1 - j) * row_width])
+                                          : st[(size_t)(taps - 1 + at) * channels + c];
+            u = fmaf(w[(size_t)j * channels], p, u);
+          }
+        }
+      }
+      buf[c] = u;
+      ss = fmaf(u, u, ss);
+    }
+    __syncwarp();
+    T* dst = nullptr;
+    if (is_q) {
+      dst = q_out + ((size_t)t * H + head) * d;
+    } else if (write_cache) {
+      const int p = positions[t];
+      const long long page = block_table[(size_t)b * max_pages + p / page_size];
+      if (page < 0 || page >= num_pages) {
+        if (lane == 0) atomicOr(err, SB_ERR_BAD_PAGE);
+      } else if (is_v) {
+        dst = cache + page * page_stride + (size_t)G * page_size * d + ((size_t)(head - H - G) * page_size + p % page_size) * dv;
+      } else {
+        dst = cache + page * page_stride + ((size_t)(head - H) * page_size + p % page_size) * d;
+      }
+    }
+    if (is_v) {
+      if (dst != nullptr)
+        for (int c = lane; c < n; c += 32) dst[c] = from_f32<T>(buf[c]);
+    } else {
+      const float inv = (is_q ? q_scale : 1.0f) / sqrtf(warp_sum(ss) / (float)d + eps);
+      const float* cs = prep_smem + 2 * r * half;
+      if (dst != nullptr) {
+        for (int c = lane; c < n; c += 32) {
+          float v = buf[c] * scale_w[c];
+          if (c < rot_dims) {
+            const int a = interleaved ? c >> 1 : (c < half ? c : c - half);
+            const bool low = interleaved ? (c & 1) == 0 : c < half;
+            const int other = interleaved ? c ^ 1 : (low ? c + half : c - half);
+            const float o = buf[other] * scale_w[other];
+            v = low ? v * cs[a] - o * cs[half + a] : v * cs[a] + o * cs[half + a];
+          }
+          v *= inv;
+          for (int k = 0; k < copies; ++k) dst[(is_q ? (size_t)k * H * d : 0) + c] = from_f32<T>(v);
+        }
+      }
+    }
+    __syncwarp();
+  }
+}
+
+extern "C" int sb_conv_headnorm_store(const void* proj, int row_width, int dtype, const float* conv_w, int taps, float* state,
+                                      const int* slots, int num_slots, int num_seqs, int alone, const float* q_norm,
+                                      const float* k_norm, float eps, float q_scale, const float* rot_freq, int rot_dims,
+                                      int interleaved, void* q_out, void* cache, const int* block_table, int max_pages,
+                                      const int* token_seq, const int* cu_q, const int* positions, int num_tokens, int H,
+                                      int G, int d, int dv, int page_size, int num_pages, int write_cache, int* err,
+                                      cudaStream_t stream) {
+  if (num_tokens == 0) return 0;
+  if (rot_freq == nullptr) rot_dims = 0;
+  if (rot_dims % 2 || rot_dims > d) return -4;
+  if (taps < 0 || (taps > 1 && state == nullptr) || G <= 0 || H % G) return -13;
+  const int rows = num_tokens >= 1024 ? 4 : 1;
+  const dim3 grid((unsigned)((num_tokens + rows - 1) / rows), (unsigned)((H + 2 * G + PREP_WARPS - 1) / PREP_WARPS));
+  const size_t smem = ((size_t)rows * rot_dims + (size_t)PREP_WARPS * (d > dv ? d : dv)) * sizeof(float);
+  if (smem > 200 * 1024 || grid.y > 65535) return -2;
+#define SB_PREP2(T_, TAPS_)                                                                                          \
+  do {                                                                                                               \
+    auto k = conv_headnorm_store_kernel<T_, TAPS_>;                                                                  \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);           \
+    sb_launch(k, grid, PREP_WARPS * 32, smem, stream, (const T_*)proj, row_width, conv_w, taps, state, slots,        \
+              num_slots, num_seqs, alone, q_norm, k_norm, eps, q_scale, rot_freq, rot_dims, interleaved, (T_*)q_out, \
+              (T_*)cache, block_table, max_pages, token_seq, cu_q, positions, num_tokens, rows, H, G, d, dv,         \
+              page_size, num_pages, write_cache, err);                                                               \
+  } while (0)
+#define SB_PREP(T_)                  \
+  switch (taps) {                    \
+    case 0: SB_PREP2(T_, 0); break;  \
+    case 2: SB_PREP2(T_, 2); break;  \
+    case 3: SB_PREP2(T_, 3); break;  \
+    case 4: SB_PREP2(T_, 4); break;  \
+    default: SB_PREP2(T_, -1);       \
+  }
+  if (dtype == SB_DTYPE_F32) {
+    SB_PREP(float)
+  } else {
+    SB_PREP(bf16)
+  }
+#undef SB_PREP
+#undef SB_PREP2
+  SB_LAUNCH_CHECK();
+  return 0;
+}
+
+// ---------------------------------------------------------------------------
 // Output gate: x[t, c] *= sigmoid(gate[t, c]), the gate read from a wider row (a column range of
 // the fused projection).
 // ---------------------------------------------------------------------------

@@ -85,7 +85,9 @@ struct TcParams {
   const float* distance;
   int linear;
   int key_chunk;      // > 0 (without a window): position i sees the keys from (i / C) * C on
-  const float* sink;  // optional, float32 [Hq]: exp(sink) joins the denominator (not together with a cap)
+  const float* sink;  // optional, float32 [Hq]: exp(sink) joins the denominator
+  int keep_first;     // with a window: keys 0 .. keep_first - 1 stay visible (their tiles come ahead of the window's)
+  int exact_cap;      // the cap's tanh to float32 accuracy (tanh.approx has 11 bits)
   // 1: the block first writes the term for every (distance, head of its kv head) into shared memory
   // behind the tiles, [window][group] floats, and the softmax threads read it there
   int bias_table;
@@ -103,6 +105,10 @@ __device__ __forceinline__ float fast_tanh(float x) {
   float y;
   asm("tanh.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
+}
+// tanh z = 1 - 2 / (e^(2 z) + 1): its absolute error stays at a few 2^-24
+__device__ __forceinline__ float tanh_by_exp(float x) {
+  return 1.0f - __fdividef(2.0f, fast_exp2(x * (2.0f * LOG2E)) + 1.0f);
 }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -144,7 +150,9 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
   const int lo = lowest_key(p, p0);     // lowest key this tile can see
   const int kv_hi = p1 + 1;
   const int tile0 = (lo / BN) * BN;
-  const int n_tiles = (kv_hi - tile0 + BN - 1) / BN;
+  const int n_kept = (min(p.keep_first, tile0) + BN - 1) / BN;  // tiles of kept first keys ahead of the window's
+  const int n_tiles = n_kept + (kv_hi - tile0 + BN - 1) / BN;
+  auto tile_start = [&](int j) { return j < n_kept ? j * BN : tile0 + (j - n_kept) * BN; };
 
   if (threadIdx.x == 0) {
     mbar_init(&q_full, 1);
@@ -208,18 +216,18 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
             break;
           }
         }
-        const int j0 = tile0 + j * BN;
+        const int j0 = tile_start(j);
         int boxes = 0;
         for (int r = 0; r < BN; r += p.box_rows) {
           const int key = j0 + r;
-          if (key >= kv_hi || key + p.box_rows <= kv_lo) continue;
+          if (key >= kv_hi || (key + p.box_rows <= kv_lo && key >= p.keep_first)) continue;
           const long long page = p.block_table[(size_t)b * p.max_pages + key / p.page_size];
           if (page >= 0 && page < p.num_pages) ++boxes;
         }
         mbar_arrive_expect_tx(&full[s], boxes * slabs * p.box_rows * 128);
         for (int r = 0; r < BN; r += p.box_rows) {
           const int key = j0 + r;
-          if (key >= kv_hi || key + p.box_rows <= kv_lo) continue;
+          if (key >= kv_hi || (key + p.box_rows <= kv_lo && key >= p.keep_first)) continue;
           const long long page = p.block_table[(size_t)b * p.max_pages + key / p.page_size];
           if (page < 0 || page >= p.num_pages) {
             atomicOr(p.err, SB_ERR_BAD_PAGE);
@@ -327,6 +335,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
     const bool rows_full = quarter * 32 + 31 < rows_valid;
     const int warp_pos_lo = p0 + (quarter * 32) / group, warp_pos_hi = p0 + (quarter * 32 + 31) / group;
     const int row_lo = lowest_key(p, pos), warp_lo = lowest_key(p, warp_pos_hi);  // the lowest keys seen
+    const bool fast_cap = p.cap > 0.f && !p.exact_cap;
     const float inv_cap = p.cap > 0.f ? 1.0f / p.cap : 0.f;
     const float scale2 = p.cap > 0.f ? p.cap * LOG2E : LOG2E;  // from x (tanh's value, or the score) to log2 units
     // The distance bias of this thread's row: r1 ln 2 and r2 of its head.
@@ -358,7 +367,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
     }
     for (int j = grp; j < n_tiles; j += GROUPS) {
       const int sb = j % S_BUFS, s = j % V_STAGES;
-      const int j0 = tile0 + j * BN;
+      const int j0 = tile_start(j);
       const int use = j / GROUPS;  // how often this group's barriers have been used
       if (!mbar_wait_bounded(&s_full[j % (2 * S_BUFS)], (j / (2 * S_BUFS)) & 1)) {
         ok = false;
@@ -369,12 +378,16 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
       tmem_load_32x32(tmem + lane_base + S_COL0 + sb * BN + part * CW, sr);
       tmem_wait_load();
       const bool need_mask = !rows_full || j0 + BN - 1 > warp_pos_lo || j0 < warp_lo;
+      if (p.exact_cap) {
+#pragma unroll
+        for (int c = 0; c < CW; ++c) sr[c] = __float_as_uint(tanh_by_exp(__uint_as_float(sr[c]) * inv_cap));
+      }
       float mx = -INFINITY;
       if (need_mask) {
 #pragma unroll
         for (int c = 0; c < CW; ++c) {
           float v = __uint_as_float(sr[c]);
-          if (p.cap > 0.f) v = fast_tanh(v * inv_cap);
+          if (fast_cap) v = fast_tanh(v * inv_cap);
           const int key = j0 + part * CW + c;
           if (linear) {
             v -= bias_r1 * (float)max(pos - key, 0);
@@ -383,7 +396,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
             v -= tabled ? bias_tab[min(d, p.window - 1) * group + head_in_group]
                         : bias_r1 * __log2f(fmaf(bias_r2, (float)d, 1.0f));
           }
-          v = (key <= pos && key >= row_lo) ? v : -INFINITY;
+          v = (key <= pos && (key >= row_lo || key < p.keep_first)) ? v : -INFINITY;
           sr[c] = __float_as_uint(v);
           mx = fmaxf(mx, v);
         }
@@ -391,7 +404,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
 #pragma unroll
         for (int c = 0; c < CW; ++c) {
           float v = __uint_as_float(sr[c]);
-          if (p.cap > 0.f) v = fast_tanh(v * inv_cap);
+          if (fast_cap) v = fast_tanh(v * inv_cap);
           if (linear) {
             v -= bias_r1 * (float)(pos - (j0 + part * CW + c));
           } else if (biased) {
@@ -488,7 +501,7 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
         for (int i = (quarter + 4 * part) * 32 + lane; i < BN * VSLABS * 8; i += 128 * SPLIT) {
           const int key_row = (i / 8) % BN, sl = i / (8 * BN), c = i % 8;
           const int key = j0 + key_row;
-          if (key < kv_lo || key >= kv_hi)
+          if ((key < kv_lo && key >= p.keep_first) || key >= kv_hi)
             *reinterpret_cast<uint4*>(sv + s * V_TILE_BYTES + sl * (BN * 128) + key_row * 128 + c * 16) = make_uint4(0, 0, 0, 0);
         }
         fence_proxy_async();  // the zeroed value rows are visible to the tensor core's reads
@@ -592,10 +605,11 @@ static_assert(V_STAGES == 2, "the zeroing of value rows looks two tiles back");
 static int prefill_tc_launch(const void* q, const void* cache, const int* block_table, int max_pages,
                              const int* cu_q, const int* q_start, void* out, int num_tokens,
                              int num_q_heads, int num_kv_heads, int page_size, int num_pages, float cap,
-                             int window, const float* distance, int linear, const float* sink, int key_chunk,
+                             int window, const float* distance, int linear, const float* sink, int key_chunk, int keep_first,
                              const int* items, int num_items, int* err, cudaStream_t stream) {
   if (num_items == 0) return 0;
-  if ((distance != nullptr || sink != nullptr) && cap > 0.f) return -13;
+  if (distance != nullptr && cap > 0.f) return -13;
+  if (keep_first < 0 || (keep_first > 0 && window <= 0)) return -13;
   if (key_chunk > 0 && window > 0) return -13;
   if (num_kv_heads <= 0 || num_q_heads % num_kv_heads) return -8;
   const int group = num_q_heads / num_kv_heads;
@@ -627,6 +641,8 @@ static int prefill_tc_launch(const void* q, const void* cache, const int* block_
   p.num_q_heads = num_q_heads; p.num_kv_heads = num_kv_heads; p.page_size = page_size; p.num_pages = num_pages;
   p.cap = cap; p.window = window; p.items = items; p.box_rows = box_rows; p.err = err;
   p.distance = distance; p.linear = linear; p.sink = sink; p.key_chunk = key_chunk;
+  p.keep_first = keep_first;
+  p.exact_cap = cap > 0.f && (sink != nullptr || keep_first > 0);
   size_t table_bytes = 0;
   static int table_allowed = -1;  // SIMPLY_B200_BIAS_TABLE=0: every softmax thread computes its terms (experiments)
   if (table_allowed < 0) {
@@ -653,16 +669,17 @@ extern "C" int SB_FN(sb_attn_prefill_tc)(const void* q, const void* cache, const
                                          int num_q_heads, int num_kv_heads, int page_size, int num_pages, float cap,
                                          int window, const int* items, int num_items, int* err, cudaStream_t stream) {
   return prefill_tc_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_tokens, num_q_heads, num_kv_heads,
-                           page_size, num_pages, cap, window, nullptr, 0, nullptr, 0, items, num_items, err, stream);
+                           page_size, num_pages, cap, window, nullptr, 0, nullptr, 0, 0, items, num_items, err, stream);
 }
 
-// The same with a distance bias, chunks of keys and a sink (each optional, see TcParams); no cap beside them.
+// The same with a distance bias, chunks of keys, a sink and kept first keys (each optional, see TcParams); no cap
+// beside a distance bias.
 extern "C" int SB_FN(sb_attn_prefill_tc_biased)(const void* q, const void* cache, const int* block_table,
                                                 int max_pages, const int* cu_q, const int* q_start, void* out,
                                                 int num_tokens, int num_q_heads, int num_kv_heads, int page_size,
                                                 int num_pages, float cap, int window, const int* items,
                                                 int num_items, const float* distance, int linear, const float* sink,
-                                                int key_chunk, int* err, cudaStream_t stream) {
+                                                int key_chunk, int keep_first, int* err, cudaStream_t stream) {
   return prefill_tc_launch(q, cache, block_table, max_pages, cu_q, q_start, out, num_tokens, num_q_heads, num_kv_heads,
-                           page_size, num_pages, cap, window, distance, linear, sink, key_chunk, items, num_items, err, stream);
+                           page_size, num_pages, cap, window, distance, linear, sink, key_chunk, keep_first, items, num_items, err, stream);
 }

@@ -274,6 +274,91 @@ extern "C" int sb_residual_norm(float* h, const void* branch, const void* branch
 }
 
 // ---------------------------------------------------------------------------
+// The norm behind a sum.  One block per row:
+//   v = scale * h + branch,  h = v * rsqrt(mean(v^2) + eps) * (w [+ 1])   in float32, in place
+//   y = h in the activation dtype (if given): what the next sublayer reads
+// ---------------------------------------------------------------------------
+template <typename T>
+__global__ void norm_of_sum_kernel(float* __restrict__ h, const T* __restrict__ branch, float scale,
+                                   const void* __restrict__ w, int w_f32, float eps, int plus_one,
+                                   T* __restrict__ y, int width) {
+  extern __shared__ float row[];  // width floats (only where a row is more than one chunk per thread) + 33 scratch
+  constexpr int N = Vec<T>::N;
+  const bool vec = width % N == 0;
+  const bool one_chunk = vec && width <= (int)blockDim.x * N;
+  float* scratch = one_chunk ? row : row + width;
+  const float one = plus_one ? 1.f : 0.f;
+  const int i0 = threadIdx.x * N;
+  const bool on = one_chunk && i0 < width;
+  float wv[N];
+#pragma unroll
+  for (int k = 0; k < N; ++k) wv[k] = 0.f;
+  if (on) load_scalars<N>(w, w_f32, i0, wv);  // (weights: before the wait)
+  pdl_wait_block();
+  pdl_launch_dependents();
+  float* hp = h + (size_t)blockIdx.x * width;
+  const T* bp = branch + (size_t)blockIdx.x * width;
+  T* yp = y != nullptr ? y + (size_t)blockIdx.x * width : nullptr;
+  float ss = 0.f;
+  if (one_chunk) {
+    float v[N], b[N];
+#pragma unroll
+    for (int k = 0; k < N; ++k) v[k] = b[k] = 0.f;
+    if (on) {
+      Vec<T>::load(bp + i0, b);
+#pragma unroll
+      for (int k = 0; k < N; k += 4) Vec<float>::load(hp + i0 + k, v + k);
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      v[k] = fmaf(scale, v[k], b[k]);
+      ss = fmaf(v[k], v[k], ss);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+    if (on) {
+#pragma unroll
+      for (int k = 0; k < N; ++k) v[k] = v[k] * inv * (wv[k] + one);
+#pragma unroll
+      for (int k = 0; k < N; k += 4) Vec<float>::store(hp + i0 + k, v + k);
+      if (yp != nullptr) Vec<T>::store(yp + i0, v);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float v = fmaf(scale, hp[i], to_f32<T>(bp[i]));
+    row[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) {
+    const float v = row[i] * inv * (load_scalar(w, w_f32, i) + one);
+    hp[i] = v;
+    if (yp != nullptr) yp[i] = from_f32<T>(v);
+  }
+}
+
+extern "C" int sb_norm_of_sum(float* h, const void* branch, int dtype, float scale, const void* w, int w_f32, float eps,
+                              int plus_one, void* y, int num_rows, int width, cudaStream_t stream) {
+  if (num_rows == 0) return 0;
+  const int vec = dtype == SB_DTYPE_F32 ? 4 : 8;
+  const bool one_chunk = width % vec == 0 && width / vec <= 1024;
+  const int threads = one_chunk ? max(((width / vec + 31) / 32) * 32, 32) : 512;
+  const size_t smem = ((one_chunk ? 0 : (size_t)width) + 33) * sizeof(float);
+  if (smem > 200 * 1024) return -2;
+#define SB_NORM_SUM(T_)                                                                                            \
+  do {                                                                                                             \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(norm_of_sum_kernel<T_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    sb_launch(norm_of_sum_kernel<T_>, num_rows, threads, smem, stream, h, (const T_*)branch, scale, w, w_f32, eps, \
+              plus_one, (T_*)y, width);                                                                            \
+  } while (0)
+  if (dtype == SB_DTYPE_F32) SB_NORM_SUM(float);
+  else SB_NORM_SUM(bf16);
+#undef SB_NORM_SUM
+  SB_LAUNCH_CHECK();
+  return 0;
+}
+
+// ---------------------------------------------------------------------------
 // Stand-alone RMS norm of rows stored as Tin, result stored as Tout.
 // ---------------------------------------------------------------------------
 template <typename Tin, typename Tout>

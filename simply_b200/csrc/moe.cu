@@ -3,8 +3,9 @@
 //
 //   route    per token: router logits z = W_r x (+ a learned offset per expert) (float32), scores
 //            s = softmax(z) (or sigmoid),
-//            the `top` experts with the largest s + correction, weights s * scale (optionally
-//            divided by their sum), and the shared expert's gate sigmoid(w_sg . x)
+//            the `top` experts with the largest s + correction (of those in the `keep` of `groups`
+//            equal groups of neighbours whose two best add up to most), weights s * scale
+//            (optionally divided by their sum), and the shared expert's gate sigmoid(w_sg . x)
 //   group    the (token, choice) pairs sorted by expert, cut into tiles of TILE_M rows of one
 //            expert each; experts with index >= E ("identity" experts) take no rows
 //   product  out[r, :] = A[row(r), :] . W[expert of r's tile]^T over those tiles, once with two
@@ -29,11 +30,11 @@ __global__ void __launch_bounds__(1024)
 moe_route_kernel(const T* __restrict__ x, int width, const float* __restrict__ router_w,
                  const float* __restrict__ correction, const float* __restrict__ shared_gate_w,
                  const float* __restrict__ bias, int NE, int top,
-                 float scale, int score_fn, int renormalize, int* __restrict__ chosen, float* __restrict__ weight,
+                 float scale, int score_fn, int renormalize, int groups, int keep_groups, int* __restrict__ chosen, float* __restrict__ weight,
                  float* __restrict__ shared_gate) {
   pdl_wait_block();
   pdl_launch_dependents();
-  extern __shared__ __align__(16) float route_smem[];  // x [width], z [NE + 1], choice [NE]
+  extern __shared__ __align__(16) float route_smem[];  // x [width], z [NE + 1], choice [NE], value [groups]
   float* xs = route_smem;
   float* z = xs + width;
   float* choice = z + NE + 1;
@@ -80,6 +81,28 @@ moe_route_kernel(const T* __restrict__ x, int width, const float* __restrict__ r
   }
   for (int e = lane; e < NE; e += 32) choice[e] = z[e] + (correction != nullptr ? correction[e] : 0.f);
   __syncwarp();
+  if (keep_groups < groups) {
+    // What is left of a group that is not kept counts as minus infinity (a choice score may be negative).
+    float* value = choice + NE;
+    const int size = NE / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float first = -INFINITY, second = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float v = choice[e];
+        if (v > first) { second = first; first = v; }
+        else if (v > second) second = v;
+      }
+      value[g] = size > 1 ? first + second : first;
+    }
+    __syncwarp();
+    for (int e = lane; e < NE; e += 32) {
+      const int mine = e / size;
+      int ahead = 0;  // groups worth more (of equals: those before)
+      for (int g = 0; g < groups; ++g) ahead += value[g] > value[mine] || (value[g] == value[mine] && g < mine) ? 1 : 0;
+      if (ahead >= keep_groups) choice[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
   float total = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY;
@@ -105,15 +128,16 @@ moe_route_kernel(const T* __restrict__ x, int width, const float* __restrict__ r
     __syncwarp();
   }
   if (renormalize && lane == 0)
-    for (int j = 0; j < top; ++j) weight[(size_t)t * top + j] /= total;
+    for (int j = 0; j < top; ++j) weight[(size_t)t * top + j] /= total + 1e-20f;
 }
 
 extern "C" int sb_moe_route(const void* x, int dtype, int num_tokens, int width, const float* router_w,
                             const float* correction, const float* shared_gate_w, const float* bias, int NE, int top,
-                            float scale, int score_fn, int renormalize, int* chosen, float* weight,
+                            float scale, int score_fn, int renormalize, int groups, int keep_groups, int* chosen, float* weight,
                             float* shared_gate, cudaStream_t stream) {
   if (num_tokens == 0) return 0;
-  const size_t smem = ((size_t)width + 2 * NE + 1) * sizeof(float);
+  const size_t smem = ((size_t)width + 2 * NE + 1 + groups) * sizeof(float);
+  if (groups < 1 || NE % groups || keep_groups < 1 || keep_groups > groups) return -13;
   if (top < 1 || top > NE || smem > 200 * 1024) return -13;
   // A warp per router row where a block can hold them (at least 8, at most 32 warps): a row's
   // fetches are then one round for all rows instead of one round after the other.
@@ -122,11 +146,11 @@ extern "C" int sb_moe_route(const void* x, int dtype, int num_tokens, int width,
   if (dtype == SB_DTYPE_F32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     sb_launch(moe_route_kernel<float>, num_tokens, 32 * warps, smem, stream, (const float*)x, width, router_w, correction,
-              shared_gate_w, bias, NE, top, scale, score_fn, renormalize, chosen, weight, shared_gate);
+              shared_gate_w, bias, NE, top, scale, score_fn, renormalize, groups, keep_groups, chosen, weight, shared_gate);
   } else {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     sb_launch(moe_route_kernel<bf16>, num_tokens, 32 * warps, smem, stream, (const bf16*)x, width, router_w, correction,
-              shared_gate_w, bias, NE, top, scale, score_fn, renormalize, chosen, weight, shared_gate);
+              shared_gate_w, bias, NE, top, scale, score_fn, renormalize, groups, keep_groups, chosen, weight, shared_gate);
   }
   SB_LAUNCH_CHECK();
   return 0;

@@ -317,6 +317,24 @@ extern "C" int sb_short_conv(const void* x, int x_width, int offset, int dtype, 
   return 0;
 }
 
+// The state alone, for a kernel of another file that convolves on its way (same arguments as above).
+extern "C" int sb_short_conv_state(const void* x, int x_width, int offset, int dtype, float* state, const int* cu_q,
+                                   const int* slots, int num_seqs, int num_slots, int taps, int channels,
+                                   cudaStream_t stream) {
+  if (num_seqs == 0 || channels == 0 || taps < 2) return 0;
+  const int threads = channels >= 256 ? 256 : ((channels + 31) / 32) * 32;
+  const unsigned tiles = (unsigned)((channels + threads - 1) / threads);
+  if (tiles > 65535) return -13;
+  if (dtype == SB_DTYPE_F32)
+    sb_launch(short_conv_state_kernel<float>, dim3((unsigned)num_seqs, tiles), threads, 0, stream, (const float*)x,
+              x_width, offset, state, cu_q, slots, num_slots, taps, channels);
+  else
+    sb_launch(short_conv_state_kernel<bf16>, dim3((unsigned)num_seqs, tiles), threads, 0, stream, (const bf16*)x,
+              x_width, offset, state, cu_q, slots, num_slots, taps, channels);
+  SB_LAUNCH_CHECK();
+  return 0;
+}
+
 // ---------------------------------------------------------------------------
 // Group norm with a gate.  o [T, N] float32; gate [T, gate_width] of T at gate_offset (null: none).
 // gate_kind 1: sigmoid after the norm; 2: silu before it.  Grid (token, group).

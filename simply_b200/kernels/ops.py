@@ -90,14 +90,15 @@ class AttentionGraphPlan:
 
   def __init__(self, ops: "CudaOps", window: int | None, group: int, num_kv_heads: int, head_dim: int,
                batch: int, bucket: int, max_burst: int, page_size: int, key_chunk: int | None = None,
-               value_dim: int | None = None):
-    self.key = ops._plan_key(window, group, num_kv_heads, head_dim, page_size, key_chunk, value_dim)
+               value_dim: int | None = None, keep_first: int = 0):
+    self.key = ops._plan_key(window, group, num_kv_heads, head_dim, page_size, key_chunk, value_dim, keep_first)
     self.window, self.key_chunk, self.group, self.batch = window, key_chunk, group, batch
+    self.keep_first = keep_first
     # Most keys a sequence of this bucket sees in such a layer during a burst.
     reach = window or key_chunk
     span = min(bucket, reach + max_burst + 64) if reach else bucket
     self.chunk = ops.decode_chunk_for([bucket - span] * batch, [bucket] * batch, num_kv_heads, head_dim, value_dim)
-    self.per_seq = -(-span // self.chunk) + 1
+    self.per_seq = -(-span // self.chunk) + 1 + -(-keep_first // self.chunk)
     self.words = batch * self.per_seq * 2 + 2 * batch
 
   def bind(self, view: torch.Tensor) -> dict:
@@ -107,7 +108,8 @@ class AttentionGraphPlan:
                 split_start=view[n:n + self.batch], split_count=view[n + self.batch:])
 
   def fill(self, host_words: np.ndarray, lengths: np.ndarray, steps: int) -> None:
-    items, start, count = CudaOps.static_decode_plan(lengths, steps, self.window, self.chunk, self.per_seq, self.key_chunk)
+    items, start, count = CudaOps.static_decode_plan(lengths, steps, self.window, self.chunk, self.per_seq, self.key_chunk,
+                                                           self.keep_first)
     n = items.size
     host_words[:n] = items.reshape(-1)
     host_words[n:n + self.batch] = start
@@ -255,7 +257,12 @@ class CudaOps:
                                        c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void, c_void],
         "sb_paged_attention_general": [c_void, c_int, c_void, c_void, c_int, c_void, c_void, c_void, c_int,
                                        c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void, c_void,
-                                       c_int, c_int, c_int, c_int, c_void, c_void, c_int, c_int, c_void, c_void],
+                                       c_int, c_int, c_int, c_int, c_void, c_void, c_int, c_int, c_int, c_void, c_void],
+        "sb_norm_of_sum": [c_void, c_void, c_int, c_float, c_void, c_int, c_float, c_int, c_void, c_int, c_int, c_void],
+        "sb_conv_headnorm_store": [c_void, c_int, c_int, c_void, c_int, c_void, c_void, c_int, c_int, c_int, c_void,
+                                   c_void, c_float, c_float, c_void, c_int, c_int, c_void, c_void, c_void, c_int, c_void,
+                                   c_void, c_void, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void, c_void],
+        "sb_short_conv_state": [c_void, c_int, c_int, c_int, c_void, c_void, c_void, c_int, c_int, c_int, c_int, c_void],
         "sb_residual_two_norms": [c_void, c_void, c_void, c_void, c_int, c_void, c_int, c_float, c_int, c_void, c_int,
                                   c_float, c_int, c_void, c_void, c_int, c_void, c_void, c_void, c_int, c_int, c_int,
                                   c_void, c_void, c_int, c_void, c_void],
@@ -307,7 +314,7 @@ class CudaOps:
         "sb_forget_scan": [c_void, c_int, c_int, c_void, c_void, c_void, c_void, c_void, c_int, c_int, c_int, c_int,
                            c_int, c_int, c_int, c_void, c_void, c_void, c_void],
         "sb_moe_route": [c_void, c_int, c_int, c_int, c_void, c_void, c_void, c_void, c_int, c_int, c_float, c_int, c_int,
-                         c_void, c_void, c_void, c_void],
+                         c_int, c_int, c_void, c_void, c_void, c_void],
         "sb_moe_group": [c_void, c_int, c_int, c_int, c_void, c_void, c_void, c_void, c_void, c_void],
         "sb_moe_product": [c_void, c_void, c_int, c_void, c_int, c_int, c_int, c_int, c_void, c_void, c_void, c_int,
                            c_int, c_float, c_void, c_void],
@@ -443,10 +450,10 @@ class CudaOps:
       decode = getattr(lib, f"sb_attn_decode_{suffix}")
       decode.argtypes = [c_void, c_void, c_void, c_int, c_void, c_void, c_void, c_void, c_int, c_int, c_int,
                          c_int, c_int, c_float, c_int, c_void, c_int, c_int, c_void, c_void, c_void, c_int,
-                         c_void, c_void, c_int, c_void, c_int, c_void, c_int, c_void, c_int, c_void, c_void]
+                         c_void, c_void, c_int, c_void, c_int, c_void, c_int, c_void, c_int, c_int, c_void, c_void]
       decode.restype = c_int
       prefill_biased = getattr(lib, f"sb_attn_prefill_biased_{suffix}")
-      prefill_biased.argtypes = prefill.argtypes[:-2] + [c_void, c_int, c_void, c_int, c_void, c_void]
+      prefill_biased.argtypes = prefill.argtypes[:-2] + [c_void, c_int, c_void, c_int, c_int, c_void, c_void]
       prefill_biased.restype = c_int
       make_map = getattr(lib, f"sb_attn_tensor_map_{suffix}")
       make_map.argtypes = [c_void, c_void, ctypes.c_longlong, c_int]
@@ -456,7 +463,7 @@ class CudaOps:
                              c_int, c_float, c_int, c_void, c_int, c_void, c_void]
       prefill_tc.restype = c_int
       prefill_tc_biased = getattr(lib, f"sb_attn_prefill_tc_biased_{suffix}")
-      prefill_tc_biased.argtypes = prefill_tc.argtypes[:-2] + [c_void, c_int, c_void, c_int, c_void, c_void]
+      prefill_tc_biased.argtypes = prefill_tc.argtypes[:-2] + [c_void, c_int, c_void, c_int, c_int, c_void, c_void]
       prefill_tc_biased.restype = c_int
       prefill_pair = None
       if head_dim in (128, 256) and value_dim == head_dim:
@@ -534,12 +541,13 @@ class CudaOps:
 
   @staticmethod
   def static_decode_plan(q_start: np.ndarray, steps: int, window: int | None, chunk: int,
-                         items_per_seq: int, key_chunk: int | None = None) -> tuple[np.ndarray, np.ndarray, np.ndarray]:
+                         items_per_seq: int, key_chunk: int | None = None, keep_first: int = 0) -> tuple[np.ndarray, np.ndarray, np.ndarray]:
     """Work list of the split-key kernel for a decode burst replayed from a CUDA graph.
 
     Every sequence gets exactly `items_per_seq` items, so the launch has a fixed size:
     the chunks that hold keys between the lowest key visible at the first step and the
-    highest at the last step, then fillers (sequence -1).  A chunk that holds nothing
+    highest at the last step (ahead of them those that hold kept first keys), then fillers
+    (sequence -1).  A chunk that holds nothing
     visible at some step of the burst yields an empty partial result there.
     Returns (items [B * items_per_seq, 2], split_start [B], split_count [B]).
     """
@@ -548,11 +556,13 @@ class CudaOps:
     count = np.zeros(b, dtype=np.int32)
     firsts, lasts = CudaOps.decode_chunk_range(q_start, steps, window, chunk, key_chunk)
     for i, (first, last) in enumerate(zip(firsts.tolist(), lasts.tolist())):
-      n = last - first + 1
+      kept = min(-(-keep_first // chunk), first)
+      n = kept + last - first + 1
       if n > items_per_seq:
         raise KernelError(f"decode burst needs {n} chunks per sequence, the graph holds {items_per_seq}")
       items[i, :n, 0] = i
-      items[i, :n, 1] = np.arange(first, last + 1)
+      items[i, :kept, 1] = np.arange(kept)
+      items[i, kept:n, 1] = np.arange(first, last + 1)
       count[i] = n
     start = (np.arange(b) * items_per_seq).astype(np.int32)
     return items.reshape(-1, 2), start, count
@@ -594,24 +604,26 @@ class CudaOps:
     return self.prefill_rows or 64
 
   def _plan_key(self, window: int | None, group: int, num_kv_heads: int, head_dim: int, page_size: int,
-                key_chunk: int | None = None, value_dim: int | None = None) -> tuple:
+                key_chunk: int | None = None, value_dim: int | None = None, keep_first: int = 0) -> tuple:
     """Where a step keeps the work lists of one kind of attention layer in `ctx.memo`.  Layers
     share lists only if everything the lists are cut for agrees: the window, the group, the
     number of kv heads and the head size (they set the chunk length) and the rows of a prefill tile."""
     key = ("attention_plan", window, group, num_kv_heads, head_dim, self._prefill_rows(head_dim, group, page_size))
     other_values = value_dim if value_dim != head_dim else None
+    if keep_first:
+      return key + (key_chunk, other_values, keep_first)
     return key if key_chunk is None and other_values is None else key + (key_chunk, other_values)
 
   def attention_graph_plan(self, *, window: int | None, num_heads: int, num_kv_heads: int, head_dim: int,
                            batch: int, bucket: int, max_burst: int, page_size: int, key_chunk: int | None = None,
-                           value_dim: int | None = None):
+                           value_dim: int | None = None, keep_first: int = 0):
     """The static work list a decode graph needs for one kind of attention layer, or None when
     the kernel that serves it reads no list (the general kernel)."""
     group = num_heads // num_kv_heads
     if not self._uses_tensor_core_attention(head_dim, group, value_dim):
       return None
     return AttentionGraphPlan(self, window, group, num_kv_heads, head_dim, batch, bucket, max_burst, page_size,
-                              key_chunk, value_dim)
+                              key_chunk, value_dim, keep_first)
 
   def pooled_attention_graph_plan(self, *, window: int | None, num_heads: int, num_kv_heads: int, head_dim: int,
                                   value_dim: int, pool: int, batch: int, page_size: int):
@@ -624,7 +636,7 @@ class CudaOps:
 
   def _attention_plan(self, ctx: Any, window: int | None, group: int, force_rows: int = 0,
                       num_kv_heads: int = 1, head_dim: int = 0, tag: tuple = (), all_tiles: bool = False,
-                      key_chunk: int | None = None, value_dim: int | None = None) -> dict:
+                      key_chunk: int | None = None, value_dim: int | None = None, keep_first: int = 0) -> dict:
     """Work lists of the two tensor-core kernels for this step, per kind of layer (`_plan_key`).
 
     Sequences with at most 16 query rows per kv head (one or a few new tokens) go to the
@@ -632,7 +644,7 @@ class CudaOps:
     absolute position, one work item per chunk.  The others are cut into tiles of
     64 // group or 128 // group tokens for the prefill kernel, heaviest tile first.
     """
-    key = self._plan_key(window, group, num_kv_heads, head_dim, ctx.page_size, key_chunk, value_dim) + tag
+    key = self._plan_key(window, group, num_kv_heads, head_dim, ctx.page_size, key_chunk, value_dim, keep_first) + tag
     plan = ctx.memo.get(key)
     if plan is not None:
       return plan
@@ -649,7 +661,7 @@ class CudaOps:
         last = int(q_start[b]) + min(i0 + tokens_per_tile, int(q_len[b]))
         at = int(q_start[b]) + i0
         first = max(at - window + 1, 0) if window else at // key_chunk * key_chunk if key_chunk else 0
-        pre.append((last - first, int(b), i0))
+        pre.append((last - first + min(keep_first, first), int(b), i0))
     pre.sort(key=lambda x: -x[0])
     if force_rows in (128, 256):
       # The tcgen05 kernels' blocks, one per (tile of queries, kv head), longest walk first over all
@@ -671,9 +683,10 @@ class CudaOps:
     dec_items = []
     for b in dec:
       first, last = int(kv_lo[b]) // chunk, (int(kv_hi[b]) - 1) // chunk
+      chunks = list(range(min(-(-keep_first // chunk), first))) + list(range(first, last + 1))
       split_start[b] = len(dec_items)
-      split_count[b] = last - first + 1
-      dec_items += [(int(b), c) for c in range(first, last + 1)]
+      split_count[b] = len(chunks)
+      dec_items += [(int(b), c) for c in chunks]
     decode_items = np.array(dec_items, dtype=np.int32).reshape(-1, 2)
     flat = np.concatenate([prefill_items.reshape(-1), decode_items.reshape(-1), split_start, split_count])
     dev = torch.from_numpy(flat).to(self.device, non_blocking=True)
@@ -859,6 +872,15 @@ class CudaOps:
         _ptr(rows), _ptr(y), num_rows, width, h.shape[0], _ptr(self.err))
     return y
 
+  def norm_of_sum(self, h: torch.Tensor, branch: torch.Tensor, scale: float, norm: Any) -> torch.Tensor:
+    """h <- norm(scale * h + branch), float32 in place; returns h in the activation dtype (csrc/elementwise.cu)."""
+    if branch.dtype != self.dtype:
+      branch = self.cast(branch, self.dtype)
+    y = self._new(*h.shape) if self.dtype != torch.float32 else None
+    self._call("sb_norm_of_sum", _ptr(h), _ptr(branch), _code(branch), float(scale), _ptr(norm.weight),
+               int(norm.weight.dtype == torch.float32), float(norm.eps), int(norm.plus_one), _ptr(y), h.shape[0], h.shape[1])
+    return h if y is None else y
+
   def residual_two_norms(self, h: torch.Tensor, branch: torch.Tensor | None, branch2: torch.Tensor | None, norm: Any,
                          norm2: Any, shift: torch.Tensor | None, state: torch.Tensor | None, ctx: Any):
     """(h + branch + branch2, y, y2): y = norm(h + ...), with `shift` (float32 [width]) moved towards the
@@ -1034,7 +1056,8 @@ class CudaOps:
                       num_heads: int, num_kv_heads: int, head_dim: int, logit_softcap: float,
                       window: int | None, value_dim: int | None = None, pooled: tuple | None = None,
                       values_in_keys: bool = False, sink: torch.Tensor | None = None,
-                      distance_bias: torch.Tensor | None = None, key_chunk: int | None = None) -> torch.Tensor:
+                      distance_bias: torch.Tensor | None = None, key_chunk: int | None = None,
+                      keep_first: int = 0) -> torch.Tensor:
     """`value_dim`: size of a value head where it is not the key heads'.  `pooled`: (storage of block
     entries, its block table, block length): with a window, one key and value per whole block that
     has left the window, under the same softmax.  `values_in_keys`: an entry's value is the first
@@ -1042,13 +1065,19 @@ class CudaOps:
     head whose exponential joins the softmax's denominator (csrc/attention_generic.cu).
     `distance_bias`: float32 [2, heads], r1 and r2 per head: the score of query i and key j loses
     r1 log(1 + r2 (i - j)); float32 [1, heads]: it loses r1 (i - j).  `key_chunk` C (without a
-    window): a query sees its own chunk's keys, from (i // C) * C on."""
+    window): a query sees its own chunk's keys, from (i // C) * C on.  `keep_first` n (with a window): a
+    query also sees its sequence's first n keys."""
     t = q.shape[0]
     value_dim = head_dim if value_dim is None else value_dim
     out = self._new(t, num_heads * value_dim, dtype=q.dtype)
     group = num_heads // num_kv_heads
-    if (values_in_keys or sink is not None or key_chunk is not None) and (logit_softcap or pooled is not None):
-      raise KernelError("latent rows and sinks go with neither a score cap nor pooled blocks")
+    if (values_in_keys or key_chunk is not None) and (logit_softcap or pooled is not None):
+      raise KernelError("latent rows and chunks of keys go with neither a score cap nor pooled blocks")
+    if sink is not None and pooled is not None:
+      raise KernelError("a sink does not go with pooled blocks")
+    keep_first = int(keep_first) if window else 0
+    if keep_first and (pooled is not None or values_in_keys):
+      raise KernelError("kept first keys go with neither pooled blocks nor latent rows")
     if distance_bias is not None and (pooled is not None or values_in_keys):
       raise KernelError("a distance bias goes with neither pooled blocks nor latent rows")
     if key_chunk is not None and (window or pooled is not None or values_in_keys):
@@ -1056,7 +1085,7 @@ class CudaOps:
     linear_bias = int(distance_bias is not None and distance_bias.shape[0] == 1)
     # What the tensor-core kernels below take beside a window: value heads of another size (the mma.sync
     # kernels), and the options that their general entry points have.
-    special = distance_bias is not None or sink is not None or key_chunk is not None
+    special = distance_bias is not None or sink is not None or key_chunk is not None or keep_first > 0
     on_tensor_cores = (q.dtype == torch.bfloat16 and self._uses_tensor_core_attention(head_dim, group, value_dim)
                        and pooled is None and not values_in_keys)
     if pooled is not None or values_in_keys or ((special or value_dim != head_dim) and not on_tensor_cores):
@@ -1071,7 +1100,7 @@ class CudaOps:
                    block_table.shape[1], _ptr(ctx.token_seq), _ptr(ctx.positions), _ptr(out), t, num_heads,
                    num_kv_heads, head_dim, value_dim, ctx.page_size, storage.shape[0], float(logit_softcap),
                    int(window or 0), *pool_args, int(values_in_keys), _ptr(sink), _ptr(distance_bias), linear_bias,
-                   int(key_chunk or 0), _ptr(self.err))
+                   int(key_chunk or 0), keep_first, _ptr(self.err))
 
       # bfloat16 with key size = value size: the tensor-core tile kernel (mma.sync tiles of 64 rows,
       # the block entries in tiles of their own ahead of the tokens) for prompt portions and single
@@ -1119,12 +1148,12 @@ class CudaOps:
     if on_tensor_cores:
       fns = self._attention_lib(head_dim, value_dim)
       prefill, decode, _, prefill_tc, prefill_pair = fns[:5]
-      # A distance bias, a sink or chunks of keys: the tcgen05 kernel by single blocks where it takes the
-      # shape (no cap beside them), else the mma.sync tile kernel; not the kernel by pairs.
-      options = (_ptr(distance_bias), linear_bias, _ptr(sink), int(key_chunk or 0)) if special else (None, 0, None, 0)
-      kind = dict(key_chunk=key_chunk, value_dim=value_dim)
+      # A distance bias, a sink, chunks of keys or kept first keys: the tcgen05 kernel by single blocks where
+      # it takes the shape (no cap beside a distance bias), else the mma.sync tile kernel; not the kernel by pairs.
+      options = (_ptr(distance_bias), linear_bias, _ptr(sink), int(key_chunk or 0), keep_first) if special else (None, 0, None, 0, 0)
+      kind = dict(key_chunk=key_chunk, value_dim=value_dim, keep_first=keep_first)
       use_tc = (self._prefill_uses_tcgen05(head_dim, group, ctx.page_size, special or value_dim != head_dim)
-                and (not special or not logit_softcap))
+                and (distance_bias is None or not logit_softcap))
       use_pair = (prefill_pair is not None and self._prefill_uses_pairs(head_dim, group, ctx.page_size)
                   and not special)
       plan = self._attention_plan(ctx, window, group, 256 if use_pair else (128 if use_tc else 0), num_kv_heads, head_dim, **kind)
@@ -1245,6 +1274,35 @@ class CudaOps:
                _ptr(ctx.token_seq), _ptr(ctx.positions), t, num_heads, num_kv_heads, head_dim, value_dim,
                ctx.page_size, storage.shape[0] if storage is not None else 0, int(storage is not None),
                _ptr(self.err))
+    return q
+
+  def conv_headnorm_rotate_store(self, proj: torch.Tensor, conv_weight: torch.Tensor | None,
+                                 conv_state: torch.Tensor | None, q_norm: torch.Tensor, k_norm: torch.Tensor, eps: float,
+                                 q_scale: float, rot_freq: torch.Tensor | None, *, interleaved: bool, num_heads: int,
+                                 num_kv_heads: int, head_dim: int, value_dim: int, storage: torch.Tensor | None,
+                                 block_table: torch.Tensor, ctx: Any) -> torch.Tensor:
+    """proj [T, q | k | v | ...] -> queries [T, num_heads, head_dim]; keys and values go into the pages of
+    `storage`.  Every channel first passes a causal convolution over time (`conv_weight` float32 [taps,
+    channels], or None) whose earlier inputs `conv_state` [slots, taps - 1, channels] keeps; query and
+    key heads are then RMS-normed with the scales q_norm and k_norm (float32 [head_dim]) and turned,
+    queries multiplied by `q_scale` (csrc/attention_prepare.cu)."""
+    t = proj.shape[0]
+    q = self._new(t, num_heads, head_dim, dtype=proj.dtype)
+    if storage is not None and storage.dtype != proj.dtype:
+      raise KernelError("cache and activations must share one dtype")
+    taps = conv_weight.shape[0] if conv_weight is not None else 0
+    alone = ctx.max_q_len == 1  # every sequence brings one token: the kernel that reads a state row moves it on
+    self._call("sb_conv_headnorm_store", _ptr(proj), proj.shape[1], _code(proj), _ptr(conv_weight), taps, _ptr(conv_state),
+               _ptr(ctx.slots), conv_state.shape[0] if conv_state is not None else 0, ctx.num_seqs, int(alone),
+               _ptr(q_norm), _ptr(k_norm), float(eps), float(q_scale), _ptr(rot_freq),
+               2 * rot_freq.numel() if rot_freq is not None else 0, int(interleaved), _ptr(q), _ptr(storage),
+               _ptr(block_table), block_table.shape[1], _ptr(ctx.token_seq), _ptr(ctx.cu_q), _ptr(ctx.positions), t,
+               num_heads, num_kv_heads, head_dim, value_dim, ctx.page_size,
+               storage.shape[0] if storage is not None else 0, int(storage is not None), _ptr(self.err))
+    if taps > 1 and not alone:
+      channels = conv_weight.shape[1]
+      self._call("sb_short_conv_state", _ptr(proj), proj.shape[1], 0, _code(proj), _ptr(conv_state), _ptr(ctx.cu_q),
+                 _ptr(ctx.slots), ctx.num_seqs, conv_state.shape[0], taps, channels)
     return q
 
   def sigmoid_gate(self, x: torch.Tensor, proj: torch.Tensor, offset: int, per: int = 1) -> torch.Tensor:
@@ -1429,15 +1487,17 @@ class CudaOps:
 
   def route_tokens(self, x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None,
                    shared_gate_w: torch.Tensor | None, *, top: int, scale: float, score: int = 0,
-                   renormalize: bool = False, bias: torch.Tensor | None = None):
+                   renormalize: bool = False, bias: torch.Tensor | None = None, groups: tuple[int, int] | None = None):
     """Per token the `top` chosen experts (int32 [T, top]), their weights (float32 [T, top]) and the
-    shared expert's gate (float32 [T], or None)."""
+    shared expert's gate (float32 [T], or None).  `groups` (count, keep): of that many equal groups of
+    neighbouring experts only those `keep` are open to the choice whose two best experts add up to most."""
     t, width = x.shape
     chosen = self._new(t, top, dtype=torch.int32)
     weight = self._new(t, top, dtype=torch.float32)
     gate = self._new(t, dtype=torch.float32) if shared_gate_w is not None else None
     self._call("sb_moe_route", _ptr(x), _code(x), t, width, _ptr(router), _ptr(correction), _ptr(shared_gate_w),
-               _ptr(bias), router.shape[0], top, float(scale), int(score), int(renormalize), _ptr(chosen), _ptr(weight), _ptr(gate))
+               _ptr(bias), router.shape[0], top, float(scale), int(score), int(renormalize),
+               *(groups or (1, 1)), _ptr(chosen), _ptr(weight), _ptr(gate))
     return chosen, weight, gate
 
   def route_by_table(self, token_ids: torch.Tensor, table: torch.Tensor, num_experts: int):

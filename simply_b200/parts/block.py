@@ -22,6 +22,8 @@ With a norm of its own for the feed-forward (`names["feed_forward_norm"]`) both 
 With `token_shift` the mixer reads, in place of y = norm_1(h), y + (y' - y) * shift with a learned
 factor per channel and y' the previous token's y (zeros before the first; the last y is part of
 a request's state).  The pending branches' adds, both norms and the shift are one kernel.
+`normed_sum` norms the sum itself, and its sublayers read the stream as it is:
+  h = norm_1(a h + mixer(h));  h = norm_2(a h + feed_forward(h))
 """
 
 from __future__ import annotations
@@ -50,6 +52,7 @@ class ResidualStream:
     self._post: Norm | None = None
     self._second: torch.Tensor | None = None
     self._second_post: Norm | None = None
+    self._as_read: tuple | None = None  # (h, the same in the activation dtype), while h holds what the copy does
     # A stream that is kept several times (`hyper_connection` blocks): float32 [T, copies, width]
     # in place of `h`, and the write that is still to be done (branch, mix [from, to], out [to]).
     self.lanes: torch.Tensor | None = None
@@ -89,6 +92,7 @@ class ResidualStream:
     return self.h.clone() if self.lanes is None else self.lanes.sum(dim=1)
 
   def add(self, branch: torch.Tensor, post_norm: Norm | None, ctx: Any) -> None:
+    self._as_read = None
     if self._branch is not None and self._second is None and (
         post_norm is None or (isinstance(post_norm, ChannelScale) and isinstance(self._post, (ChannelScale, type(None))))):
       self._second, self._second_post = branch, post_norm  # rides along: h + first + second in one kernel
@@ -101,6 +105,7 @@ class ResidualStream:
     (when the activation dtype would round it) it is added at once."""
     if x.dtype == self.h.dtype and x.dtype != ctx.ops.dtype:
       self.flush(ctx)
+      self._as_read = None
       ctx.ops.add_to_residual(self.h, x)
     else:
       self.add(x, None, ctx)
@@ -129,6 +134,22 @@ class ResidualStream:
     self.h, y, y2 = ctx.ops.residual_two_norms(self.h, self._branch, self._second, norm, norm2, shift, state, ctx)
     self._branch = self._second = None
     return y, y2
+
+  def plain(self, ctx: Any) -> torch.Tensor:
+    """The stream itself in the activation dtype, for sublayers that read it without a norm."""
+    if self.lanes is not None:
+      raise TypeError("a stream kept several times is read through a norm")
+    self.flush(ctx)
+    if self._as_read is None or self._as_read[0] is not self.h:
+      self._as_read = (self.h, ctx.ops.cast(self.h, ctx.ops.dtype))
+    return self._as_read[1]
+
+  def norm_sum(self, scale: float, branch: torch.Tensor, norm: Norm, ctx: Any) -> None:
+    """h <- norm(scale * h + branch), in one kernel that leaves `plain`'s copy as well."""
+    if self.lanes is not None or not isinstance(norm, RMSNorm):
+      raise TypeError("the norm of a sum: an RMS norm, and a stream that is kept once")
+    self.flush(ctx)
+    self._as_read = (self.h, ctx.ops.norm_of_sum(self.h, branch, scale, norm))
 
   def _ones(self, ctx: Any) -> torch.Tensor:
     key = ("stream_ones", self.lanes.shape[1])
@@ -321,3 +342,48 @@ class ParallelResidualBlock(Block):
     stream.add(self.mixer.forward(y, ctx, cache, writes_cache), self.mixer_scale, ctx)
     if self.feed_forward is not None:
       stream.add(self.feed_forward.forward(y2, ctx), self.feed_forward_scale, ctx)
+
+
+@BLOCKS.register("normed_sum")
+class NormedSumBlock(Block):
+  """The norm stands behind the sum: h <- norm(stream_scale * h + sublayer(h)), for the mixer and then for
+  the feed-forward (if the layer has one).  `names`: {"mixer_norm", "feed_forward_norm"}: the scales'
+  tensor names after the layer's prefix."""
+
+  def __init__(self, prefix: str, width: int, norm: PartSpec, mixer: Mixer, feed_forward: FeedForward,
+               names: dict[str, str] | None = None, stream_scale: float = 1.0):
+    self.prefix, self.stream_scale = prefix, float(stream_scale)
+    self.mixer = mixer
+    self.feed_forward = None if isinstance(feed_forward, NoFeedForward) else feed_forward
+    def make(role: str) -> Norm:
+      name = f"{prefix}.{(names or {}).get(role, role)}"
+      return build_part(NORMS, PartSpec(norm.kind, name, {"width": width, **norm.params, "name": name}))
+    self.mixer_norm, self.feed_forward_norm = make("mixer_norm"), make("feed_forward_norm")
+
+  def _parts(self) -> list:
+    rest = [self.feed_forward, self.feed_forward_norm] if self.feed_forward is not None else []
+    return [self.mixer, self.mixer_norm, *rest]
+
+  def cache_need(self):
+    return self.mixer.cache_need()
+
+  @property
+  def graph_safe(self) -> bool:
+    return all(p.graph_safe for p in self._parts())
+
+  def tensor_specs(self) -> list[TensorSpec]:
+    specs = [s for p in self._parts() for s in p.tensor_specs()]
+    if self.feed_forward is None:  # (not used, but a folder may hold it)
+      specs += [dataclasses.replace(s, optional=True) for s in self.feed_forward_norm.tensor_specs()]
+    return specs
+
+  def bind(self, tensors, ops) -> None:
+    for p in self._parts():
+      p.bind(tensors, ops)
+
+  def forward(self, stream: ResidualStream, ctx: Any, cache: Any, writes_cache: bool = True) -> None:
+    y = self.mixer.forward(stream.plain(ctx), ctx, cache, writes_cache)
+    stream.norm_sum(self.stream_scale, y, self.mixer_norm, ctx)
+    if self.feed_forward is not None:
+      y = self.feed_forward.forward(stream.plain(ctx), ctx)
+      stream.norm_sum(self.stream_scale, y, self.feed_forward_norm, ctx)

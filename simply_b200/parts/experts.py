@@ -7,6 +7,9 @@ Per token y:
   s = softmax(z)   (`score` "sigmoid": sigmoid(z))
   chosen = the `top` experts with the largest s + c   (`correction`: c is a learned number per
            expert that shifts the choice only)
+           With `groups` = (count, keep) the experts form `count` equal groups of neighbours, a group
+           is worth the sum of its two largest s + c, and only experts of the `keep` groups worth
+           most can be chosen
   a_e = s_e * weight_scale                  (`renormalize`: divided by the chosen experts' sum of s)
   out = sum over chosen e of a_e * expert_e(y)  +  sigmoid(w_sg . y) * shared(y)
 
@@ -48,7 +51,12 @@ class RoutedExperts(FeedForward):
                num_identity: int = 0, weight_scale: float = 1.0, score: str = "softmax", correction: bool = False,
                renormalize: bool = False, shared_hidden: int = 0, shared_gate: bool = False,
                names: dict[str, str] | None = None, router_bias: bool = False, limit: float = 0.0,
-               shared_limit: float | None = None):
+               shared_limit: float | None = None, groups: tuple[int, int] | None = None):
+    if groups is not None:
+      count, keep = groups
+      if num_identity or num_experts % count or not 1 <= keep <= count or top > num_experts // count * keep:
+        raise ValueError(f"{prefix}: {keep} of {count} groups do not fit a choice of {top} among {num_experts} experts")
+    self.groups = groups
     if score not in _SCORES:
       raise ValueError(f"{prefix}: router score must be one of {sorted(_SCORES)}, got {score!r}")
     if not 1 <= top <= num_experts + num_identity:
@@ -115,7 +123,9 @@ class RoutedExperts(FeedForward):
   def forward(self, x: torch.Tensor, ctx: Any) -> torch.Tensor:
     ops = ctx.ops
     # (only what differs from the plain case is passed on: see HeadNormAttention._store_options)
-    more = {"bias": self.router_bias} if self.router_bias is not None else {}
+    more: dict[str, Any] = {"bias": self.router_bias} if self.router_bias is not None else {}
+    if self.groups is not None and self.groups[1] < self.groups[0]:
+      more["groups"] = self.groups
     chosen, weight, gate = ops.route_tokens(
         x, self.router, self.correction, self.shared_gate_w, top=self.top, scale=self.weight_scale,
         score=self.score, renormalize=self.renormalize, **more)

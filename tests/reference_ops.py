@@ -140,6 +140,10 @@ class ReferenceOps:
   def linear_relu_squared(self, x, w):
     return torch.relu(self.linear(x, w).float()).pow(2).to(self.dtype)
 
+  def norm_of_sum(self, h, branch, scale, norm):
+    h.copy_(self._rms(scale * h + branch.float(), norm.weight, norm.eps, norm.plus_one))
+    return h.to(self.dtype) if self.dtype != torch.float32 else h
+
   def residual_two_norms(self, h, branch, branch2, norm, norm2, shift, state, ctx):
     for b in (branch, branch2):
       if b is not None:
@@ -202,12 +206,13 @@ class ReferenceOps:
   # ---- attention ------------------------------------------------------------
   def paged_attention(self, q, storage, block_table, ctx, *, num_heads, num_kv_heads, head_dim,
                       logit_softcap, window, value_dim=None, pooled=None, values_in_keys=False, sink=None,
-                      distance_bias=None, key_chunk=None):
+                      distance_bias=None, key_chunk=None, keep_first=0):
     if (pooled is not None or (value_dim is not None and value_dim != head_dim) or values_in_keys or sink is not None
-        or distance_bias is not None or key_chunk is not None):
-      assert not logit_softcap
+        or distance_bias is not None or key_chunk is not None or keep_first):
+      assert not logit_softcap or (pooled is None and not values_in_keys and key_chunk is None and distance_bias is None)
       return self._general_attention(q, storage, block_table, ctx, num_heads, num_kv_heads, head_dim,
-                                     value_dim or head_dim, window, pooled, values_in_keys, sink, distance_bias, key_chunk)
+                                     value_dim or head_dim, window, pooled, values_in_keys, sink, distance_bias, key_chunk,
+                                     keep_first, logit_softcap)
     t = q.shape[0]
     out = torch.zeros(t, num_heads, head_dim, dtype=torch.float32, device=q.device)
     group = num_heads // num_kv_heads
@@ -306,7 +311,8 @@ class ReferenceOps:
     return y.reshape(t, num_heads * dim).to(self.dtype)
 
   def _general_attention(self, q, storage, block_table, ctx, num_heads, num_kv_heads, head_dim, value_dim,
-                         window, pooled, values_in_keys=False, sink=None, distance_bias=None, key_chunk=None):
+                         window, pooled, values_in_keys=False, sink=None, distance_bias=None, key_chunk=None,
+                         keep_first=0, cap=0.0):
     t = q.shape[0]
     ps = ctx.page_size
     if values_in_keys:  # one row per entry: the key, whose first value_dim numbers are the value
@@ -326,6 +332,8 @@ class ReferenceOps:
         if key_chunk is not None:  # the query's own chunk only
           lo = i // key_chunk * key_chunk
         j = torch.arange(lo, i + 1, device=q.device)
+        if window is not None and keep_first:  # the sequence's first tokens stay visible
+          j = torch.cat([torch.arange(min(keep_first, lo), device=q.device), j])
         page = block_table[b, j // ps].long()
         assert (page >= 0).all(), "attention would read a page the request does not hold"
         k = keys[page, :, j % ps, :].float()
@@ -344,6 +352,8 @@ class ReferenceOps:
         for n in range(num_heads):
           m = n // group
           scores = k[:, m] @ q[r, n].float()
+          if cap:
+            scores = cap * torch.tanh(scores / cap)
           if distance_bias is not None and distance_bias.shape[0] == 1:  # [1, heads]: slope * distance
             assert pooled is None
             scores = scores - distance_bias[0, n] * (i - j).float()
@@ -396,6 +406,37 @@ class ReferenceOps:
       values[page, :, pos % ps, :] = v.to(storage.dtype)
     return (prepare(q) * q_scale).to(self.dtype)
 
+  def conv_headnorm_rotate_store(self, proj, conv_weight, conv_state, q_norm, k_norm, eps, q_scale, rot_freq, *,
+                                 interleaved, num_heads, num_kv_heads, head_dim, value_dim, storage, block_table, ctx):
+    t = proj.shape[0]
+    nq, nk, nv = num_heads * head_dim, num_kv_heads * head_dim, num_kv_heads * value_dim
+    cols = proj[:, :nq + nk + nv].float()
+    if conv_weight is not None:  # [taps, channels]
+      cols = self.short_conv(cols, conv_weight.t(), None, conv_state, ctx, out_dtype=torch.float32)
+
+    def prepare(x, heads, scale):
+      x = x.reshape(t, heads, head_dim)
+      x = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * scale.float()
+      if rot_freq is not None:
+        dims = 2 * rot_freq.numel()
+        angle = ctx.positions.float()[:, None, None] * rot_freq.float()[None, None, :]
+        c, s = torch.cos(angle), torch.sin(angle)
+        ia = torch.arange(0, dims, 2) if interleaved else torch.arange(0, dims // 2)
+        ib = ia + 1 if interleaved else ia + dims // 2
+        a, b = x[..., ia], x[..., ib]
+        x[..., ia], x[..., ib] = a * c - b * s, b * c + a * s
+      return x
+
+    if storage is not None:
+      ps = ctx.page_size
+      pos = ctx.positions.long()
+      page = block_table[ctx.token_seq.long(), pos // ps].long()
+      assert (page >= 0).all(), "a token would be written to a page the request does not hold"
+      keys, values = self._kv_views(storage, num_kv_heads, ps, head_dim, value_dim)
+      keys[page, :, pos % ps, :] = prepare(cols[:, nq:nq + nk], num_kv_heads, k_norm).to(storage.dtype)
+      values[page, :, pos % ps, :] = cols[:, nq + nk:].reshape(t, num_kv_heads, value_dim).to(storage.dtype)
+    return (prepare(cols[:, :nq], num_heads, q_norm) * q_scale).to(self.dtype)
+
   def sigmoid_gate(self, x, proj, offset, per=1):
     gate = torch.sigmoid(proj[:, offset:offset + x.shape[1] // per].float())
     return (x.float() * gate.repeat_interleave(per, dim=1)).to(self.dtype)
@@ -440,12 +481,20 @@ class ReferenceOps:
     return out
 
   # ---- routed experts ---------------------------------------------------------------
-  def route_tokens(self, x, router, correction, shared_gate_w, *, top, scale, score=0, renormalize=False, bias=None):
+  def route_tokens(self, x, router, correction, shared_gate_w, *, top, scale, score=0, renormalize=False, bias=None,
+                   groups=None):
     z = x.float() @ router.float().t()
     if bias is not None:
       z = z + bias.float()
     s = torch.softmax(z, dim=-1) if score == 0 else torch.sigmoid(z)
     choice = s + (correction.float() if correction is not None else 0.0)
+    if groups is not None:
+      count, keep = groups
+      parts = choice.view(choice.shape[0], count, -1)
+      worth = parts.sort(dim=-1, descending=True).values[..., :2].sum(-1)
+      out = torch.argsort(-worth, dim=-1, stable=True)[:, keep:]
+      choice = parts.masked_fill(torch.zeros_like(worth, dtype=torch.bool).scatter_(1, out, True)[..., None],
+                                 float("-inf")).reshape(choice.shape)
     chosen = torch.argsort(-choice, dim=-1, stable=True)[:, :top]
     weight = torch.gather(s, 1, chosen)
     weight = weight / weight.sum(-1, keepdim=True) * scale if renormalize else weight * scale
