@@ -596,6 +596,167 @@ conv_headnorm_store_kernel(const T* __restrict__ proj, int row_width, const floa
   }
 }
 
+// The same for steps with prompt portions, two neighbouring channels per lane: the taps' weights of a warp's
+// head and its last rows stay in registers from token to token.  Heads of up to 64 * NCH channels, whole
+// pairs of channels everywhere (d, dv, the row width and half the turned dims are even).
+template <typename T> struct Pair;
+template <> struct Pair<float> {
+  __device__ static float2 load(const float* p) { return *reinterpret_cast<const float2*>(p); }
+  __device__ static void store(float* p, float2 v) { *reinterpret_cast<float2*>(p) = v; }
+};
+template <> struct Pair<bf16> {
+  __device__ static float2 load(const bf16* p) {
+    const uint32_t v = *reinterpret_cast<const uint32_t*>(p);
+    return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u));
+  }
+  __device__ static void store(bf16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
+};
+
+template <typename T, int TAPS, int NCH>
+__global__ void __launch_bounds__(PREP_WARPS * 32)
+conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, const float* __restrict__ conv_w,
+                                 const float* __restrict__ state, const int* __restrict__ slots, int num_slots,
+                                 const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps, float q_scale,
+                                 const float* __restrict__ rot_freq, int rot_dims, int interleaved, T* __restrict__ q_out,
+                                 T* __restrict__ cache, const int* __restrict__ block_table, int max_pages,
+                                 const int* __restrict__ token_seq, const int* __restrict__ cu_q,
+                                 const int* __restrict__ positions, int num_tokens, int rows_per_block, int H, int G, int d, int dv,
+                                 int page_size, int num_pages, int write_cache, int* err) {
+  extern __shared__ float prep_smem[];
+  const int half = rot_dims / 2, hd = max(d, dv);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t0 = blockIdx.x * rows_per_block, rows = min(rows_per_block, num_tokens - t0);
+  const int head = blockIdx.y * PREP_WARPS + warp;
+  const bool on = head < H + 2 * G, is_q = head < H, is_v = head >= H + G;
+  const int n = is_v ? dv : d;
+  const int c0 = is_v ? (H + G) * d + (head - H - G) * dv : head * d;
+  const int channels = (H + G) * d + G * dv;
+  constexpr int W = TAPS > 0 ? TAPS : 1;
+  float2 w[W][NCH], scale[NCH];
+  if (on) {  // (weights: before the wait)
+    const float* scale_w = is_q ? q_norm : k_norm;
+#pragma unroll
+    for (int k = 0; k < NCH; ++k) {
+      const int c = 2 * lane + 64 * k;
+      scale[k] = c < n && !is_v ? Pair<float>::load(scale_w + c) : make_float2(0.f, 0.f);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+        w[j][k] = c < n ? Pair<float>::load(conv_w + (size_t)j * channels + c0 + c) : make_float2(0.f, 0.f);
+    }
+  }
+  pdl_wait_block();
+  pdl_launch_dependents();
+  for (int i = threadIdx.x; i < rows * half; i += blockDim.x) {
+    const int r = i / half, a = i - r * half;
+    sincosf((float)positions[t0 + r] * rot_freq[a], prep_smem + (2 * r + 1) * half + a, prep_smem + 2 * r * half + a);
+  }
+  __syncthreads();
+  if (!on) return;
+  float* buf = prep_smem + 2 * rows_per_block * half + (size_t)warp * hd;
+  const size_t page_stride = (size_t)G * page_size * (d + dv);
+  float2 past[W][NCH];  // the rows before the token, oldest first (W - 1 of them)
+
+  for (int r = 0; r < rows; ++r) {
+    const int t = t0 + r, b = token_seq[t];
+    const int i = t - cu_q[b];
+    const T* x = proj + (size_t)t * row_width + c0;
+    if (TAPS > 1 && (r == 0 || i == 0)) {
+      const int slot = slots[b];
+      const bool bad = slot < 0 || slot >= num_slots;
+      if (bad && lane == 0) atomicOr(err, SB_ERR_BAD_SLOT);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) {
+        const int at = i - (TAPS - 1) + j;
+#pragma unroll
+        for (int k = 0; k < NCH; ++k) {
+          const int c = 2 * lane + 64 * k;
+          float2 v = make_float2(0.f, 0.f);
+          if (c < n) {
+            if (at >= 0) v = Pair<T>::load(x + c - (long long)(TAPS - 1 - j) * row_width);
+            else if (!bad) v = Pair<float>::load(state + ((size_t)slot * (TAPS - 1) + TAPS - 1 + at) * channels + c0 + c);
+          }
+          past[j][k] = v;
+        }
+      }
+    }
+    float2 u[NCH];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NCH; ++k) {
+      const int c = 2 * lane + 64 * k;
+      const float2 own = c < n ? Pair<T>::load(x + c) : make_float2(0.f, 0.f);
+      u[k] = own;
+      if (TAPS > 0) {
+        u[k] = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) {
+          u[k].x = fmaf(w[j][k].x, past[j][k].x, u[k].x);
+          u[k].y = fmaf(w[j][k].y, past[j][k].y, u[k].y);
+        }
+        u[k].x = fmaf(w[W - 1][k].x, own.x, u[k].x);
+        u[k].y = fmaf(w[W - 1][k].y, own.y, u[k].y);
+#pragma unroll
+        for (int j = 0; j + 2 < TAPS; ++j) past[j][k] = past[j + 1][k];
+        if (TAPS > 1) past[W > 1 ? W - 2 : 0][k] = own;
+      }
+      ss = fmaf(u[k].x, u[k].x, fmaf(u[k].y, u[k].y, ss));
+    }
+    T* dst = nullptr;
+    if (is_q) {
+      dst = q_out + ((size_t)t * H + head) * d;
+    } else if (write_cache) {
+      const int p = positions[t];
+      const long long page = block_table[(size_t)b * max_pages + p / page_size];
+      if (page < 0 || page >= num_pages) {
+        if (lane == 0) atomicOr(err, SB_ERR_BAD_PAGE);
+      } else if (is_v) {
+        dst = cache + page * page_stride + (size_t)G * page_size * d + ((size_t)(head - H - G) * page_size + p % page_size) * dv;
+      } else {
+        dst = cache + page * page_stride + ((size_t)(head - H) * page_size + p % page_size) * d;
+      }
+    }
+    if (is_v) {
+#pragma unroll
+      for (int k = 0; k < NCH; ++k) {
+        const int c = 2 * lane + 64 * k;
+        if (c < n && dst != nullptr) Pair<T>::store(dst + c, u[k]);
+      }
+      continue;
+    }
+    const float inv = (is_q ? q_scale : 1.0f) / sqrtf(warp_sum(ss) / (float)d + eps);
+    const float* cs = prep_smem + 2 * r * half;
+#pragma unroll
+    for (int k = 0; k < NCH; ++k) {
+      u[k].x *= inv * scale[k].x;
+      u[k].y *= inv * scale[k].y;
+      const int c = 2 * lane + 64 * k;
+      if (!interleaved && c < rot_dims) Pair<float>::store(buf + c, u[k]);
+    }
+    __syncwarp();
+#pragma unroll
+    for (int k = 0; k < NCH; ++k) {
+      const int c = 2 * lane + 64 * k;
+      if (c >= n) continue;
+      float2 v = u[k];
+      if (c < rot_dims) {
+        if (interleaved) {
+          const float cc = cs[c >> 1], sn = cs[half + (c >> 1)];
+          v = make_float2(u[k].x * cc - u[k].y * sn, u[k].y * cc + u[k].x * sn);
+        } else {
+          const bool low = c < half;
+          const int a = low ? c : c - half;
+          const float2 o = Pair<float>::load(buf + (low ? c + half : a));
+          const float2 cc = Pair<float>::load(cs + a), sn = Pair<float>::load(cs + half + a);
+          v = low ? make_float2(v.x * cc.x - o.x * sn.x, v.y * cc.y - o.y * sn.y)
+                  : make_float2(v.x * cc.x + o.x * sn.x, v.y * cc.y + o.y * sn.y);
+        }
+      }
+      if (dst != nullptr) Pair<T>::store(dst + c, v);
+    }
+    __syncwarp();  // the row in shared memory is read before the next token's
+  }
+}
+
 extern "C" int sb_conv_headnorm_store(const void* proj, int row_width, int dtype, const float* conv_w, int taps, float* state,
                                       const int* slots, int num_slots, int num_seqs, int alone, const float* q_norm,
                                       const float* k_norm, float eps, float q_scale, const float* rot_freq, int rot_dims,
@@ -611,6 +772,43 @@ extern "C" int sb_conv_headnorm_store(const void* proj, int row_width, int dtype
   const dim3 grid((unsigned)((num_tokens + rows - 1) / rows), (unsigned)((H + 2 * G + PREP_WARPS - 1) / PREP_WARPS));
   const size_t smem = ((size_t)rows * rot_dims + (size_t)PREP_WARPS * (d > dv ? d : dv)) * sizeof(float);
   if (smem > 200 * 1024 || grid.y > 65535) return -2;
+  // (in the activation dtype's pairs: rows, heads and the turned halves start on whole pairs)
+  const bool pairs = !alone && taps != 1 && taps <= 4 && d % 2 == 0 && dv % 2 == 0 && row_width % 2 == 0 &&
+                     (interleaved || rot_dims % 4 == 0) && d <= 256 && dv <= 256;
+  const int widest = d > dv ? d : dv;
+#define SB_PAIRS(T_, TAPS_, NCH_)                                                                                      \
+  do {                                                                                                                 \
+    auto k = conv_headnorm_store_pairs_kernel<T_, TAPS_, NCH_>;                                                        \
+    sb_launch(k, grid, PREP_WARPS * 32, smem, stream, (const T_*)proj, row_width, conv_w, (const float*)state, slots,  \
+              num_slots, q_norm, k_norm, eps, q_scale, rot_freq, rot_dims, interleaved, (T_*)q_out, (T_*)cache,        \
+              block_table, max_pages, token_seq, cu_q, positions, num_tokens, rows, H, G, d, dv, page_size, num_pages, \
+              write_cache, err);                                                                                       \
+  } while (0)
+#define SB_PAIRS_OF(T_, TAPS_)                          \
+  do {                                                  \
+    if (widest <= 64) SB_PAIRS(T_, TAPS_, 1);           \
+    else if (widest <= 128) SB_PAIRS(T_, TAPS_, 2);     \
+    else SB_PAIRS(T_, TAPS_, 4);                        \
+  } while (0)
+#define SB_PAIRS_ANY(T_)                          \
+  switch (taps) {                                 \
+    case 0: SB_PAIRS_OF(T_, 0); break;            \
+    case 2: SB_PAIRS_OF(T_, 2); break;            \
+    case 3: SB_PAIRS_OF(T_, 3); break;            \
+    default: SB_PAIRS_OF(T_, 4);                  \
+  }
+  if (pairs && smem <= 48 * 1024) {
+    if (dtype == SB_DTYPE_F32) {
+      SB_PAIRS_ANY(float)
+    } else {
+      SB_PAIRS_ANY(bf16)
+    }
+    SB_LAUNCH_CHECK();
+    return 0;
+  }
+#undef SB_PAIRS_ANY
+#undef SB_PAIRS_OF
+#undef SB_PAIRS
 #define SB_PREP2(T_, TAPS_)                                                                                          \
   do {                                                                                                               \
     auto k = conv_headnorm_store_kernel<T_, TAPS_>;                                                                  \

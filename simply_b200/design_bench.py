@@ -1,8 +1,8 @@
 """Prefill and decode throughput of a design beside the engine's closest other model at equal size
 (Generax beside Gemma 2, Sapivik beside Generax, Zesapel beside Sapivik, Nulezen beside Sapivik, Mononex beside
-Sapivik and Zesapel), and the time of every kernel call of one step of each with its share of the measured peaks.
+Sapivik and Zesapel, Pibulix beside Sapivik and Mononex), and the time of every kernel call of one step of each with its share of the measured peaks.
 
-Used by `bench.py --design generax|sapivik|zesapel|nulezen|mononex` (the default benchmark does not import this file).  Layer
+Used by `bench.py --design generax|sapivik|zesapel|nulezen|mononex|pibulix` (the default benchmark does not import this file).  Layer
 shapes resemble a real model's; weights are random.  Per size and design:
 
 * prefill: one 2,048-token prompt in one step, median of 5 after 3 warm-up steps, CUDA events;
@@ -142,6 +142,30 @@ def mononex_dict(s: dict) -> dict:
           "decay_rank": RANK, "max_context": 8192}
 
 
+def pibulix_dict(s: dict) -> dict:
+  """The Sapivik arm's arrangement: one layer in three is attention (here over a window, with four kept
+  first tokens and convolutions of four taps) with a dense feed-forward, the others recurrent with
+  sixteen experts of a quarter of the dense hidden size, four per token (in four groups of which
+  two are open) and a shared one; the first three layers' weights serve three more, as the other
+  arm's first three layers run twice."""
+  att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+         "softcap": 30.0, "conv": TAPS, "mask": {"size": WINDOW, "keep_first": 4},
+         "rot": {"dims": s["dim"] // 2, "base": 10000.0}}
+  rec = {"heads": s["heads"], "dim": s["dim"], "vdim": s["dim"], "tau": 16.0}
+  experts = {"kind": "moe", "expert": {"ff": s["ff"] // 4}, "shared": {"ff": s["ff"] // 4},
+             "router": {"experts": 16, "top": 4, "scale": 1.0, "groups": {"count": 4, "keep": 2}}}
+  layers = []
+  for i in range(s["layers"]):
+    if i % 3 == 0:
+      layers.append({"type": "attention", "mixer": dict(att), "mlp": {"kind": "dense", "ff": s["ff"]}})
+    else:
+      layers.append({"type": "gla", "mixer": dict(rec), "mlp": dict(experts)})
+    if i >= 3:
+      layers[-1]["weights_of"] = i - 3
+  return {"architecture": "Pibulix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "postln_alpha": 2.0,
+          "layers": layers, "decay_rank": RANK, "max_context": 8192}
+
+
 def gemma2_dict(s: dict) -> dict:
   return {"architectures": ["Gemma2ForCausalLM"], "hidden_size": s["width"], "num_hidden_layers": s["layers"],
           "num_attention_heads": s["heads"], "num_key_value_heads": s["kv_heads"], "head_dim": s["dim"],
@@ -196,7 +220,8 @@ class TimedOps:
         if args[3] is not None:
           flops = 2.0 * t_ * top_ * (args[3].shape[1] + args[4].shape[1]) * args[3].shape[2]
       if name in ("paged_attention", "project_rotate_store", "rope_and_cache_write", "qk_norm_rotate_store", "pool_blocks",
-                  "delta_rule_inputs", "gated_delta_scan", "rotate_headnorm_store", "forget_gate_scan", "latent_prepare"):
+                  "delta_rule_inputs", "gated_delta_scan", "rotate_headnorm_store", "forget_gate_scan", "latent_prepare",
+                  "conv_headnorm_rotate_store"):
         moved -= big if name != "delta_rule_inputs" else 0  # the cache (or state) storage is not read whole
       if name == "paged_attention" and ctx is not None:
         q = args[0]
@@ -209,15 +234,23 @@ class TimedOps:
           pos = np.arange(s0, s0 + n)
           chunk = kw.get("key_chunk")
           keys = pos % chunk + 1 if chunk else np.minimum(pos + 1, window)
+          kept = kw.get("keep_first") or 0
+          keys = keys + np.clip(pos + 1 - window, 0, kept)
           if kw.get("pooled") is not None:
             keys = keys + np.maximum(pos - window + 1, 0) // kw["pooled"][2]
           pairs += int(keys.sum())
           if chunk:
             seen += int(s0 + n - s0 // chunk * chunk)
             continue
-          seen += int(min(s0 + n, window + n)) + (int((s0 + n) // kw["pooled"][2]) if kw.get("pooled") is not None else 0)
+          seen += int(min(s0 + n, window + n + kept)) + (int((s0 + n) // kw["pooled"][2]) if kw.get("pooled") is not None else 0)
         flops = 2.0 * pairs * heads * (dim + vdim)
         moved += seen * kv_heads * (dim + (0 if kw.get("values_in_keys") else vdim)) * args[1].element_size()
+      if name == "conv_headnorm_rotate_store":  # keys and values go into pages
+        moved += args[0].shape[0] * kw["num_kv_heads"] * (kw["head_dim"] + kw["value_dim"]) * args[0].element_size()
+        if args[2] is not None:
+          moved += 2 * args[2][0].numel() * 4 * ctx.num_seqs - _nbytes(args[2])
+      if name == "norm_of_sum":  # the stream is read and written
+        moved += _nbytes(args[0])
       if name == "gated_delta_scan" and ctx is not None:
         state = args[5]
         per_slot = state[0].numel() * 4
@@ -291,9 +324,10 @@ def _prefill_ms(engine, tokens: int, vocab: int) -> float:
 
 
 PAIRS = {"generax": ("generax", "gemma2"), "sapivik": ("sapivik", "generax"), "zesapel": ("zesapel", "sapivik"),
-         "nulezen": ("nulezen", "sapivik"), "mononex": ("mononex", "sapivik", "zesapel")}
+         "nulezen": ("nulezen", "sapivik"), "mononex": ("mononex", "sapivik", "zesapel"),
+         "pibulix": ("pibulix", "sapivik", "mononex")}
 DICTS = {"generax": generax_dict, "gemma2": gemma2_dict, "sapivik": sapivik_dict, "zesapel": zesapel_dict,
-         "nulezen": nulezen_dict, "mononex": mononex_dict}
+         "nulezen": nulezen_dict, "mononex": mononex_dict, "pibulix": pibulix_dict}
 
 
 def run(args, peaks: dict, time_decode, design: str = "generax") -> dict:

@@ -109,13 +109,14 @@ def attend(q, k, v, m, first=0):
   for r in range(q.shape[0]):
     i = first + r
     seen = [j for j in range(i + 1) if sees(i, j, mask)]
+    k_seen, v_seen = k[seen], v[seen]
     for a in range(m["heads"]):
-      s = (k[seen, a // per] @ q[r, a]) * m["scale"]
+      s = (k_seen[:, a // per] @ q[r, a]) * m["scale"]
       if cap:
         s = cap * np.tanh(s / cap)
       top = max(float(s.max()), 0.0)
       e = np.exp(s - top)
-      out[r, a] = (e / (math.exp(-top) + e.sum())) @ v[seen, a // per]
+      out[r, a] = (e / (math.exp(-top) + e.sum())) @ v_seen[:, a // per]
   return out
 
 
