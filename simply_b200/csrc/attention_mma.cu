@@ -135,22 +135,15 @@ __device__ __forceinline__ float fast_tanh(float x) {
   asm("tanh.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
-// tanh z = 1 - 2 / (e^(2 z) + 1): its absolute error stays at a few 2^-24
-__device__ __forceinline__ float tanh_by_exp(float x) {
-  return 1.0f - __fdividef(2.0f, fast_exp2(x * (2.0f * LOG2E)) + 1.0f);
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
 }
-// |z| <= TANH_SMALL without the special-function pipe: z p(z^2), p the least-squares fit of tanh(z) / z in z^2 over
-// Chebyshev nodes (weighted with z); absolute error below 8e-8 in float32
-constexpr float TANH_SMALL = 0.75f;
-__device__ __forceinline__ float tanh_small(float x) {
-  const float y = x * x;
-  float p = fmaf(1.6347697408740994e-3f, y, -7.470196173116038e-3f);
-  p = fmaf(p, y, 2.132028146757693e-2f);
-  p = fmaf(p, y, -5.3848173879808225e-2f);
-  p = fmaf(p, y, 0.13331961800290978f);
-  p = fmaf(p, y, -0.3333326357338127f);
-  p = fmaf(p, y, 0.9999999896724786f);
-  return x * p;
+// cap tanh(s / cap) = cap - 2 cap / (e^(2 s / cap) + 1): the absolute error stays at a few 2^-24 of the cap
+// (tanh.approx: 2^-11).  `rate`: 2 log2(e) / cap.
+__device__ __forceinline__ float exact_cap_of(float s, float cap, float rate) {
+  return fmaf(-2.0f * cap, fast_rcp(fast_exp2(s * rate) + 1.0f), cap);
 }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -296,26 +289,11 @@ __device__ __forceinline__ float distance_loss(const RowBias& b, int d, int kind
 // The cap on a warp's scores to float32 accuracy, ahead of `softmax_pv` (which then gets no cap).
 template <int NKT>
 __device__ __forceinline__ void exact_caps(float (&s)[NKT][4], float cap) {
-  const float inv_cap = 1.0f / cap;
-  float big = 0.f;
+  const float rate = 2.0f * LOG2E / cap;
 #pragma unroll
   for (int i = 0; i < NKT; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      s[i][e] *= inv_cap;
-      big = fmaxf(big, fabsf(s[i][e]));
-    }
-  if (__any_sync(0xffffffffu, big > TANH_SMALL)) {
-#pragma unroll
-    for (int i = 0; i < NKT; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[i][e] = cap * tanh_by_exp(s[i][e]);
-  } else {
-#pragma unroll
-    for (int i = 0; i < NKT; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[i][e] = cap * tanh_small(s[i][e]);
-  }
+    for (int e = 0; e < 4; ++e) s[i][e] = exact_cap_of(s[i][e], cap, rate);
 }
 
 template <int NKT>
@@ -947,7 +925,7 @@ attn_decode8_kernel(const AttnParams p, int* work_counter, int total_work, const
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           float v = s0[e] + s1[e];
-          if (p.cap > 0.f) v = p.cap * (OPT && p.exact_cap ? tanh_by_exp(v * inv_cap) : fast_tanh(v * inv_cap));
+          if (p.cap > 0.f) v = OPT && p.exact_cap ? exact_cap_of(v, p.cap, 2.0f * LOG2E * inv_cap) : p.cap * fast_tanh(v * inv_cap);
           const int j = j_first + g + (e >> 1) * 8;
           const int pos = (e & 1) ? pos1 : pos0;
           if (biased) v -= distance_loss((e & 1) ? bias1 : bias0, pos - j, biased);
@@ -1290,7 +1268,7 @@ attn_decode8ws_kernel(const AttnParams p, int* work_counter, int total_work, con
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         float v = s0[e] + s1[e];
-        if (p.cap > 0.f) v = p.cap * (OPT && p.exact_cap ? tanh_by_exp(v * inv_cap) : fast_tanh(v * inv_cap));
+        if (p.cap > 0.f) v = OPT && p.exact_cap ? exact_cap_of(v, p.cap, 2.0f * LOG2E * inv_cap) : p.cap * fast_tanh(v * inv_cap);
         const int j = j_first + g + (e >> 1) * 8;
         const int pos = (e & 1) ? pos1 : pos0;
         if (biased) v -= distance_loss((e & 1) ? bias1 : bias0, pos - j, biased);

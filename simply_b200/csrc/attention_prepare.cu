@@ -474,6 +474,7 @@ extern "C" int sb_rotate_headnorm_store(const void* proj, int row_width, int dty
 // ---------------------------------------------------------------------------
 #define SB_ERR_BAD_SLOT 16
 constexpr int PREP_WARPS = 8;
+constexpr int PREP_ROWS = 8;  // most tokens of a block
 
 template <typename T, int TAPS>  // TAPS: 0 none, 2 .. 4, -1 any number
 __global__ void __launch_bounds__(PREP_WARPS * 32)
@@ -623,6 +624,8 @@ conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, cons
                                  const int* __restrict__ positions, int num_tokens, int rows_per_block, int H, int G, int d, int dv,
                                  int page_size, int num_pages, int write_cache, int* err) {
   extern __shared__ float prep_smem[];
+  // per token of the block: its place in its sequence's part of the step, its state slot, its page and place there
+  __shared__ int s_place[PREP_ROWS], s_slot[PREP_ROWS], s_page[PREP_ROWS], s_off[PREP_ROWS];
   const int half = rot_dims / 2, hd = max(d, dv);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int t0 = blockIdx.x * rows_per_block, rows = min(rows_per_block, num_tokens - t0);
@@ -646,6 +649,21 @@ conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, cons
   }
   pdl_wait_block();
   pdl_launch_dependents();
+  for (int r = threadIdx.x; r < rows; r += blockDim.x) {
+    const int t = t0 + r, b = token_seq[t], p = positions[t];
+    s_place[r] = t - cu_q[b];
+    const int slot = TAPS > 1 ? slots[b] : 0;
+    const bool bad_slot = TAPS > 1 && (slot < 0 || slot >= num_slots);
+    s_slot[r] = bad_slot ? -1 : slot;
+    int page = write_cache ? block_table[(size_t)b * max_pages + p / page_size] : 0;
+    if (page < 0 || page >= num_pages) {
+      if (write_cache && blockIdx.y == 0) atomicOr(err, SB_ERR_BAD_PAGE);
+      page = -1;
+    }
+    if (bad_slot && blockIdx.y == 0) atomicOr(err, SB_ERR_BAD_SLOT);
+    s_page[r] = page;
+    s_off[r] = p % page_size;
+  }
   for (int i = threadIdx.x; i < rows * half; i += blockDim.x) {
     const int r = i / half, a = i - r * half;
     sincosf((float)positions[t0 + r] * rot_freq[a], prep_smem + (2 * r + 1) * half + a, prep_smem + 2 * r * half + a);
@@ -655,15 +673,24 @@ conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, cons
   float* buf = prep_smem + 2 * rows_per_block * half + (size_t)warp * hd;
   const size_t page_stride = (size_t)G * page_size * (d + dv);
   float2 past[W][NCH];  // the rows before the token, oldest first (W - 1 of them)
+  float2 own[NCH], next[NCH];
+#pragma unroll
+  for (int k = 0; k < NCH; ++k) {
+    const int c = 2 * lane + 64 * k;
+    next[k] = c < n ? Pair<T>::load(proj + (size_t)t0 * row_width + c0 + c) : make_float2(0.f, 0.f);
+  }
 
   for (int r = 0; r < rows; ++r) {
-    const int t = t0 + r, b = token_seq[t];
-    const int i = t - cu_q[b];
+    const int t = t0 + r, i = s_place[r];
     const T* x = proj + (size_t)t * row_width + c0;
+#pragma unroll
+    for (int k = 0; k < NCH; ++k) {  // this token's row is there; the next one's is fetched meanwhile
+      const int c = 2 * lane + 64 * k;
+      own[k] = next[k];
+      if (r + 1 < rows && c < n) next[k] = Pair<T>::load(x + row_width + c);
+    }
     if (TAPS > 1 && (r == 0 || i == 0)) {
-      const int slot = slots[b];
-      const bool bad = slot < 0 || slot >= num_slots;
-      if (bad && lane == 0) atomicOr(err, SB_ERR_BAD_SLOT);
+      const int slot = s_slot[r];
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j) {
         const int at = i - (TAPS - 1) + j;
@@ -673,7 +700,7 @@ conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, cons
           float2 v = make_float2(0.f, 0.f);
           if (c < n) {
             if (at >= 0) v = Pair<T>::load(x + c - (long long)(TAPS - 1 - j) * row_width);
-            else if (!bad) v = Pair<float>::load(state + ((size_t)slot * (TAPS - 1) + TAPS - 1 + at) * channels + c0 + c);
+            else if (slot >= 0) v = Pair<float>::load(state + ((size_t)slot * (TAPS - 1) + TAPS - 1 + at) * channels + c0 + c);
           }
           past[j][k] = v;
         }
@@ -683,9 +710,7 @@ conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, cons
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < NCH; ++k) {
-      const int c = 2 * lane + 64 * k;
-      const float2 own = c < n ? Pair<T>::load(x + c) : make_float2(0.f, 0.f);
-      u[k] = own;
+      u[k] = own[k];
       if (TAPS > 0) {
         u[k] = make_float2(0.f, 0.f);
 #pragma unroll
@@ -693,27 +718,21 @@ conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, cons
           u[k].x = fmaf(w[j][k].x, past[j][k].x, u[k].x);
           u[k].y = fmaf(w[j][k].y, past[j][k].y, u[k].y);
         }
-        u[k].x = fmaf(w[W - 1][k].x, own.x, u[k].x);
-        u[k].y = fmaf(w[W - 1][k].y, own.y, u[k].y);
+        u[k].x = fmaf(w[W - 1][k].x, own[k].x, u[k].x);
+        u[k].y = fmaf(w[W - 1][k].y, own[k].y, u[k].y);
 #pragma unroll
         for (int j = 0; j + 2 < TAPS; ++j) past[j][k] = past[j + 1][k];
-        if (TAPS > 1) past[W > 1 ? W - 2 : 0][k] = own;
+        if (TAPS > 1) past[W > 1 ? W - 2 : 0][k] = own[k];
       }
       ss = fmaf(u[k].x, u[k].x, fmaf(u[k].y, u[k].y, ss));
     }
     T* dst = nullptr;
     if (is_q) {
       dst = q_out + ((size_t)t * H + head) * d;
-    } else if (write_cache) {
-      const int p = positions[t];
-      const long long page = block_table[(size_t)b * max_pages + p / page_size];
-      if (page < 0 || page >= num_pages) {
-        if (lane == 0) atomicOr(err, SB_ERR_BAD_PAGE);
-      } else if (is_v) {
-        dst = cache + page * page_stride + (size_t)G * page_size * d + ((size_t)(head - H - G) * page_size + p % page_size) * dv;
-      } else {
-        dst = cache + page * page_stride + ((size_t)(head - H) * page_size + p % page_size) * d;
-      }
+    } else if (write_cache && s_page[r] >= 0) {
+      T* page = cache + s_page[r] * page_stride;
+      dst = is_v ? page + (size_t)G * page_size * d + ((size_t)(head - H - G) * page_size + s_off[r]) * dv
+                 : page + ((size_t)(head - H) * page_size + s_off[r]) * d;
     }
     if (is_v) {
 #pragma unroll

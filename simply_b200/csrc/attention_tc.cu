@@ -106,22 +106,10 @@ __device__ __forceinline__ float fast_tanh(float x) {
   asm("tanh.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
-// tanh z = 1 - 2 / (e^(2 z) + 1): its absolute error stays at a few 2^-24
-__device__ __forceinline__ float tanh_by_exp(float x) {
-  return 1.0f - __fdividef(2.0f, fast_exp2(x * (2.0f * LOG2E)) + 1.0f);
-}
-// |z| <= TANH_SMALL without the special-function pipe: z p(z^2), p the least-squares fit of tanh(z) / z in z^2 over
-// Chebyshev nodes (weighted with z); absolute error below 8e-8 in float32
-constexpr float TANH_SMALL = 0.75f;
-__device__ __forceinline__ float tanh_small(float x) {
-  const float y = x * x;
-  float p = fmaf(1.6347697408740994e-3f, y, -7.470196173116038e-3f);
-  p = fmaf(p, y, 2.132028146757693e-2f);
-  p = fmaf(p, y, -5.3848173879808225e-2f);
-  p = fmaf(p, y, 0.13331961800290978f);
-  p = fmaf(p, y, -0.3333326357338127f);
-  p = fmaf(p, y, 0.9999999896724786f);
-  return x * p;
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
 }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -350,7 +338,9 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
     const int row_lo = lowest_key(p, pos), warp_lo = lowest_key(p, warp_pos_hi);  // the lowest keys seen
     const bool fast_cap = p.cap > 0.f && !p.exact_cap;
     const float inv_cap = p.cap > 0.f ? 1.0f / p.cap : 0.f;
-    const float scale2 = p.cap > 0.f ? p.cap * LOG2E : LOG2E;  // from x (tanh's value, or the score) to log2 units
+    // from x (tanh's value, or half of that less one, or the score) to log2 units
+    const float scale2 = p.cap > 0.f ? p.cap * LOG2E * (p.exact_cap ? 2.0f : 1.0f) : LOG2E;
+    const float exact_rate = 2.0f * LOG2E * inv_cap;
     // The distance bias of this thread's row: r1 ln 2 and r2 of its head.
     const bool biased = p.distance != nullptr;
     const bool tabled = p.bias_table != 0;
@@ -392,20 +382,11 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
       tmem_wait_load();
       const bool need_mask = !rows_full || j0 + BN - 1 > warp_pos_lo || j0 < warp_lo;
       if (p.exact_cap) {
-        float big = 0.f;
+        // cap tanh(s / cap) = cap - 2 cap r with r = 1 / (e^(2 s / cap) + 1), good to a few 2^-24 of the cap (tanh.approx: 2^-11):
+        // what follows works with -r, in units of 2 cap, and leaves out the constant
 #pragma unroll
-        for (int c = 0; c < CW; ++c) {
-          const float v = __uint_as_float(sr[c]) * inv_cap;
-          sr[c] = __float_as_uint(v);
-          big = fmaxf(big, fabsf(v));
-        }
-        if (__any_sync(0xffffffffu, big > TANH_SMALL)) {
-#pragma unroll
-          for (int c = 0; c < CW; ++c) sr[c] = __float_as_uint(tanh_by_exp(__uint_as_float(sr[c])));
-        } else {
-#pragma unroll
-          for (int c = 0; c < CW; ++c) sr[c] = __float_as_uint(tanh_small(__uint_as_float(sr[c])));
-        }
+        for (int c = 0; c < CW; ++c)
+          sr[c] = __float_as_uint(fast_rcp(-1.0f - fast_exp2(__uint_as_float(sr[c]) * exact_rate)));
       }
       float mx = -INFINITY;
       if (need_mask) {
@@ -546,7 +527,8 @@ attn_prefill_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap map
       l = 0.f;
 #pragma unroll
       for (int q = 0; q < GROUPS * SPLIT; ++q) l += row_sum[q][r];
-      if (p.sink != nullptr && r < rows_valid) l += fast_exp2(p.sink[head] * LOG2E - m_final);  // it has no value
+      if (p.sink != nullptr && r < rows_valid)  // it has no value
+        l += fast_exp2((p.sink[head] - (p.exact_cap ? p.cap : 0.f)) * LOG2E - m_final);
     }
     if (ok && !mbar_wait_bounded(&o_done, 0)) ok = false;
     tc_fence_after_sync();

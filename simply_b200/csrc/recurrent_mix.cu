@@ -930,7 +930,8 @@ gated_linear_inputs_kernel(const T* __restrict__ pre, int row_width, int low_off
     float z[TOKENS];
 #pragma unroll
     for (int i = 0; i < TOKENS; ++i) z[i] = bias[c];
-#pragma unroll 8
+    constexpr int AHEAD = TOKENS == 1 ? 32 : 8;  // (few blocks: a thread's own loads have to cover the latency)
+#pragma unroll AHEAD
     for (int r = 0; r < rank; ++r) {
       const float wr = w[(size_t)r * n_qf + c];
 #pragma unroll
