@@ -474,7 +474,6 @@ extern "C" int sb_rotate_headnorm_store(const void* proj, int row_width, int dty
 // ---------------------------------------------------------------------------
 #define SB_ERR_BAD_SLOT 16
 constexpr int PREP_WARPS = 8;
-constexpr int PREP_ROWS = 8;  // most tokens of a block
 
 template <typename T, int TAPS>  // TAPS: 0 none, 2 .. 4, -1 any number
 __global__ void __launch_bounds__(PREP_WARPS * 32)
@@ -598,7 +597,7 @@ conv_headnorm_store_kernel(const T* __restrict__ proj, int row_width, const floa
 }
 
 // The same for steps with prompt portions, two neighbouring channels per lane: the taps' weights of a warp's
-// head and its last rows stay in registers from token to token.  Heads of up to 64 * NCH channels, whole
+// head and all rows of a block stay in registers.  Heads of up to 64 * NCH channels, whole
 // pairs of channels everywhere (d, dv, the row width and half the turned dims are even).
 template <typename T> struct Pair;
 template <> struct Pair<float> {
@@ -613,7 +612,7 @@ template <> struct Pair<bf16> {
   __device__ static void store(bf16* p, float2 v) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v.x, v.y); }
 };
 
-template <typename T, int TAPS, int NCH>
+template <typename T, int TAPS, int NCH, int ROWS>
 __global__ void __launch_bounds__(PREP_WARPS * 32)
 conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, const float* __restrict__ conv_w,
                                  const float* __restrict__ state, const int* __restrict__ slots, int num_slots,
@@ -621,20 +620,20 @@ conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, cons
                                  const float* __restrict__ rot_freq, int rot_dims, int interleaved, T* __restrict__ q_out,
                                  T* __restrict__ cache, const int* __restrict__ block_table, int max_pages,
                                  const int* __restrict__ token_seq, const int* __restrict__ cu_q,
-                                 const int* __restrict__ positions, int num_tokens, int rows_per_block, int H, int G, int d, int dv,
+                                 const int* __restrict__ positions, int num_tokens, int H, int G, int d, int dv,
                                  int page_size, int num_pages, int write_cache, int* err) {
   extern __shared__ float prep_smem[];
   // per token of the block: its place in its sequence's part of the step, its state slot, its page and place there
-  __shared__ int s_place[PREP_ROWS], s_slot[PREP_ROWS], s_page[PREP_ROWS], s_off[PREP_ROWS];
+  __shared__ int s_place[ROWS], s_slot[ROWS], s_page[ROWS], s_off[ROWS];
   const int half = rot_dims / 2, hd = max(d, dv);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int t0 = blockIdx.x * rows_per_block, rows = min(rows_per_block, num_tokens - t0);
+  const int t0 = blockIdx.x * ROWS, rows = min(ROWS, num_tokens - t0);
   const int head = blockIdx.y * PREP_WARPS + warp;
   const bool on = head < H + 2 * G, is_q = head < H, is_v = head >= H + G;
   const int n = is_v ? dv : d;
   const int c0 = is_v ? (H + G) * d + (head - H - G) * dv : head * d;
   const int channels = (H + G) * d + G * dv;
-  constexpr int W = TAPS > 0 ? TAPS : 1;
+  constexpr int W = TAPS > 0 ? TAPS : 1, BACK = W - 1;  // rows before a token that it reads
   float2 w[W][NCH], scale[NCH];
   if (on) {  // (weights: before the wait)
     const float* scale_w = is_q ? q_norm : k_norm;
@@ -670,59 +669,37 @@ conv_headnorm_store_pairs_kernel(const T* __restrict__ proj, int row_width, cons
   }
   __syncthreads();
   if (!on) return;
-  float* buf = prep_smem + 2 * rows_per_block * half + (size_t)warp * hd;
+  float* buf = prep_smem + 2 * ROWS * half + (size_t)warp * hd;
   const size_t page_stride = (size_t)G * page_size * (d + dv);
-  float2 past[W][NCH];  // the rows before the token, oldest first (W - 1 of them)
-  float2 own[NCH], next[NCH];
+  // The block's rows and the BACK rows ahead of them, all under way at once (those of another sequence are not used).
+  float2 row[BACK + ROWS][NCH];
 #pragma unroll
-  for (int k = 0; k < NCH; ++k) {
-    const int c = 2 * lane + 64 * k;
-    next[k] = c < n ? Pair<T>::load(proj + (size_t)t0 * row_width + c0 + c) : make_float2(0.f, 0.f);
+  for (int a = 0; a < BACK + ROWS; ++a) {
+    const int t = t0 - BACK + a;
+#pragma unroll
+    for (int k = 0; k < NCH; ++k) {
+      const int c = 2 * lane + 64 * k;
+      row[a][k] = c < n && t >= 0 && t < num_tokens ? Pair<T>::load(proj + (size_t)t * row_width + c0 + c) : make_float2(0.f, 0.f);
+    }
   }
 
-  for (int r = 0; r < rows; ++r) {
-    const int t = t0 + r, i = s_place[r];
-    const T* x = proj + (size_t)t * row_width + c0;
 #pragma unroll
-    for (int k = 0; k < NCH; ++k) {  // this token's row is there; the next one's is fetched meanwhile
-      const int c = 2 * lane + 64 * k;
-      own[k] = next[k];
-      if (r + 1 < rows && c < n) next[k] = Pair<T>::load(x + row_width + c);
-    }
-    if (TAPS > 1 && (r == 0 || i == 0)) {
-      const int slot = s_slot[r];
-#pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) {
-        const int at = i - (TAPS - 1) + j;
-#pragma unroll
-        for (int k = 0; k < NCH; ++k) {
-          const int c = 2 * lane + 64 * k;
-          float2 v = make_float2(0.f, 0.f);
-          if (c < n) {
-            if (at >= 0) v = Pair<T>::load(x + c - (long long)(TAPS - 1 - j) * row_width);
-            else if (slot >= 0) v = Pair<float>::load(state + ((size_t)slot * (TAPS - 1) + TAPS - 1 + at) * channels + c0 + c);
-          }
-          past[j][k] = v;
-        }
-      }
-    }
+  for (int r = 0; r < ROWS; ++r) {
+    if (r >= rows) break;
+    const int t = t0 + r, i = s_place[r], slot = s_slot[r];
     float2 u[NCH];
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < NCH; ++k) {
-      u[k] = own[k];
-      if (TAPS > 0) {
-        u[k] = make_float2(0.f, 0.f);
+      const int c = 2 * lane + 64 * k;
+      u[k] = TAPS > 0 ? make_float2(0.f, 0.f) : row[BACK + r][k];
 #pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) {
-          u[k].x = fmaf(w[j][k].x, past[j][k].x, u[k].x);
-          u[k].y = fmaf(w[j][k].y, past[j][k].y, u[k].y);
-        }
-        u[k].x = fmaf(w[W - 1][k].x, own[k].x, u[k].x);
-        u[k].y = fmaf(w[W - 1][k].y, own[k].y, u[k].y);
-#pragma unroll
-        for (int j = 0; j + 2 < TAPS; ++j) past[j][k] = past[j + 1][k];
-        if (TAPS > 1) past[W > 1 ? W - 2 : 0][k] = own[k];
+      for (int j = 0; j < TAPS; ++j) {
+        float2 v = row[r + j][k];
+        if (i < BACK - j)  // before the step's first token of the sequence
+          v = c < n && slot >= 0 ? Pair<float>::load(state + ((size_t)slot * BACK + i + j) * channels + c0 + c) : make_float2(0.f, 0.f);
+        u[k].x = fmaf(w[j][k].x, v.x, u[k].x);
+        u[k].y = fmaf(w[j][k].y, v.y, u[k].y);
       }
       ss = fmaf(u[k].x, u[k].x, fmaf(u[k].y, u[k].y, ss));
     }
@@ -797,10 +774,14 @@ extern "C" int sb_conv_headnorm_store(const void* proj, int row_width, int dtype
   const int widest = d > dv ? d : dv;
 #define SB_PAIRS(T_, TAPS_, NCH_)                                                                                      \
   do {                                                                                                                 \
-    auto k = conv_headnorm_store_pairs_kernel<T_, TAPS_, NCH_>;                                                        \
+    if (rows == 4) SB_PAIRS_ROWS(T_, TAPS_, NCH_, 4); else SB_PAIRS_ROWS(T_, TAPS_, NCH_, 1);                          \
+  } while (0)
+#define SB_PAIRS_ROWS(T_, TAPS_, NCH_, ROWS_)                                                                                      \
+  do {                                                                                                                 \
+    auto k = conv_headnorm_store_pairs_kernel<T_, TAPS_, NCH_, ROWS_>;                                                        \
     sb_launch(k, grid, PREP_WARPS * 32, smem, stream, (const T_*)proj, row_width, conv_w, (const float*)state, slots,  \
               num_slots, q_norm, k_norm, eps, q_scale, rot_freq, rot_dims, interleaved, (T_*)q_out, (T_*)cache,        \
-              block_table, max_pages, token_seq, cu_q, positions, num_tokens, rows, H, G, d, dv, page_size, num_pages, \
+              block_table, max_pages, token_seq, cu_q, positions, num_tokens, H, G, d, dv, page_size, num_pages,       \
               write_cache, err);                                                                                       \
   } while (0)
 #define SB_PAIRS_OF(T_, TAPS_)                          \
@@ -828,6 +809,7 @@ extern "C" int sb_conv_headnorm_store(const void* proj, int row_width, int dtype
 #undef SB_PAIRS_ANY
 #undef SB_PAIRS_OF
 #undef SB_PAIRS
+#undef SB_PAIRS_ROWS
 #define SB_PREP2(T_, TAPS_)                                                                                          \
   do {                                                                                                               \
     auto k = conv_headnorm_store_kernel<T_, TAPS_>;                                                                  \

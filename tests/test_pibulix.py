@@ -160,6 +160,33 @@ def test_long_prompts_pages_of_64_and_sizes_of_the_tensor_core_kernels(dtype):
   engine.ops.check_errors()
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_step_of_more_than_a_thousand_tokens(dtype):
+  """Enough tokens for blocks that serve several tokens and for experts one by one; two requests in one step, then
+  single tokens and a second long portion."""
+  cfg_dict = px.config(
+      [px.attention(heads=8, kv_heads=2, dim=64, vdim=64, window=300, keep_first=5, dims=32, base=1e4, softcap=12.0, scale=0.2),
+       px.gla(heads=2, dim=64, vdim=32), px.attention(heads=3, kv_heads=1, dim=32, vdim=48, window=90, keep_first=70, dims=16, conv=4), 1],
+      [px.moe(ff=64, experts=4, top=4, groups=(2, 2), shared=32), px.dense(64), px.moe(ff=32, experts=3, top=3, groups=None), None],
+      width=64, vocab=300)  # (every expert is chosen: no close calls)
+  cfg, t = px.weights(cfg_dict, seed=3)
+  engine = px.build_engine(cfg, t, dtype, "cuda", None, page_size=64, slots=2, max_seq_len=2560, poison=True)
+  requests = [random_tokens(cfg_dict, n, i) for i, n in enumerate((2450, 143))]
+  w = px.as_numpy(t)
+  want = [plain.forward(cfg_dict, w, r) for r in requests]
+  slots, got, at = [engine.open_request() for _ in requests], [[], []], [0, 0]
+  for portions in ((1301, 61), (2, 1), (1, 1), (1, 80), (1145, 0)):
+    entries = [StepEntry(slots[i], requests[i][at[i]:at[i] + n], tuple(range(n))) for i, n in enumerate(portions) if n]
+    rows = engine.step_raw(entries).float().cpu().numpy()
+    for i, n in enumerate(portions):
+      got[i].append(rows[:n])
+      rows, at[i] = rows[n:], at[i] + n
+  for i in range(2):
+    px.check_close(np.concatenate(got[i]), want[i], dtype, f"request {i}")
+  engine.ops.check_errors()
+
+
 @pytest.mark.parametrize("where", WHERE)
 def test_many_query_heads_per_kv_head(where):
   """32 and 12 query heads per kv head: a single token's rows no longer fit the split-key kernel's

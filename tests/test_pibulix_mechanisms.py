@@ -113,6 +113,59 @@ def test_convolved_heads_are_normed_turned_and_stored(heads, kv_heads, d, dv, ta
     ops.check_errors()
 
 
+@pytest.mark.parametrize("where", WHERE)
+@pytest.mark.parametrize("heads,kv_heads,d,dv,taps", [(5, 1, 64, 64, 3), (4, 2, 128, 128, 4), (2, 1, 24, 40, 2), (2, 1, 256, 192, 4),
+                                                      (3, 1, 32, 16, 0), (2, 2, 7, 9, 3), (2, 1, 16, 16, 5)])
+def test_convolved_heads_of_a_long_step(heads, kv_heads, d, dv, taps, where):
+  """Well over a thousand tokens in one step, where a block serves several: requests begin and end inside one."""
+  ops, dtype = table(where)
+  device = where[1]
+  rng = np.random.default_rng(2)
+  counts, before, page = [7, 1061, 1, 2, 70, 1, 3], [5, 9, 0, 1, 0, 4, 2], 64
+  dims = d // 4 * 2 if d % 4 == 0 else 2
+  channels = heads * d + kv_heads * (d + dv)
+  manager = CacheManager({"c": PagedKVNeed(kv_heads, d, None, value_dim=None if dv == d else dv)}, page_size=page, max_slots=7,
+                         max_seq_len=1152, max_cache_tokens=7 * 1152, dtype=dtype, device=device)
+  conv = rng.standard_normal((taps, channels)) * 0.5 if taps else None
+  conv_t = f32(conv, device) if taps else None
+  scale, freq = rng.uniform(0.5, 1.5, d), rotation_frequencies(dims, 5000.0)
+  pre = [held(rng.standard_normal((b + n, channels)), dtype, device) for b, n in zip(before, counts)]
+  state = torch.zeros((7, max(taps - 1, 1), channels), device=device)
+  for i, b in enumerate(before):
+    assert manager.acquire_slot(i) == i
+    if b:
+      manager.extend([(i, b)])
+    for r in range(taps - 1):
+      if b - (taps - 1) + r >= 0:
+        state[i, r] = pre[i][0][b - (taps - 1) + r].float()
+  manager.extend(list(enumerate(counts)))
+  ctx = context(ops, device, before, counts, tables=[g.tables for g in manager.groups], page_size=page)
+  x = torch.cat([pre[i][0][b:] for i, b in enumerate(before)]).contiguous()
+  storage = manager.paged["c"].storage
+  q = f64(ops.conv_headnorm_rotate_store(
+      x, conv_t, state if taps > 1 else None, f32(scale, device), f32(scale, device), 1e-4, 0.5, torch.from_numpy(freq).to(device),
+      interleaved=False, num_heads=heads, num_kv_heads=kv_heads, head_dim=d, value_dim=dv, storage=storage,
+      block_table=ctx.block_tables[0], ctx=ctx)).reshape(-1, heads, d)
+  flat = storage.view(storage.shape[0], -1)
+  keys = f64(flat[:, :kv_heads * page * d]).reshape(-1, kv_heads, page, d)
+  values = f64(flat[:, kv_heads * page * d:]).reshape(-1, kv_heads, page, dv)
+  at, scale64 = 0, f64(f32(scale, "cpu"))
+  for i, (b, n) in enumerate(zip(before, counts)):
+    u = plain.short_convolution(pre[i][1], f64(conv_t).T) if taps else pre[i][1]
+    pos = np.arange(b + n, dtype=np.float64)
+    turned = lambda lo, hh: plain.turn_halves(plain.unit_rms(u[:, lo:lo + hh * d].reshape(-1, hh, d), 1e-4) * scale64, pos, dims, 5000.0)[b:]
+    close(q[at:at + n], turned(0, heads) * 0.5, dtype, f"queries of request {i}", f32=1e-4)
+    rows = [(manager.groups[0].tables[i, p // page], p % page) for p in range(b, b + n)]
+    close(np.stack([keys[r, :, o] for r, o in rows]), turned(heads * d, kv_heads), dtype, f"keys of request {i}", f32=1e-4)
+    close(np.stack([values[r, :, o] for r, o in rows]), u[b:, (heads + kv_heads) * d:].reshape(n, kv_heads, dv), dtype, f"values of request {i}")
+    if taps > 1:
+      tail = np.concatenate([np.zeros((taps, channels)), pre[i][1]])[-(taps - 1):]
+      close(f64(state[i]), tail, torch.float32, f"state of request {i}")
+    at += n
+  if device == "cuda":
+    ops.check_errors()
+
+
 @pytest.mark.gpu
 @pytest.mark.parametrize("copies", [1, 3])
 def test_rows_that_repeat_a_request_get_what_its_first_row_gets(copies):
