@@ -169,7 +169,7 @@ def test_a_step_of_more_than_a_thousand_tokens(dtype):
       [px.attention(heads=8, kv_heads=2, dim=64, vdim=64, window=300, keep_first=5, dims=32, base=1e4, softcap=12.0, scale=0.2),
        px.gla(heads=2, dim=64, vdim=32), px.attention(heads=3, kv_heads=1, dim=32, vdim=48, window=90, keep_first=70, dims=16, conv=4), 1],
       [px.moe(ff=64, experts=4, top=4, groups=(2, 2), shared=32), px.dense(64), px.moe(ff=32, experts=3, top=3, groups=None), None],
-      width=64, vocab=300)  # (every expert is chosen: no close calls)
+      width=64, vocab=300, max_context=4096)  # (every expert is chosen: no close calls)
   cfg, t = px.weights(cfg_dict, seed=3)
   engine = px.build_engine(cfg, t, dtype, "cuda", None, page_size=64, slots=2, max_seq_len=2560, poison=True)
   requests = [random_tokens(cfg_dict, n, i) for i, n in enumerate((2450, 143))]
